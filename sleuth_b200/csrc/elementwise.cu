@@ -265,17 +265,39 @@ __global__ void stream_inject_kernel(float* __restrict__ x, const float* __restr
   }
 }
 
+// Sine and cosine of the angle that `turns` whole turns a position make at position p. The fraction of a turn is taken in
+// 64-bit, so the angle keeps its accuracy however far the position.
+__device__ __forceinline__ void place_pair(double turns, double p, float& s, float& c) {
+  const double t = turns * p;
+  sincospif(2.0f * (float)(t - rint(t)), &s, &c);
+}
+
+// x[t, 2i] += sin(a), x[t, 2i + 1] += cos(a), a = 2 pi * turns[i] * position of token t. A block per token.
+__global__ void sinusoid_add_kernel(float* __restrict__ x, const int* __restrict__ tok_pos, const double* __restrict__ turns,
+                                    int dim) {
+  pdl_enter();
+  const double p = (double)tok_pos[blockIdx.x];
+  float* row = x + (size_t)blockIdx.x * dim;
+  for (int k = threadIdx.x; 2 * k < dim; k += blockDim.x) {
+    float s, c;
+    place_pair(turns[k], p, s, c);
+    row[2 * k] += s;
+    if (2 * k + 1 < dim) row[2 * k + 1] += c;
+  }
+}
+
 // A hashed table of token pairs added to the embedding: x[t, :] += pairs[row(t), :] with
 // row = (previous token * mul_prev + token * mul_cur) mod buckets, and row = buckets (the table's last row) for a
 // sequence's first token. With `table` the token's own row comes in the same pass: x[t, :] = table[token, :] * scale +
-// pairs[row(t), :]. The previous token of a step's first token comes from last[slot], the sequence's state; the
-// block of that token then leaves the step's last token there for the next step (it alone reads and writes the entry).
+// pairs[row(t), :]; with `turns` the position vector of sinusoid_add_kernel joins as well. The previous token of a
+// step's first token comes from last[slot], the sequence's state; the block of that token then leaves the step's last
+// token there for the next step (it alone reads and writes the entry).
 template <typename TW>
 __global__ void pair_embed_kernel(const int* __restrict__ ids, const int* __restrict__ map, const TW* __restrict__ pairs,
                                   float* __restrict__ x, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                                   const int* __restrict__ seq_start, const int* __restrict__ slots, int* __restrict__ last,
                                   int dim, int vocab, int buckets, long long mul_prev, long long mul_cur,
-                                  const TW* __restrict__ table, float scale) {
+                                  const TW* __restrict__ table, float scale, const double* __restrict__ turns) {
   pdl_enter();
   const int t = blockIdx.x;
   const int seq = tok_seq[t];
@@ -291,7 +313,17 @@ __global__ void pair_embed_kernel(const int* __restrict__ ids, const int* __rest
   }
   const TW* src = pairs + (size_t)row * dim;
   float* out = x + (size_t)t * dim;
-  if (table) {
+  if (turns) {
+    const TW* own = table ? table + (size_t)tok * dim : nullptr;
+    const double p = (double)tok_pos[t];
+    for (int k = threadIdx.x; 2 * k < dim; k += blockDim.x) {
+      float s, c;
+      place_pair(turns[k], p, s, c);
+      const int i = 2 * k;
+      out[i] = (own ? fmaf(to_f32(own[i]), scale, to_f32(src[i])) : out[i] + to_f32(src[i])) + s;
+      if (i + 1 < dim) out[i + 1] = (own ? fmaf(to_f32(own[i + 1]), scale, to_f32(src[i + 1])) : out[i + 1] + to_f32(src[i + 1])) + c;
+    }
+  } else if (table) {
     const TW* own = table + (size_t)tok * dim;
     for (int i = threadIdx.x; i < dim; i += blockDim.x) out[i] = fmaf(to_f32(own[i]), scale, to_f32(src[i]));
   } else {
@@ -630,7 +662,7 @@ extern "C" int slb_stream_inject(float* x, const float* again, const float* row,
 extern "C" int slb_pair_embed(const int* ids, const int* map, const void* pairs, int table_dtype, float* x, const int* tok_seq,
                               const int* tok_pos, const int* seq_start, const int* slots, int* last, int tokens, int dim,
                               int vocab, int buckets, long long mul_prev, long long mul_cur, const void* table, float scale,
-                              void* stream) {
+                              const double* turns, void* stream) {
   SLB_REQUIRE(tokens >= 0 && dim > 0 && vocab > 0 && buckets > 0, "pair_embed: tokens=%d dim=%d vocab=%d buckets=%d", tokens, dim,
               vocab, buckets);
   SLB_REQUIRE(mul_prev >= 0 && mul_cur >= 0 && mul_prev < (1LL << 31) && mul_cur < (1LL << 31), "pair_embed: multipliers %lld, %lld",
@@ -640,13 +672,20 @@ extern "C" int slb_pair_embed(const int* ids, const int* map, const void* pairs,
   const int threads = dim >= 256 ? 256 : 64;
   if (table_dtype == kF32)
     launch(pair_embed_kernel<float>, dim3(tokens), dim3(threads), 0, s, ids, map, (const float*)pairs, x, tok_seq, tok_pos, seq_start,
-           slots, last, dim, vocab, buckets, mul_prev, mul_cur, (const float*)table, scale);
+           slots, last, dim, vocab, buckets, mul_prev, mul_cur, (const float*)table, scale, turns);
   else if (table_dtype == kBF16)
     launch(pair_embed_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, s, ids, map, (const __nv_bfloat16*)pairs, x, tok_seq,
-           tok_pos, seq_start, slots, last, dim, vocab, buckets, mul_prev, mul_cur, (const __nv_bfloat16*)table, scale);
+           tok_pos, seq_start, slots, last, dim, vocab, buckets, mul_prev, mul_cur, (const __nv_bfloat16*)table, scale, turns);
   else
     return fail(1, "pair_embed: unknown dtype %d", table_dtype);
   return check_launch("pair_embed");
+}
+
+extern "C" int slb_sinusoid_add(float* x, const int* tok_pos, const double* turns, int tokens, int dim, void* stream) {
+  SLB_REQUIRE(tokens >= 0 && dim > 0, "sinusoid_add: tokens=%d dim=%d", tokens, dim);
+  if (tokens == 0) return 0;
+  launch(sinusoid_add_kernel, dim3(tokens), dim3(dim >= 512 ? 256 : 64), 0, (cudaStream_t)stream, x, tok_pos, turns, dim);
+  return check_launch("sinusoid_add");
 }
 
 extern "C" int slb_gated_norm_add(float* x, float* y, const float* g, long long g_stride, const float* b, const float* w,

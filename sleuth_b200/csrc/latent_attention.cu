@@ -16,6 +16,7 @@
 //   head_prompt_mma_kernel  whole prompts (every sequence starts at 0): per-head keys and values formed from the step's
 //                         latents by one product, then ordinary causal attention per head on the tensor cores
 //   latent_gate_kernel    y[t, h, :] = value[h, t, :] * sigmoid(g[t, h, :])
+// The three attention kernels take an optional sink per head: a learned score that joins the softmax denominator.
 #include "mma_sync.cuh"
 
 namespace slb {
@@ -73,6 +74,18 @@ __global__ void latent_post_kernel(const float* __restrict__ lat, const float* _
   }
 }
 
+// What a row's weighted sum is multiplied by when its last key is done: one over the mass, with the head's sink (a score
+// without key and value, unscaled) joined to the maximum and the mass here, once. `m` is the running maximum in units of
+// e, `l` the mass relative to it.
+__device__ __forceinline__ float row_factor(float m, float l, const float* __restrict__ sinks, int head) {
+  if (sinks == nullptr) return l > 0.f ? 1.0f / l : 0.f;
+  const float sink = sinks[head], top = fmaxf(m, sink);
+  const float f = expf(m - top);
+  return f / (l * f + expf(sink - top));
+}
+
+constexpr float kLn2 = 0.6931471805599453f;
+
 struct LatentAttnArgs {
   const void* q_lat;      // [H, T, R]
   const void* q_raw;      // [T, H, dn + P]; the rotated part starts at dn
@@ -85,6 +98,7 @@ struct LatentAttnArgs {
   const int* past;
   const int* counts;
   const int* table;
+  const float* sinks;     // [H], or null: no sink
   int stride, T, H, R, P, dn, rot, window, splits, chunk, tq, hb, kstride;
   float scale;
 };
@@ -266,7 +280,7 @@ __global__ void __launch_bounds__(kLatWarps * 32) latent_attn_kernel(const Laten
     const int row = warp * kLatRowsPerWarp + r;
     const int tok = tok0 + row / a.hb, h = h0 + row % a.hb;
     if (a.splits == 1) {
-      const float inv = l[r] > 0.f ? 1.0f / l[r] : 0.f;
+      const float inv = row_factor(m[r], l[r], a.sinks, h);
       T* o = (T*)a.out + ((size_t)h * a.T + tok) * a.R;
 #pragma unroll
       for (int i = 0; i < RV; ++i) {
@@ -483,7 +497,7 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(const LatentAttnAr
     const int row = warp * 16 + g + 8 * h;
     const int tok = tok0 + row / a.hb, head = h0 + row % a.hb;
     if (a.splits == 1) {
-      const float inv = l_r[h] > 0.f ? 1.0f / l_r[h] : 0.f;
+      const float inv = row_factor(m_r[h] * kLn2, l_r[h], a.sinks, head);
       __nv_bfloat16* dst = (__nv_bfloat16*)a.out + ((size_t)head * a.T + tok) * a.R;
 #pragma unroll
       for (int i = 0; i < 2 * NTM; ++i) {
@@ -502,7 +516,7 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(const LatentAttnAr
         }
       }
       if (grp == 0 && t4 == 0) {
-        dst[a.R] = m_r[h] == -INFINITY ? -INFINITY : m_r[h] * 0.6931471805599453f;      // the merge works with e, not 2
+        dst[a.R] = m_r[h] == -INFINITY ? -INFINITY : m_r[h] * kLn2;      // the merge works with e, not 2
         dst[a.R + 1] = l_r[h];
       }
     }
@@ -525,6 +539,7 @@ struct HeadPromptArgs {
   const float* sin_t;
   const int* seq_start;
   const int* counts;
+  const float* sinks;            // [H], or null: no sink
   int T, H, dn, P, dv, rot, window;
   float scale;
 };
@@ -742,7 +757,7 @@ __global__ void __launch_bounds__(128, NV <= 8 ? 3 : 2) head_prompt_mma_kernel(c
 #pragma unroll
   for (int hh = 0; hh < 2; ++hh) {
     if (pos_r[hh] < 0) continue;
-    const float inv = l_r[hh] > 0.f ? 1.0f / l_r[hh] : 0.f;
+    const float inv = row_factor(m_r[hh] * kLn2, l_r[hh], a.sinks, h);
     __nv_bfloat16* dst = a.out + ((size_t)h * a.T + tok0 + pos_r[hh]) * a.dv;
 #pragma unroll
     for (int i = 0; i < 2 * NV; ++i)
@@ -755,7 +770,7 @@ __global__ void __launch_bounds__(128, NV <= 8 ? 3 : 2) head_prompt_mma_kernel(c
 // columns over the slices in slice order.
 template <typename T>
 __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ parts, T* __restrict__ out, int rows, int Tn,
-                                                           int H, int R, int splits) {
+                                                           int H, int R, int splits, const float* __restrict__ sinks) {
   pdl_enter();
   __shared__ float factor[64];
   const int row = blockIdx.x;
@@ -764,7 +779,8 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
     const int lane = threadIdx.x;
     float m0 = lane < splits ? parts[((size_t)lane * rows + row) * (R + 2) + R] : -INFINITY;
     float m1 = lane + 32 < splits ? parts[((size_t)(lane + 32) * rows + row) * (R + 2) + R] : -INFINITY;
-    const float mx = warp_max(fmaxf(m0, m1));
+    float mx = warp_max(fmaxf(m0, m1));
+    if (sinks != nullptr) mx = fmaxf(mx, sinks[h]);      // the sink joins once, here, whatever the number of slices
     float f0 = m0 == -INFINITY ? 0.f : expf(m0 - mx), f1 = m1 == -INFINITY ? 0.f : expf(m1 - mx);
     float l0 = lane < splits ? parts[((size_t)lane * rows + row) * (R + 2) + R + 1] : 0.f;
     float l1 = lane + 32 < splits ? parts[((size_t)(lane + 32) * rows + row) * (R + 2) + R + 1] : 0.f;
@@ -774,7 +790,10 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
     __syncwarp();
     float mass = 0.f;
     if (lane == 0)
+    {
       for (int s = 0; s < splits; ++s) mass += factor[s];
+      if (sinks != nullptr) mass += expf(sinks[h] - mx);
+    }
     mass = __shfl_sync(0xffffffffu, mass, 0);
     const float inv = mass > 0.f ? 1.0f / mass : 0.f;
     __syncwarp();
@@ -910,7 +929,7 @@ extern "C" int slb_latent_attention(const void* q_lat, const void* q_raw, const 
                                     const float* cos_t, const float* sin_t, const int* seq_start, const int* past,
                                     const int* counts, const int* table, int stride, int n_seqs, int max_count, int T,
                                     int H, int R, int P, int dn, int rot, int window, float scale, int splits,
-                                    int dtype, void* stream) {
+                                    const float* sinks, int dtype, void* stream) {
   SLB_REQUIRE(n_seqs >= 0 && max_count >= 0 && T >= 0 && H > 0 && R > 0 && P >= 0 && dn >= 0 && rot >= 0 && rot <= P &&
                   rot % 2 == 0 && splits >= 1 && window >= 0,
               "latent_attention: seqs=%d max=%d heads=%d rank=%d rot_dim=%d splits=%d", n_seqs, max_count, H, R, P, splits);
@@ -922,6 +941,7 @@ extern "C" int slb_latent_attention(const void* q_lat, const void* q_raw, const 
   a.q_lat = q_lat; a.q_raw = q_raw; a.pool = pool; a.out = out; a.parts = parts; a.cos_t = cos_t; a.sin_t = sin_t;
   a.seq_start = seq_start; a.past = past; a.counts = counts; a.table = table; a.stride = stride; a.T = T; a.H = H;
   a.R = R; a.P = P; a.dn = dn; a.rot = rot; a.window = window; a.splits = splits; a.scale = scale;
+  a.sinks = sinks;
   cudaStream_t s = (cudaStream_t)stream;
   const bool aligned = ((uintptr_t)q_lat | (uintptr_t)q_raw | (uintptr_t)pool | (uintptr_t)out) % 16 == 0;
   if (dtype == kBF16 && R % 16 == 0 && (R + P) % 16 == 0 && aligned && (size_t)128 * (R + P + 8) * 2 <= kLatMaxSmem &&
@@ -952,7 +972,7 @@ extern "C" int slb_latent_attention(const void* q_lat, const void* q_raw, const 
     if (rc || splits == 1) return rc;
     const int rows = T * H;
     launch(latent_merge_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, s, (const float*)parts,
-           (__nv_bfloat16*)out, rows, T, H, R, splits);
+           (__nv_bfloat16*)out, rows, T, H, R, splits, sinks);
     return check_launch("latent_merge");
   }
   size_t bytes;
@@ -987,10 +1007,11 @@ extern "C" int slb_latent_attention(const void* q_lat, const void* q_raw, const 
   if (rc || splits == 1) return rc;
   const int rows = T * H;
   if (dtype == kF32)
-    launch(latent_merge_kernel<float>, dim3(rows), dim3(128), 0, s, (const float*)parts, (float*)out, rows, T, H, R, splits);
+    launch(latent_merge_kernel<float>, dim3(rows), dim3(128), 0, s, (const float*)parts, (float*)out, rows, T, H, R, splits,
+           sinks);
   else
     launch(latent_merge_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, s, (const float*)parts,
-           (__nv_bfloat16*)out, rows, T, H, R, splits);
+           (__nv_bfloat16*)out, rows, T, H, R, splits, sinks);
   return check_launch("latent_merge");
 }
 
@@ -1004,7 +1025,7 @@ extern "C" int slb_head_prompt_supported(int dn, int P, int dv) {
 extern "C" int slb_head_prompt_attention(const void* q, const void* kv, const void* k_rot, void* out, const float* cos_t,
                                          const float* sin_t, const int* seq_start, const int* counts, int n_seqs,
                                          int max_count, int T, int H, int dn, int P, int dv, int rot, int window,
-                                         float scale, void* stream) {
+                                         float scale, const float* sinks, void* stream) {
   SLB_REQUIRE(slb_head_prompt_supported(dn, P, dv), "head_prompt_attention: head sizes %d + %d, %d are not taken", dn, P, dv);
   SLB_REQUIRE(n_seqs >= 0 && max_count >= 0 && T >= 0 && H > 0 && rot >= 0 && rot <= P && rot % 2 == 0 && window >= 0,
               "head_prompt_attention: seqs=%d max=%d heads=%d", n_seqs, max_count, H);
@@ -1015,6 +1036,7 @@ extern "C" int slb_head_prompt_attention(const void* q, const void* kv, const vo
   a.q = (const __nv_bfloat16*)q; a.kv = (const __nv_bfloat16*)kv; a.k_rot = (const __nv_bfloat16*)k_rot;
   a.out = (__nv_bfloat16*)out; a.cos_t = cos_t; a.sin_t = sin_t; a.seq_start = seq_start; a.counts = counts;
   a.T = T; a.H = H; a.dn = dn; a.P = P; a.dv = dv; a.rot = rot; a.window = window; a.scale = scale;
+  a.sinks = sinks;
   // two key buffers where four blocks still fit an SM's shared memory with them, else one
   const size_t smem2 = (size_t)(192 * (dn + P + 8) + 128 * (dv + 8)) * 2, smem1 = (size_t)(128 * (dn + P + 8) + 64 * (dv + 8)) * 2;
   const int nbuf = smem2 * 3 <= kLatMaxSmem ? 2 : 1;

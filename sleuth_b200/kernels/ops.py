@@ -138,12 +138,13 @@ def stream_inject(x: torch.Tensor, again: torch.Tensor | None, row: torch.Tensor
 
 
 def pair_embed(ids, ids_map, pairs, x, tok_seq, tok_pos, seq_start, slots, last, vocab: int, buckets: int, mul_prev: int,
-               mul_cur: int, stream=None, table=None, scale: float = 1.0) -> None:
+               mul_cur: int, stream=None, table=None, scale: float = 1.0, turns=None) -> None:
     """x[t] += pairs[(previous token * mul_prev + token * mul_cur) mod buckets], or pairs[buckets] for a sequence's first
     token. ``pairs`` [buckets + 1, dim]; ``last`` int32 [slots]: every sequence's last token so far, read for the first
     token of a step and left for the next step. With ``table`` [vocab, dim] (of ``pairs``' dtype) the token's own row comes
-    in the same pass: x[t] = table[token] * scale + the pair's row."""
-    _cuda(ids, ids_map, pairs, x, tok_seq, tok_pos, seq_start, slots, last, table)
+    in the same pass: x[t] = table[token] * scale + the pair's row. With ``turns`` (float64 [(dim + 1) // 2], see
+    ``sinusoid_add``) the position vector is added too."""
+    _cuda(ids, ids_map, pairs, x, tok_seq, tok_pos, seq_start, slots, last, table, turns)
     T, d = x.shape
     _need(x.dtype == torch.float32 and pairs.dtype in DT and tuple(pairs.shape) == (buckets + 1, d), "pair_embed: table or stream")
     _need(last.dtype == torch.int32 and last.dim() >= 1 and ids.dtype == torch.int32, "pair_embed: int32 ids and state")
@@ -151,9 +152,20 @@ def pair_embed(ids, ids_map, pairs, x, tok_seq, tok_pos, seq_start, slots, last,
     _need(table is None or (table.dtype == pairs.dtype and tuple(table.shape) == (vocab, d)), "pair_embed: the token table")
     for t in (tok_seq, tok_pos, seq_start, slots):
         _need(t.dtype == torch.int32, "pair_embed: the batch tables are int32")
+    _need(turns is None or (turns.dtype == torch.float64 and turns.numel() == (d + 1) // 2), "pair_embed: turns of the position vector")
     lib().call("slb_pair_embed", _p(ids), _p(ids_map), _p(pairs), DT[pairs.dtype], _p(x), _p(tok_seq), _p(tok_pos), _p(seq_start),
                _p(slots), _p(last), T, d, int(vocab), int(buckets), int(mul_prev), int(mul_cur), _p(table), float(scale),
-               stream if stream is not None else current_stream())
+               _p(turns), stream if stream is not None else current_stream())
+
+
+def sinusoid_add(x, tok_pos, turns, stream=None) -> None:
+    """x[t, 2i] += sin(a), x[t, 2i + 1] += cos(a) with a = 2 pi * turns[i] * tok_pos[t]; ``turns`` float64
+    [(dim + 1) // 2]. The fraction of a turn is taken in 64-bit, its sine and cosine in float32."""
+    _cuda(x, tok_pos, turns)
+    T, d = x.shape
+    _need(x.dtype == torch.float32 and tok_pos.dtype == torch.int32 and tok_pos.numel() >= T, "sinusoid_add: stream or positions")
+    _need(turns.dtype == torch.float64 and turns.numel() == (d + 1) // 2, "sinusoid_add: turns of the position vector")
+    lib().call("slb_sinusoid_add", _p(x), _p(tok_pos), _p(turns), T, d, stream if stream is not None else current_stream())
 
 
 def gated_norm_add(x, y, g, bias, gain, eps: float, stream=None) -> None:
@@ -935,11 +947,13 @@ def latent_scratch_floats(tokens: int, heads: int, rank: int, splits: int) -> in
 
 def latent_attention(q_lat, q_raw, pool, out, cos, sin, seq_start, past, counts, block_table, max_count: int,
                      heads: int, rank: int, rot_dim: int, plain_dim: int, rotated: int, window: int, scale: float,
-                     splits: int = 1, scratch=None, stream=None) -> None:
+                     splits: int = 1, scratch=None, stream=None, sinks=None) -> None:
     """Causal softmax attention of every head over the latent cache rows. q_lat [heads, T, rank]: the queries' plain
     part carried into the latent space; q_raw [T, heads, plain_dim + rot_dim]: the up-projected queries, whose
-    rotated part (from ``plain_dim`` on) is turned as it is read; out [heads, T, rank]."""
+    rotated part (from ``plain_dim`` on) is turned as it is read; out [heads, T, rank]. ``sinks`` (float32 [heads]): a
+    score per head that joins the softmax denominator."""
     _cuda(q_lat, q_raw, pool, out, cos, sin, seq_start, past, counts, block_table, scratch)
+    _sinks_ok(sinks, heads)
     T = q_raw.shape[0]
     _need(q_lat.shape == (heads, T, rank) and out.shape == (heads, T, rank), "latent_attention: latent query or output shape")
     _need(q_raw.shape == (T, heads, plain_dim + rot_dim), "latent_attention: query shape")
@@ -954,7 +968,7 @@ def latent_attention(q_lat, q_raw, pool, out, cos, sin, seq_start, past, counts,
     n = past.numel()
     lib().call("slb_latent_attention", _p(q_lat), _p(q_raw), _p(pool), _p(out), _p(scratch), _p(cos), _p(sin),
                _p(seq_start), _p(past), _p(counts), _p(block_table), block_table.shape[1], n, int(max_count), T, heads,
-               rank, rot_dim, plain_dim, rotated, int(window), float(scale), int(splits), DT[out.dtype],
+               rank, rot_dim, plain_dim, rotated, int(window), float(scale), int(splits), _p(sinks), DT[out.dtype],
                stream if stream is not None else current_stream())
 
 
@@ -968,12 +982,13 @@ def head_prompt_supported(plain_dim: int, rot_dim: int, value_dim: int, dtype: t
 
 
 def head_prompt_attention(q, kv, k_rot, out, cos, sin, seq_start, counts, max_count: int, heads: int, plain_dim: int,
-                          rot_dim: int, value_dim: int, rotated: int, window: int, scale: float, stream=None) -> None:
+                          rot_dim: int, value_dim: int, rotated: int, window: int, scale: float, stream=None, sinks=None) -> None:
     """Causal attention of whole prompts (every sequence starts at position 0) with per-head keys and values, bfloat16.
     q [T, heads, plain_dim + rot_dim] (rotated part turned as it is read); kv [T, heads * plain_dim + heads *
     value_dim]: every head's unrotated key values, then every head's values; k_rot [T, rot_dim] turned already;
-    out [heads, T, value_dim]."""
+    out [heads, T, value_dim]. ``sinks`` (float32 [heads]): a score per head that joins the softmax denominator."""
     _cuda(q, kv, k_rot, out, cos, sin, seq_start, counts)
+    _sinks_ok(sinks, heads)
     T = q.shape[0]
     _need(q.shape == (T, heads, plain_dim + rot_dim) and kv.shape == (T, heads * (plain_dim + value_dim))
           and k_rot.shape == (T, rot_dim) and out.shape == (heads, T, value_dim), "head_prompt_attention: shapes")
@@ -982,7 +997,7 @@ def head_prompt_attention(q, kv, k_rot, out, cos, sin, seq_start, counts, max_co
         _need(cos is not None and cos.dtype == torch.float32 and cos.shape[1] == rotated // 2, "head_prompt_attention: rotation tables")
     lib().call("slb_head_prompt_attention", _p(q), _p(kv), _p(k_rot), _p(out), _p(cos), _p(sin), _p(seq_start), _p(counts),
                counts.numel(), int(max_count), T, heads, plain_dim, rot_dim, value_dim, rotated, int(window), float(scale),
-               stream if stream is not None else current_stream())
+               _p(sinks), stream if stream is not None else current_stream())
 
 
 def latent_gate(val, g, y, stream=None) -> None:

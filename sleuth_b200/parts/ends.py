@@ -2,6 +2,8 @@
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..kernels import ops
@@ -11,14 +13,25 @@ from ..cache.paged import StateRequest
 from .spec import EmbeddingSpec, HeadSpec, PairEmbeddingSpec
 
 
+def sinusoid_turns(dim: int, base: float, device) -> torch.Tensor:
+    """How many whole turns channel pair i of a position vector makes from one position to the next, base^(-2i / dim) / 2 pi,
+    in 64-bit: the kernels multiply by the position and keep the fraction of a turn, so an angle is as exact at position
+    100,000 as at position 1."""
+    if not base > 0:
+        raise ValueError(f"a position vector needs a positive base, got {base}")
+    i = torch.arange((dim + 1) // 2, dtype=torch.float64)
+    return (base ** (-2.0 * i / dim) / (2.0 * math.pi)).to(device)
+
+
 class TokenEmbedding(Part):
     """x[t] = table[ids[t]] * scale into the float32 stream (sleuth/forge/model/transformer.py:345-348); with
-    ``spec.norm`` the rows are then normalised in place, in float32."""
+    ``spec.norm`` the rows are then normalised in place, in float32; with ``spec.sinusoid`` a position vector is added."""
 
     def __init__(self, spec: EmbeddingSpec, ctx: BuildContext):
         self.spec, self.ctx = spec, ctx
         self.table = None
         self.norm = build_norm(spec.norm, ctx) if spec.norm is not None else None
+        self.turns = sinusoid_turns(spec.dim, spec.sinusoid, ctx.device) if spec.sinusoid else None
 
     def declare(self):
         d = {"weight": ParamDecl((self.spec.vocab, self.spec.dim))}
@@ -37,19 +50,22 @@ class TokenEmbedding(Part):
         ops.embed(b.token_ids, self.table, x, self.spec.scale, b.stream, b.ids_map)
         if self.norm is not None:
             self.norm.forward(x, x, stream=b.stream)
+        if self.turns is not None:
+            ops.sinusoid_add(x, b.tok_pos, self.turns, b.stream)
 
 
 class PairEmbedding(Part):
     """x[t] = table[ids[t]] * scale + pairs[(previous token * mul_prev + token * mul_cur) mod buckets]; a sequence's
     first token takes the pair table's last row. The previous token of a step's first token is per-sequence state
     (one int32 per slot, asked for through ``cache_request`` like a mixer's state), so a prompt may arrive in
-    portions and single-token steps find it without the host."""
+    portions and single-token steps find it without the host. With ``spec.sinusoid`` the same pass adds the position vector."""
 
     def __init__(self, spec: PairEmbeddingSpec, ctx: BuildContext):
         if spec.buckets < 1 or spec.mul_prev < 0 or spec.mul_cur < 0:
             raise ValueError(f"pair_embedding: buckets {spec.buckets}, multipliers {spec.mul_prev}, {spec.mul_cur}")
         self.spec, self.ctx = spec, ctx
         self.table = self.pairs = None
+        self.turns = sinusoid_turns(spec.dim, spec.sinusoid, ctx.device) if spec.sinusoid else None
 
     def declare(self):
         s = self.spec
@@ -67,7 +83,8 @@ class PairEmbedding(Part):
         if not together:
             ops.embed(b.token_ids, self.table, x, s.scale, b.stream, b.ids_map)
         ops.pair_embed(b.token_ids, b.ids_map, self.pairs, x, b.tok_seq, b.tok_pos, b.seq_start, b.slots, view.state,
-                       s.vocab, s.buckets, s.mul_prev, s.mul_cur, b.stream, self.table if together else None, s.scale)
+                       s.vocab, s.buckets, s.mul_prev, s.mul_cur, b.stream, self.table if together else None, s.scale,
+                       turns=self.turns)
 
 
 class LMHead(Part):

@@ -23,7 +23,9 @@ from the step's latents and ``head_prompt_attention`` runs ordinary per-head att
 is written the same way, and later portions and single tokens read it through the latent form.
 
 Options of the spec: ``q_rank`` 0 (the queries are W_q h, no query latent); ``window`` (a query sees the ``window`` most
-recent tokens, its own included); ``gate_span="head"`` (W_g gives one gate value per head; its rows then ride in the
+recent tokens, its own included); ``sinks`` (a learned score per head in the softmax denominator: the attention kernels join
+it to a row's maximum and mass once, at the row's end, or where the key slices are merged); ``rot_dim`` 0 (no rotated part:
+the cache row is the latent alone); ``gate_span="head"`` (W_g gives one gate value per head; its rows then ride in the
 stacked down-projection and the gate is read from that product's float32 result); a position part that pairs
 neighbouring channels (2i with 2i + 1): the rows of the query and key projections that produce the rotated parts are
 reordered once at load time so that pair i sits at channels i and i + rot/2, which the kernels turn; a dot product
@@ -67,7 +69,7 @@ class LatentAttention(Part):
         self.head_gate = spec.output_gate and spec.gate_span == "head"
         self.position = build_position(spec.position, ctx)
         self.down = self.gate = self.uq = self.o = None
-        self.w_uk = self.w_uv_t = self.q_gain = self.c_gain = None
+        self.w_uk = self.w_uv_t = self.q_gain = self.c_gain = self.sinks = None
 
     def declare(self):
         s = self.spec
@@ -85,6 +87,8 @@ class LatentAttention(Part):
              "o.weight": ParamDecl((s.hidden, s.heads * s.value_dim))})
         if s.output_gate:
             d["g.weight"] = ParamDecl((s.heads if self.head_gate else s.heads * s.value_dim, s.hidden))
+        if s.sinks:
+            d["sinks"] = ParamDecl((s.heads,), "vector")
         return d
 
     def _paired_halves(self, w: torch.Tensor, first: int, step: int, count: int) -> torch.Tensor:
@@ -118,6 +122,7 @@ class LatentAttention(Part):
         self.w_uk = t["uk.weight"].to(dt).view(s.heads, s.plain_dim, s.kv_rank).contiguous()
         self.w_uv_t = t["uv.weight"].to(dt).view(s.heads, s.value_dim, s.kv_rank).transpose(1, 2)   # [H, rank, value]
         self.q_gain, self.c_gain = t.get("dq_norm.weight"), t["dkv_norm.weight"]
+        self.sinks = t["sinks"].to(torch.float32).contiguous() if s.sinks else None
 
     def cache_request(self):
         s = self.spec
@@ -154,7 +159,7 @@ class LatentAttention(Part):
             kv = self.ukv.forward(c_out, ws=ws, stream=b.stream)
             val = ws.take((H, T, dv), dt)
             ops.head_prompt_attention(q, kv, k_out, val, cos, sin, b.seq_start, b.counts, b.max_count, H, dn, P, dv, rotated,
-                                      view.window, s.scale, b.stream)
+                                      view.window, s.scale, b.stream, sinks=self.sinks)
             self._gate_and_project(val, g, x, b, ws, T, H, dv, dt)
             ws.release(mark)
             return
@@ -167,7 +172,7 @@ class LatentAttention(Part):
         floats = ops.latent_scratch_floats(T, H, R, splits)
         scratch = ws.take((floats,), torch.float32) if floats else None
         ops.latent_attention(q_lat, q, view.pool, o_lat, cos, sin, b.seq_start, b.past, b.counts, table, b.max_count,
-                             H, R, P, dn, rotated, view.window, s.scale, splits, scratch, b.stream)
+                             H, R, P, dn, rotated, view.window, s.scale, splits, scratch, b.stream, sinks=self.sinks)
         val = ws.take((H, T, dv), dt)
         torch.bmm(o_lat, self.w_uv_t, out=val)
         self._gate_and_project(val, g, x, b, ws, T, H, dv, dt)

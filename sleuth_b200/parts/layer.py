@@ -3,7 +3,8 @@
 ``parallel``: x += mixer(norm1(x)) + ffn(norm2(x)), both sublayers reading the same x; with one norm
 (``norm2`` absent) the feed-forward reads norm1's output too; the feed-forward may be absent.
 
-``prenorm``: x += mixer(norm1(x)); x += ffn(norm2(x)) (sleuth/forge/model/transformer.py:78,87-88,96,99).
+``prenorm``: x += mixer(norm1(x)); x += ffn(norm2(x)) (sleuth/forge/model/transformer.py:78,87-88,96,99); the feed-forward
+may be absent.
 ``sandwich``: a norm in front of and behind each sublayer, x += post1(mixer(norm1(x))), then x += post2(ffn(norm2(x)));
 with ``gated`` each sublayer's result is multiplied by sigmoid(W h + b) of the sublayer's own input h before its norm.
 
@@ -45,9 +46,11 @@ class PreNormLayer(Part):
         self.ctx = ctx
         self.norm1 = build_norm(spec.norm1, ctx)
         self.mixer = build_mixer(spec.mixer, ctx)
-        self.norm2 = build_norm(spec.norm2, ctx)
-        self.ffn = build_ffn(spec.ffn, ctx)
-        self.children = {"norm1": self.norm1, "mixer": self.mixer, "norm2": self.norm2, "ffn": self.ffn}
+        self.ffn = build_ffn(spec.ffn, ctx) if spec.ffn is not None else None
+        self.norm2 = build_norm(spec.norm2, ctx) if self.ffn is not None else None
+        self.children = {"norm1": self.norm1, "mixer": self.mixer}
+        if self.ffn is not None:
+            self.children.update({"norm2": self.norm2, "ffn": self.ffn})
         self.capturable = all(getattr(p, "capturable", True) for p in self.children.values())
 
     def declare(self):
@@ -70,6 +73,8 @@ class PreNormLayer(Part):
     def fused_decode(self):
         """x += mixer(norm1(x)); x += ffn(norm2(x)) is what the persistent single-token kernel runs: offered when all
         four parts offer their share."""
+        if self.ffn is None:
+            return None
         shares = {name: getattr(part, "fused_decode", lambda: None)() for name, part in self.children.items()}
         if any(v is None for v in shares.values()):
             return None
@@ -80,12 +85,13 @@ class PreNormLayer(Part):
     def forward(self, x, b, view, ws):
         mark = ws.mark()
         after = getattr(b, "next_read", None)    # what follows this layer
-        b.next_read = lead_weight_of(self.ffn)
+        b.next_read = lead_weight_of(self.ffn) if self.ffn is not None else after
         self.mixer.forward(self._input(self.norm1, self.mixer, x, b, ws), x, b, view, ws)
         ws.release(mark)
         b.next_read = after
-        self.ffn.forward(self._input(self.norm2, self.ffn, x, b, ws), x, b, ws)
-        ws.release(mark)
+        if self.ffn is not None:
+            self.ffn.forward(self._input(self.norm2, self.ffn, x, b, ws), x, b, ws)
+            ws.release(mark)
 
     def _input(self, norm, part, x, b, ws):
         """What ``part`` reads: the normalised tensor, or, for a part that can normalise inside its first

@@ -22,11 +22,13 @@ from typing import Mapping
 class NormSpec:
     """``kind="rmsnorm"``: x / sqrt(mean(x^2) + eps) * gain. ``kind="layernorm"``: (x - mean) / sqrt(var + eps) * gain,
     var the mean of the squared deviations, no bias. ``gain="scalar"``: the gain is one number for all channels (a
-    tensor without axes in the weight file)."""
+    tensor without axes in the weight file). ``gain_offset``: the weight file stores the gain less this constant (1 for
+    gains stored around zero)."""
     dim: int
     eps: float
     kind: str = "rmsnorm"
     gain: str = "vector"
+    gain_offset: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -161,6 +163,8 @@ class LatentAttentionSpec:
     ``output_gate``: the heads' outputs are multiplied by sigmoid(W_g h) before the output matrix; ``gate_span`` says
     whether W_g gives one value per output channel ("channel") or one per head ("head").
     ``q_rank`` 0: the queries do not pass through a latent; q = W_q h with the tensor ``q.weight``.
+    ``rot_dim`` 0: no rotated part (attention without positions; the cache row is the latent alone). ``sinks``: a learned
+    score per head joins the softmax denominator (tensor ``sinks``; no key, no value, unscaled).
     A position part with ``pairing="neighbours"`` turns channels 2i and 2i + 1 of the rotated parts together."""
     hidden: int
     heads: int
@@ -176,6 +180,7 @@ class LatentAttentionSpec:
     output_gate: bool = True
     kind: str = "latent_attention"
     gate_span: str = "channel"
+    sinks: bool = False
 
 
 @dataclass(frozen=True)
@@ -234,7 +239,8 @@ class RoutedExpertsSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    """One layer: an arrangement (``kind``) of a mixer, a feed-forward and their norms. ``kind="parallel"``:
+    """One layer: an arrangement (``kind``) of a mixer, a feed-forward and their norms. ``kind="prenorm"``:
+    x += mixer(norm1 x), then x += ffn(norm2 x); it may have no feed-forward (``ffn`` and ``norm2`` are None). ``kind="parallel"``:
     x += mixer(norm1 x) + ffn(norm2 x), both of the same x; without ``norm2`` (None) the feed-forward reads norm1's
     output too; it may have no feed-forward (``ffn`` is None). ``kind="sandwich"``: a norm in front of and behind each
     sublayer, x += post1(mixer(norm1 x)), then x += post2(ffn(norm2 x)); with ``gated`` each sublayer's result is first
@@ -291,14 +297,16 @@ class EmbeddingSpec:
     kind: str = "token_embedding"
     norm: NormSpec | None = None          # a norm applied to the looked-up rows (its gain is the tensor ``norm.weight``)
     norm_name: str = "model.embed_norm.weight"
+    sinusoid: float = 0.0                 # b > 0: a position vector is added to the rows. At position p its channel 2i holds
+                                          # sin(p * b^(-2i / dim)) and channel 2i + 1 the cosine of the same angle
 
 
 @dataclass(frozen=True)
 class PairEmbeddingSpec:
     """Token rows times ``scale`` plus a row of a hashed table of token pairs: row (previous token * ``mul_prev`` + token
     * ``mul_cur``) mod ``buckets`` of the ``[buckets + 1, dim]`` tensor ``pairs``; a sequence's first token takes the
-    last row. The previous token is kept per sequence between steps. ``names``: checkpoint names of ``weight`` and
-    ``pairs``."""
+    last row. The previous token is kept per sequence between steps. ``sinusoid``: as for ``EmbeddingSpec``. ``names``:
+    checkpoint names of ``weight`` and ``pairs``."""
     vocab: int
     dim: int
     buckets: int
@@ -308,6 +316,7 @@ class PairEmbeddingSpec:
     names: Mapping[str, str] = field(default_factory=dict)
     name: str = ""
     kind: str = "pair_embedding"
+    sinusoid: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -360,9 +369,10 @@ def looped_schedule(n_layers: int, start: int, stop: int, times: int, entry: str
     """Layers ``start .. stop - 1`` run ``times`` times in a row with the same weights, each pass with cache entries of
     its own; every pass begins by adding its row of the pass vectors. Before that, with ``entry="add"`` every pass but
     the first adds the embedding's output; with ``entry="mix"`` every pass (the first too) replaces the stream by the
-    model's mixing matrix applied to [x; embedding output]. The other layers run once."""
-    if entry not in ("add", "mix"):
-        raise ValueError(f"a loop is entered by 'add' or 'mix', not {entry!r}")
+    model's mixing matrix applied to [x; embedding output]; with ``entry="row"`` nothing else happens. The other layers
+    run once."""
+    if entry not in ("add", "mix", "row"):
+        raise ValueError(f"a loop is entered by 'add', 'mix' or 'row', not {entry!r}")
     if not (0 <= start < stop <= n_layers and times >= 1):
         raise ValueError(f"a loop over layers {start}..{stop - 1}, {times} times, does not fit {n_layers} layers")
     out, cache = [], 0
