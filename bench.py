@@ -561,6 +561,17 @@ def movalorn_config(width, layers, heads, dim, rot, vdim, kv_rank, window, gru_w
             "layers": block, "loop": {"start": 1, "stop": layers, "times": 1}}
 
 
+def nirozen_config(width, layers, heads, dim, vdim, q_rank, kv_rank, experts, top, ff, shared_ff, vocab=32768) -> dict:
+    """Attention through latents without positions, every layer's feed-forward routed with a shared expert; all layers but
+    the first form a loop that runs once."""
+    mixer = {"heads": heads, "dim": dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "scale": dim ** -0.5}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared_ff}}
+    return {"architecture": "Nirozen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65519, "mul_prev": 523, "mul_cur": 7}},
+            "layers": [{"type": "latent_attention", "mixer": mixer, "mlp": moe} for _ in range(layers)],
+            "loop": {"start": 1, "stop": layers, "times": 1}}
+
+
 def fekitar_config(width, layers, heads, kv_heads, dim, window, state, lin_heads, lin_dim, experts, top, ff, shared_ff, vocab=32768) -> dict:
     """The three mixers in turn: a rotated, soft-capped attention beside a gated linear attention; a windowed attention
     with convolutions beside a Mamba-2 recurrence; differential attention (every second one reads the keys and values of
@@ -639,11 +650,23 @@ FEKITAR_SIZES = {
                    ff=1024, shared_ff=1024),
               dict(width=2048, layers=6, heads=16, kv_heads=8, dim=128, rot=128, experts=32, top=4, ff=1024, groups=1, keep=1, shared_ff=1024)),
 }
+# Nirozen beside Lezepel, the closest existing design (attention through a query latent and a key/value latent over every
+# earlier token, a gate per channel, softmax over the chosen experts with a router bias): equal width, depth, heads, ranks
+# and experts. Nirozen has a shared expert as wide as a routed one in every layer and no rotated key part; Lezepel's first
+# feed-forward is dense, and its layers are parallel.
+NIROZEN_SIZES = {
+    "w1024": (dict(width=1024, layers=8, heads=16, dim=64, vdim=64, q_rank=384, kv_rank=256, experts=16, top=4, ff=768, shared_ff=768),
+              dict(width=1024, layers=8, heads=16, dim=64, rot=32, vdim=64, q_rank=384, kv_rank=256, experts=16, top=4, ff=768)),
+    "w2048": (dict(width=2048, layers=6, heads=16, dim=128, vdim=128, q_rank=768, kv_rank=512, experts=64, top=6, ff=1408, shared_ff=1408),
+              dict(width=2048, layers=6, heads=16, dim=128, rot=64, vdim=128, q_rank=768, kv_rank=512, experts=64, top=6, ff=1408)),
+}
 DESIGNS = {"lezepel": (lezepel_config, DESIGN_SIZES), "rabadra": (rabadra_config, RABADRA_SIZES),
-           "movalorn": (movalorn_config, MOVALORN_SIZES), "fekitar": (fekitar_config, FEKITAR_SIZES)}
+           "movalorn": (movalorn_config, MOVALORN_SIZES),
+           "nirozen": (nirozen_config, NIROZEN_SIZES), "fekitar": (fekitar_config, FEKITAR_SIZES)}
 # the model each design stands beside, and how its configuration is made from the second entry of a size
 TWINS = {"lezepel": ("qwen3", lambda kw: qwen3_like(**kw)), "rabadra": ("qwen3", lambda kw: qwen3_like(**kw)),
-         "movalorn": ("lezepel", lambda kw: lezepel_config(**kw)), "fekitar": ("rabadra", lambda kw: rabadra_config(**kw))}
+         "movalorn": ("lezepel", lambda kw: lezepel_config(**kw)), "nirozen": ("lezepel", lambda kw: lezepel_config(**kw)),
+         "fekitar": ("rabadra", lambda kw: rabadra_config(**kw))}
 
 
 def design_point(config: dict, prompt_len: int, batches, steps: int, warmup: int) -> dict:
@@ -705,9 +728,9 @@ def design_point(config: dict, prompt_len: int, batches, steps: int, warmup: int
 
 
 def run_design(args) -> dict:
-    """``--design lezepel`` / ``--design rabadra`` / ``--design movalorn`` / ``--design fekitar``: that design beside the closest
-    existing model (the Qwen3 dense decoder for the first two, Lezepel for Movalorn, Rabadra for Fekitar) at equal width, depth and active feed-forward width,
-    random weights, bfloat16: prompt and decode throughput and where the time goes. The default workload of this file
+    """``--design lezepel`` / ``--design rabadra`` / ``--design movalorn`` / ``--design fekitar`` /
+    ``--design nirozen``: that design beside the closest existing model (the Qwen3 dense decoder for the first two, Lezepel
+    for Movalorn and Nirozen, Rabadra for Fekitar) at equal width, depth and active feed-forward width, random weights, bfloat16: prompt and decode throughput and where the time goes. The default workload of this file
     does not change."""
     out = {"design": args.design, "dtype": "bf16", "data": "synthetic", "prompt": args.design_prompt, "sizes": {}}
     make, sizes = DESIGNS[args.design]
@@ -736,7 +759,7 @@ def main() -> int:
     ap.add_argument("--skip-other-configs", action="store_true",
                     help="leave out the 32-bit block and the 4B- and 8B-shaped points (a quicker run)")
     ap.add_argument("--layers5", type=int, default=0, help="layers of the 8B-shaped point (0 = all 36)")
-    ap.add_argument("--design", choices=["lezepel", "rabadra", "movalorn", "fekitar"], default=None,
+    ap.add_argument("--design", choices=sorted(DESIGNS), default=None,
                     help="instead of the default workload: this design beside the closest existing model at equal size")
     ap.add_argument("--design-size", default="all", help="one of the sizes of --design (w1024, w2048) or all")
     ap.add_argument("--design-prompt", type=int, default=2048)

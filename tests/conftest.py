@@ -106,6 +106,22 @@ def movalorn_folders(tmp_path_factory):
     return out
 
 
+@pytest.fixture(scope="session")
+def nirozen_folders(tmp_path_factory):
+    """Model folders of the tiny Nirozen configurations, float32 weights, made once per session."""
+    import torch
+
+    import tiny_nirozen
+    from sleuth_b200.weights.random_init import write_random_model
+    out = {}
+    for name, cfg in tiny_nirozen.CONFIGS.items():
+        d = tmp_path_factory.mktemp(f"nirozen_{name}")
+        write_random_model(d, cfg, seed=tiny_nirozen.SEEDS[name], dtype=torch.float32, std=tiny_nirozen.STD)
+        tiny_nirozen.sharpen(d)
+        out[name] = str(d)
+    return out
+
+
 def pytest_terminal_summary(terminalreporter):
     """The largest differences from the plain implementation that the GPU tests saw (tests/closeness.py)."""
     import closeness

@@ -203,3 +203,30 @@ def test_the_commands_serve_a_fekitar_folder_too(tmp_path):
     lines = [ln for ln in r.stdout.splitlines() if ln.strip()]
     assert [[int(t) for t in ln.split()] for ln in lines] == [fekitar_plain.greedy_generate(cfg, w, p, 6) for p in prompts]
     assert any("FekitarConfig" in ln for ln in r.stderr.splitlines())
+
+
+@pytest.mark.gpu
+def test_the_commands_serve_a_nirozen_folder_too(tmp_path):
+    """``random-model`` and ``generate`` with a Nirozen ``config.json``, through the same registry: norm gains
+    stored less one, the pair table with its extra row, sinks, a layer without feed-forward, a looped schedule."""
+    import tiny_nirozen
+    from plain import nirozen_plain
+    env = dict(os.environ, PYTHONPATH=ROOT + os.pathsep + os.environ.get("PYTHONPATH", ""))
+    cfg_path = tmp_path / "config.json"
+    cfg_path.write_text(json.dumps(tiny_nirozen.S))
+    folder = tmp_path / "model"
+    r = subprocess.run([sys.executable, "-m", "sleuth_b200", "random-model", str(cfg_path), str(folder), "--seed", "3",
+                        "--dtype", "fp32"], env=env, capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr
+    cfg, w = plain.read_model(folder)
+    assert cfg["architecture"] == "Nirozen" and w["bigram"].shape == (90, 75) and abs(float(w["l0.norm1"].mean())) < 0.2
+    assert w["l1.mix.sink"].shape == (5,) and w["loop.step"].shape == (2, 75) and "l1.norm2" not in w
+    prompts = [[5, 17, 3, 180, 9], [200, 2], [77]]
+    text = "; ".join(",".join(map(str, p)) for p in prompts)
+    r = subprocess.run([sys.executable, "-m", "sleuth_b200", "generate", str(folder), "--prompt-ids", text, "--temperature", "0",
+                        "--max-new-tokens", "6", "--dtype", "fp32", "--max-seq-len", "128"],
+                       env=env, capture_output=True, text=True, timeout=900)
+    assert r.returncode == 0, r.stderr
+    lines = [ln for ln in r.stdout.splitlines() if ln.strip()]
+    assert [[int(t) for t in ln.split()] for ln in lines] == [nirozen_plain.greedy_generate(cfg, w, p, 6) for p in prompts]
+    assert any("NirozenConfig" in ln for ln in r.stderr.splitlines())
