@@ -10,7 +10,8 @@
 //     mbarrier fire when those MMAs have read the stage. After a tile's last slice a commit arms the accumulator's
 //     "full" mbarrier; before reusing an accumulator it waits for the epilogue warps' "drained" arrivals.
 //   * warps 2 to 5: the epilogue. Each reads its 32 rows of the accumulator (tcgen05.ld, 32 columns at a
-//     time), applies the epilogue and stores: bfloat16, float32, float32 accumulate (residual stream), or the gated
+//     time), applies the epilogue and stores: bfloat16, float32, float32 accumulate (residual stream), a sigmoid gate on
+//     bfloat16 values that C already holds, or the gated
 //     activation silu(gate) * up when W holds the gate rows followed by the up rows (sleuth/forge/model/mlp.py:37-40);
 //     the block then multiplies X by 128 gate rows and the 128 matching up rows in one N = 256 instruction.
 // Rows, columns and K beyond the matrices are zero-filled by TMA and masked at the store, so every M, N and every K
@@ -36,7 +37,8 @@ __host__ __device__ constexpr int tc_stages(int bn) {
 }
 constexpr int kTcThreads = 192;       // producer warp, MMA warp, four epilogue warps
 
-enum TcMode : int { kTcBf16 = 0, kTcF32 = 1, kTcAddF32 = 2, kTcSwiglu = 3, kTcQkv = 4 };
+enum TcMode : int { kTcBf16 = 0, kTcF32 = 1, kTcAddF32 = 2, kTcSwiglu = 3, kTcQkv = 4,
+                   kTcGate = 5 };      // C <- C * sigmoid(X W^T), C bfloat16
 
 struct TcArgs {
   void* C;
@@ -227,9 +229,29 @@ __device__ __forceinline__ float fast_gated(const GateAct& f, float g, float u) 
 }
 
 // Stores 32 consecutive float32 accumulator values of one row according to the mode.
-__device__ __forceinline__ void store_row32(const TcArgs& a, int row, int col0, const float (&v)[32]) {
+__device__ __forceinline__ void store_row32(const TcArgs& a, int row, int col0, float (&v)[32]) {
   const bool full = col0 + 32 <= a.N;
-  if (a.mode == kTcBf16 || a.mode == kTcSwiglu) {
+  if (a.mode == kTcGate) {             // v becomes the gated value; it is stored below like any bfloat16 result
+    const __nv_bfloat16* old = reinterpret_cast<const __nv_bfloat16*>(a.C) + (size_t)row * a.ldc + col0;
+    if (full && (a.ldc % 16 == 0) && ((uintptr_t)a.C % 32 == 0)) {
+#pragma unroll
+      for (int j = 0; j < 32; j += 16) {
+        float raw[8];
+        ld_global_256_rw(reinterpret_cast<const float*>(old + j), raw);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const uint32_t two = __float_as_uint(raw[e]);
+          v[j + 2 * e] = __fdividef(__uint_as_float(two << 16), 1.0f + __expf(-v[j + 2 * e]));
+          v[j + 2 * e + 1] = __fdividef(__uint_as_float(two & 0xffff0000u), 1.0f + __expf(-v[j + 2 * e + 1]));
+        }
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 32; ++j)
+        if (col0 + j < a.N) v[j] = __fdividef(__bfloat162float(old[j]), 1.0f + __expf(-v[j]));
+    }
+  }
+  if (a.mode == kTcBf16 || a.mode == kTcSwiglu || a.mode == kTcGate) {
     __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(a.C) + (size_t)row * a.ldc + col0;
     if (full && (a.ldc % 16 == 0) && ((uintptr_t)a.C % 32 == 0)) {      // 32 bytes at a time (a lane holds a row)
 #pragma unroll
@@ -657,7 +679,7 @@ extern "C" int slb_tc_wait_probe(int* status, int polls, int code, void* stream)
 extern "C" int slb_gemm_tc_supported(int M, int N, int K) { return M >= 1 && N >= 1 && K >= 8 && K % 8 == 0; }
 
 // mode: 0 store bfloat16, 1 store float32, 2 add into float32, 3 gated activation (W holds N gate rows then N up
-// rows; C is [M, N] bfloat16). `status` is a device int that the caller zeroed; the kernel writes a non-zero code
+// rows; C is [M, N] bfloat16), 5 multiply the bfloat16 values that C holds by the product's sigmoid. `status` is a device int that the caller zeroed; the kernel writes a non-zero code
 // there if one of its bounded waits gave up (the result is then invalid and the caller must say so).
 static int gemm_tc_run(const void* X, const void* W, void* C, int M, int N, int K, int ldc, int mode, GateAct gate,
                        int* status, void* stream);
@@ -677,7 +699,7 @@ extern "C" int slb_gemm_tc_gated(const void* X, const void* W, void* C, int M, i
 static int gemm_tc_run(const void* X, const void* W, void* C, int M, int N, int K, int ldc, int mode, GateAct gate,
                        int* status, void* stream) {
   SLB_REQUIRE(slb_gemm_tc_supported(M, N, K), "gemm_tc: M=%d N=%d K=%d is not taken (K must be a multiple of 8)", M, N, K);
-  SLB_REQUIRE(mode >= 0 && mode <= 3 && ldc >= N && status != nullptr, "gemm_tc: mode=%d ldc=%d N=%d", mode, ldc, N);
+  SLB_REQUIRE(((mode >= 0 && mode <= 3) || mode == kTcGate) && ldc >= N && status != nullptr, "gemm_tc: mode=%d ldc=%d N=%d", mode, ldc, N);
   SLB_REQUIRE(((uintptr_t)X % 16 == 0) && ((uintptr_t)W % 16 == 0) && ((uintptr_t)C % 16 == 0),
               "gemm_tc: X, W and C must be 16-byte aligned");
   const bool gated = mode == kTcSwiglu;
@@ -761,12 +783,12 @@ extern "C" int slb_gemm_tc_qkv(const void* X, const void* W, int M, int K, int h
                                const int* tok_seq, const int* tok_pos, const int* block_table, int table_stride,
                                int* status, void* stream) {
   SLB_REQUIRE(head_dim == 64 || head_dim == 128, "gemm_tc_qkv: head size 64 or 128, got %d", head_dim);
-  SLB_REQUIRE(heads > 0 && kv_heads >= 0, "gemm_tc_qkv: heads=%d kv_heads=%d", heads, kv_heads);
+  SLB_REQUIRE(heads >= 0 && kv_heads >= 0 && heads + kv_heads > 0, "gemm_tc_qkv: heads=%d kv_heads=%d", heads, kv_heads);
   const int N = (heads + 2 * kv_heads) * head_dim;
   SLB_REQUIRE(slb_gemm_tc_supported(M, N, K), "gemm_tc_qkv: M=%d N=%d K=%d is not taken (K must be a multiple of 8)", M, N, K);
   SLB_REQUIRE((q_gain == nullptr) == (k_gain == nullptr) || kv_heads == 0, "gemm_tc_qkv: q and k gains go together");
   SLB_REQUIRE((cos_table == nullptr) == (sin_table == nullptr), "gemm_tc_qkv: cos and sin tables go together");
-  SLB_REQUIRE(q_out != nullptr && tok_pos != nullptr && status != nullptr, "gemm_tc_qkv: q_out, tok_pos and status are needed");
+  SLB_REQUIRE((q_out != nullptr || heads == 0) && tok_pos != nullptr && status != nullptr, "gemm_tc_qkv: q_out, tok_pos and status are needed");
   SLB_REQUIRE(kv_heads == 0 || (k_pool && v_pool && tok_seq && block_table && table_stride > 0),
               "gemm_tc_qkv: the cache pools and the block table are needed to store keys and values");
   SLB_REQUIRE(((uintptr_t)X % 16 == 0) && ((uintptr_t)W % 16 == 0) && ((uintptr_t)bias % 16 == 0) &&

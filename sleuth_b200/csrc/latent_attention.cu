@@ -26,6 +26,19 @@ constexpr size_t kLatMaxSmem = 227 * 1024;      // dynamic shared memory a block
 constexpr int kLatWarps = 8;
 constexpr int kLatRowsPerWarp = kLatRows / kLatWarps;
 
+// Pages of a step's own keys and values per head, for attention kernels that read pages: the sequences of a step that all
+// start at position 0 take the pages seq_start / 64 + their index onwards, which do not overlap whatever their lengths
+// (a sequence of c tokens fills ceil(c / 64) of them, and there are tokens / 64 + sequences in all). latent_post_kernel,
+// which visits every token in front of the product that fills the pages, writes the block table and clears the value rows
+// behind each sequence's last token: an attention kernel multiplies a page's rows past the end by weights of zero, and
+// what lies there must be finite for that.
+struct PromptPages {
+  int* table;                 // [sequences, stride], or null: no such pages
+  const int* seq_start;       // [sequences + 1]
+  uint4* v_pages;             // [pages, heads, 64, row16] 16-byte pieces
+  int stride, heads, row16;
+};
+
 // One block per token. lat[t] = [q_rank | R | P | anything] float32, rows `lat_stride` values apart; q_rank may be 0 (the
 // queries do not pass through a latent: nothing is written to cq).
 template <typename TO>
@@ -34,7 +47,8 @@ __global__ void latent_post_kernel(const float* __restrict__ lat, const float* _
                                    const float* __restrict__ sin_t, TO* __restrict__ cq, TO* __restrict__ pool,
                                    const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                                    const int* __restrict__ table, int stride, int q_rank, int R, int P, int rot,
-                                   float eps, TO* __restrict__ c_out, TO* __restrict__ k_out, int lat_stride) {
+                                   float eps, TO* __restrict__ c_out, TO* __restrict__ k_out, int lat_stride,
+                                   const PromptPages pp) {
   pdl_enter();
   __shared__ float scratch[33];
   const int t = blockIdx.x;
@@ -59,6 +73,20 @@ __global__ void latent_post_kernel(const float* __restrict__ lat, const float* _
     const TO v = from_f32<TO>((row[q_rank + i] * inv_c) * c_gain[i]);
     if (dst) dst[i] = v;
     if (c_out) c_out[(size_t)t * R + i] = v;      // the same values side by side, for products over the step's own tokens
+  }
+  if (pp.table != nullptr) {
+    const int seq = tok_seq[t], s0 = pp.seq_start[seq], count = pp.seq_start[seq + 1] - s0;
+    const int j = t - s0, first = s0 / kPageTokens + seq, pages = (count + kPageTokens - 1) / kPageTokens;
+    if (j % kPageTokens == 0 && threadIdx.x == 0) pp.table[(size_t)seq * pp.stride + j / kPageTokens] = first + j / kPageTokens;
+    // the tokens of the last page share its rows behind the end
+    const int in_last = count - (pages - 1) * kPageTokens, mine = j - (pages - 1) * kPageTokens;
+    if (mine >= 0) {
+      for (int r = in_last + mine; r < kPageTokens; r += in_last)
+        for (int i = threadIdx.x; i < pp.heads * pp.row16; i += blockDim.x) {
+          const int h = i / pp.row16, c = i - h * pp.row16;
+          pp.v_pages[(((size_t)(first + pages - 1) * pp.heads + h) * kPageTokens + r) * pp.row16 + c] = make_uint4(0, 0, 0, 0);
+        }
+    }
   }
   const float* kr = row + q_rank + R;
   const int half = rot / 2;
@@ -890,24 +918,29 @@ using namespace slb;
 extern "C" int slb_latent_post(const float* lat, const float* q_gain, const float* c_gain, const float* cos_t,
                                const float* sin_t, void* cq, void* pool, const int* tok_seq, const int* tok_pos,
                                const int* table, int stride, int tokens, int q_rank, int R, int P, int rot, float eps,
-                               int dtype, void* c_out, void* k_out, int lat_stride, void* stream) {
+                               int dtype, void* c_out, void* k_out, int lat_stride, int* prompt_table, int prompt_stride,
+                               const int* seq_start, void* v_pages, int v_heads, int v_dim, void* stream) {
   SLB_REQUIRE(tokens >= 0 && q_rank >= 0 && R > 0 && P >= 0 && rot >= 0 && rot <= P && rot % 2 == 0 && eps > 0.f,
               "latent_post: tokens=%d q_rank=%d rank=%d rot_dim=%d rotated=%d", tokens, q_rank, R, P, rot);
   if (lat_stride <= 0) lat_stride = q_rank + R + P;
   SLB_REQUIRE(lat_stride >= q_rank + R + P && (q_rank == 0 || cq != nullptr), "latent_post: rows of %d values hold %d + %d + %d",
               lat_stride, q_rank, R, P);
   SLB_REQUIRE(dtype == kF32 || dtype == kBF16, "latent_post: unknown dtype %d", dtype);
+  SLB_REQUIRE(prompt_table == nullptr || (dtype == kBF16 && c_out != nullptr && seq_start != nullptr && prompt_stride > 0 && v_pages != nullptr &&
+                                          (uintptr_t)v_pages % 16 == 0 && v_heads > 0 && v_dim > 0 && v_dim % 8 == 0),
+              "latent_post: pages of per-head keys and values (%d heads of %d values) are bfloat16, 16-byte aligned", v_heads, v_dim);
+  const PromptPages pp{prompt_table, seq_start, (uint4*)v_pages, prompt_stride, v_heads, v_dim / 8};
   if (tokens == 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   const int widest = q_rank > R ? q_rank : R;
   const int threads = widest > 512 ? 256 : (widest > 128 ? 128 : 64);
   if (dtype == kF32)
     launch(latent_post_kernel<float>, dim3(tokens), dim3(threads), 0, s, lat, q_gain, c_gain, cos_t, sin_t, (float*)cq,
-           (float*)pool, tok_seq, tok_pos, table, stride, q_rank, R, P, rot, eps, (float*)c_out, (float*)k_out, lat_stride);
+           (float*)pool, tok_seq, tok_pos, table, stride, q_rank, R, P, rot, eps, (float*)c_out, (float*)k_out, lat_stride, pp);
   else
     launch(latent_post_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, s, lat, q_gain, c_gain, cos_t, sin_t,
            (__nv_bfloat16*)cq, (__nv_bfloat16*)pool, tok_seq, tok_pos, table, stride, q_rank, R, P, rot, eps, (__nv_bfloat16*)c_out,
-           (__nv_bfloat16*)k_out, lat_stride);
+           (__nv_bfloat16*)k_out, lat_stride, pp);
   return check_launch("latent_post");
 }
 

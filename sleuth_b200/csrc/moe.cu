@@ -122,7 +122,8 @@ struct RouteRule {
 template <typename T>
 __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr,
                                                         const float* __restrict__ bias, const float* __restrict__ pick_bias,
-                                                        const float* __restrict__ given, int* __restrict__ choice,
+                                                        const float* __restrict__ given, const float* __restrict__ given_bias,
+                                                        int* __restrict__ choice,
                                                         float* __restrict__ weight, int tokens, int dim, int E, int top,
                                                         RouteRule rule) {
   pdl_enter();
@@ -131,8 +132,8 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ h,
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
   const T* row = h + (size_t)t * dim;
-  if (given != nullptr) {              // the logits were formed by moe_logits_kernel
-    for (int e = threadIdx.x; e < E; e += blockDim.x) z[e] = given[(size_t)t * E + e];
+  if (given != nullptr) {              // the logits were formed by moe_logits_kernel, or by a product (then without the bias)
+    for (int e = threadIdx.x; e < E; e += blockDim.x) z[e] = given[(size_t)t * E + e] + (given_bias ? given_bias[e] : 0.f);
   } else {
     for (int e = warp; e < E; e += 8) {
       const float* w = wr + (size_t)e * dim;
@@ -721,7 +722,7 @@ extern "C" int slb_moe_route(const void* h, const float* w_router, const float* 
   // from a few tokens on the logits are formed 32 tokens and 16 experts at a time, each weight read once a block
   const float* given = nullptr;
   if (logits_ready) {                             // a product in front of this call has formed the logits
-    SLB_REQUIRE(logits != nullptr && bias == nullptr, "moe_route: ready logits must be given, and hold their bias already");
+    SLB_REQUIRE(logits != nullptr, "moe_route: ready logits must be given");
     given = logits;
   } else if (logits != nullptr && tokens < 16) {         // few tokens: a warp per (token, expert)
     const dim3 lg((tokens * E + 7) / 8), lb(256);
@@ -740,10 +741,11 @@ extern "C" int slb_moe_route(const void* h, const float* w_router, const float* 
   }
   // with the logits given only the choosing warp has work: a block of one warp, so that many tokens are resident at once
   const dim3 block(given != nullptr && tokens >= 256 ? 32 : 256);
+  const float* given_bias = logits_ready ? bias : nullptr;
   if (dtype == kF32)
-    launch(moe_route_kernel<float>, grid, block, smem, s, (const float*)h, w_router, bias, pick_bias, given, choice, weight, tokens, dim, E, top, rule);
+    launch(moe_route_kernel<float>, grid, block, smem, s, (const float*)h, w_router, bias, pick_bias, given, given_bias, choice, weight, tokens, dim, E, top, rule);
   else
-    launch(moe_route_kernel<__nv_bfloat16>, grid, block, smem, s, (const __nv_bfloat16*)h, w_router, bias, pick_bias, given, choice, weight,
+    launch(moe_route_kernel<__nv_bfloat16>, grid, block, smem, s, (const __nv_bfloat16*)h, w_router, bias, pick_bias, given, given_bias, choice, weight,
            tokens, dim, E, top, rule);
   int rc = check_launch("moe_route");
   if (rc || !layout) return rc;        // a step of few pairs needs no counts and no expert order

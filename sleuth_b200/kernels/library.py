@@ -161,7 +161,7 @@ _SIGNATURES = {
     "slb_stream_pair": [P, P, P, I, I, I, P],
     "slb_scale": [P, L, I, I, F, P, P],
     "slb_mingru": [P, L, P, P, P, P, P, P, P, I, I, I, I, P],
-    "slb_latent_post": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, P, I, P],
+    "slb_latent_post": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, P, I, P, I, P, P, I, I, P],
     "slb_latent_head_gate": [P, P, L, P, I, I, I, I, P],
     "slb_head_prompt_attention": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
     "slb_latent_attention": [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, I, P],

@@ -519,6 +519,7 @@ def gemm_f32(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias=None, acc
 
 
 SKINNY_MODES = {"bf16": 0, "f32": 1, "add": 2, "swiglu": 3}
+TC_MODES = {**SKINNY_MODES, "gate": 5}
 
 
 def skinny_supported(M: int, N: int, K: int, norm: bool = False) -> bool:
@@ -632,19 +633,20 @@ def _tc_status(device) -> torch.Tensor:
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str, stream=None, gate=None) -> None:
     """out = x[M, K] @ w^T on the tcgen05 tensor cores (bfloat16 in, float32 accumulation in tensor memory).
-    mode as for ``gemm_skinny``: "bf16" / "f32" store, "add" into a float32 ``out``, "swiglu" with w = [gate; up]."""
+    mode as for ``gemm_skinny``: "bf16" / "f32" store, "add" into a float32 ``out``, "swiglu" with w = [gate; up];
+    "gate": the bfloat16 values of ``out`` are multiplied by the sigmoid of the product."""
     _cuda(x, w, out)
     M, K = x.shape
     N = out.shape[1]
-    _need(x.dtype == w.dtype == torch.bfloat16 and w.shape[1] == K and out.shape[0] == M, "gemm_tc: shapes or dtypes")
+    _need(x.dtype == w.dtype == torch.bfloat16 and w.shape[1] == K and out.shape[0] == M and out.is_contiguous(), "gemm_tc: shapes or dtypes")
     _need(w.shape[0] == (2 * N if mode == "swiglu" else N), "gemm_tc: weight rows")
-    _need(out.dtype == (torch.bfloat16 if mode in ("bf16", "swiglu") else torch.float32), "gemm_tc: output dtype")
+    _need(out.dtype == (torch.bfloat16 if mode in ("bf16", "swiglu", "gate") else torch.float32), "gemm_tc: output dtype")
     g = _gate_args(gate) if mode == "swiglu" else None
     if g is not None:       # ``gate`` = (name, limit, alpha): the gated form with another activation than SiLU
         lib().call("slb_gemm_tc_gated", _p(x), _p(w), _p(out), M, N, K, N, *g, _p(_tc_status(x.device)),
                    stream if stream is not None else current_stream())
         return
-    lib().call("slb_gemm_tc", _p(x), _p(w), _p(out), M, N, K, N, SKINNY_MODES[mode], _p(_tc_status(x.device)),
+    lib().call("slb_gemm_tc", _p(x), _p(w), _p(out), M, N, K, N, TC_MODES[mode], _p(_tc_status(x.device)),
                stream if stream is not None else current_stream())
 
 
@@ -652,12 +654,13 @@ def gemm_tc_qkv(x, w, heads: int, kv_heads: int, head_dim: int, bias, q_gain, k_
                 k_pool, v_pool, tok_seq, tok_pos, block_table, stream=None) -> None:
     """The fused q/k/v projection of many tokens with everything ``qkv_post`` does in its epilogue, on the float32
     accumulators: bias, per-head RMSNorm of q and k, rotation of the whole head, q into ``q_out [T, H, hd]``, k and v
-    into each token's cache page. ``kv_heads == 0``: ``w`` holds only q heads and nothing is written to the cache."""
+    into each token's cache page. ``kv_heads == 0``: ``w`` holds only q heads and nothing is written to the cache;
+    ``heads == 0``: only k and v heads, ``q_out`` is None."""
     _cuda(x, w, bias, q_gain, k_gain, cos, sin, q_out, k_pool, v_pool, tok_seq, tok_pos, block_table)
     M, K = x.shape
-    _need(x.dtype == w.dtype == q_out.dtype == torch.bfloat16, "gemm_tc_qkv: bfloat16 only")
+    _need(x.dtype == w.dtype == torch.bfloat16 and (q_out is None) == (heads == 0), "gemm_tc_qkv: bfloat16 only")
     _need(w.shape == ((heads + 2 * kv_heads) * head_dim, K) and w.is_contiguous() and x.is_contiguous(), "gemm_tc_qkv: weight shape")
-    _need(q_out.shape == (M, heads, head_dim) and q_out.is_contiguous(), "gemm_tc_qkv: q_out shape")
+    _need(q_out is None or (q_out.shape == (M, heads, head_dim) and q_out.is_contiguous() and q_out.dtype == torch.bfloat16), "gemm_tc_qkv: q_out shape")
     for v in (bias, q_gain, k_gain, cos, sin):
         _need(v is None or (v.dtype == torch.float32 and v.is_contiguous()), "gemm_tc_qkv: gains, biases and tables are float32")
     _need(cos is None or (cos.shape[1] == head_dim // 2 and sin.shape == cos.shape), "gemm_tc_qkv: rotation tables [positions, hd / 2]")
@@ -885,14 +888,16 @@ def sample(logits: torch.Tensor, limit: int, temperature: float, top_k: int, top
 
 # ---- attention through low-rank latents (csrc/latent_attention.cu) ----
 def latent_post(lat, q_gain, c_gain, cos, sin, cq, pool, tok_seq, tok_pos, block_table, q_rank: int, rank: int,
-                rot_dim: int, rotated: int, eps: float, stream=None, c_out=None, k_out=None, dtype=None) -> None:
+                rot_dim: int, rotated: int, eps: float, stream=None, c_out=None, k_out=None, dtype=None, pages=None) -> None:
     """lat [T, q_rank + rank + rot_dim] float32 (the two down-projections' output): the normed query latent goes to
     ``cq`` [T, q_rank]; the normed latent and the rotated key part go to the token's row of ``pool``
     [pages, 64, rank + rot_dim] (``pool`` None: nothing is stored). ``rotated``: how many leading channels of the key
     part turn. ``c_out`` [T, rank] and ``k_out`` [T, rot_dim]: the same latent and key part once more, side by side in
     the order of the step's tokens (for a step that multiplies its own tokens' latents). ``lat`` may have more columns
     than the three parts (they are not read). With ``q_rank`` 0 there is no query latent: ``q_gain`` and ``cq`` are None
-    and ``dtype`` names the dtype of what is stored."""
+    and ``dtype`` names the dtype of what is stored. ``pages`` = (table, seq_start, v_pages): the block table int32
+    [sequences, stride] of the step's own per-head pages (``prompt_pages``) is written, and the rows of ``v_pages``
+    [pages, heads, 64, width] behind every sequence's last token are cleared; the sequences all start at position 0."""
     _cuda(lat, q_gain, c_gain, cos, sin, cq, pool, tok_seq, tok_pos, block_table, c_out, k_out)
     _need((c_out is None) == (k_out is None), "latent_post: the two side-by-side outputs go together")
     T = lat.shape[0]
@@ -914,9 +919,24 @@ def latent_post(lat, q_gain, c_gain, cos, sin, cq, pool, tok_seq, tok_pos, block
         _need(block_table.dtype == torch.int32 and block_table.dim() == 2, "latent_post: block table")
         stride = block_table.shape[1]
     _need(tok_seq.dtype == torch.int32 and tok_pos.dtype == torch.int32, "latent_post: token tables are int32")
+    table2 = starts = v_pages = None
+    if pages is not None:
+        table2, starts, v_pages = pages
+        _cuda(table2, starts, v_pages)
+        n = table2.shape[0]
+        _need(table2.dtype == torch.int32 and table2.is_contiguous() and starts.dtype == torch.int32 and starts.numel() >= n + 1,
+              "latent_post: table of the per-head pages")
+        _need(v_pages.dtype == torch.bfloat16 and v_pages.is_contiguous() and v_pages.shape[2] == 64 and v_pages.shape[0] >= prompt_pages(T, n)
+              and dtype == torch.bfloat16 and c_out is not None, "latent_post: per-head value pages")
     lib().call("slb_latent_post", _p(lat), _p(q_gain), _p(c_gain), _p(cos), _p(sin), _p(cq), _p(pool), _p(tok_seq),
                _p(tok_pos), _p(block_table), stride, T, q_rank, rank, rot_dim, rotated, float(eps), DT[dtype],
-               _p(c_out), _p(k_out), lat.shape[1], stream if stream is not None else current_stream())
+               _p(c_out), _p(k_out), lat.shape[1], _p(table2), 0 if table2 is None else table2.shape[1], _p(starts), _p(v_pages),
+               0 if v_pages is None else v_pages.shape[1], 0 if v_pages is None else v_pages.shape[3], stream if stream is not None else current_stream())
+
+
+def prompt_pages(tokens: int, n_seqs: int) -> int:
+    """Pages of 64 tokens that ``n_seqs`` sequences of ``tokens`` tokens together need at most, each starting on a page."""
+    return tokens // 64 + n_seqs
 
 
 def latent_attention_supported(rank: int, rot_dim: int) -> bool:
@@ -1043,7 +1063,7 @@ def moe_route(h, w_router, bias, choice, weight, rank, counts, place, order, top
     pairs are laid out expert by expert: counts [experts], place [T * top] (a pair's row in that order), order
     [T * top] (the pair at each row). choice, rank int32 [T * top]; weight float32 [T * top]. ``logits``: float32
     scratch [T, experts]; with it, steps of many tokens form their logits 32 tokens at a time (the same sums, k
-    ascending). ``logits_ready``: ``logits`` holds the router's logits already (a product formed them; no bias).
+    ascending). ``logits_ready``: ``logits`` holds the router's logits already (a product formed them, without the bias, which is added here).
     ``layout=False`` leaves counts, place and order unwritten: ``moe_experts`` with ``choice`` does not read
     them for steps of at most ``MOE_FEW_PAIRS`` pairs."""
     _cuda(h, w_router, bias, choice, weight, rank, counts, place, order, logits, tiles, pick_bias)

@@ -20,7 +20,11 @@ A bfloat16 step in which every sequence starts at position 0 (whole prompts of 6
 way to the same result: its keys are its own tokens, so one product forms every head's unrotated keys and values
 from the step's latents and ``head_prompt_attention`` runs ordinary per-head attention, which multiplies
 ``plain_dim + rot_dim + value_dim`` values per head and pair of tokens instead of ``2 * kv_rank + rot_dim``. The cache
-is written the same way, and later portions and single tokens read it through the latent form.
+is written the same way, and later portions and single tokens read it through the latent form. Heads without a rotated part
+whose keys and values have the same width, 64 or 128, run on the tcgen05 attention kernel of the key/value cache when the
+prompts fill its tiles: the product that forms their keys and values stores them straight into pages of scratch memory
+(``gemm_tc_qkv``), ``latent_post`` writes those pages' block table, and the output gate is applied in the epilogue of the
+gate's own product.
 
 Options of the spec: ``q_rank`` 0 (the queries are W_q h, no query latent); ``window`` (a query sees the ``window`` most
 recent tokens, its own included); ``sinks`` (a learned score per head in the softmax denominator: the attention kernels join
@@ -43,8 +47,9 @@ import torch
 
 from ..cache.paged import LatentRequest
 from ..kernels import ops
+from .attention import use_tc_attention
 from .base import BuildContext, Normed, ParamDecl, Part, build_position, register_mixer, result_target
-from .linear import Linear
+from .linear import Linear, use_tc
 from .spec import LatentAttentionSpec
 
 
@@ -142,19 +147,39 @@ class LatentAttention(Part):
         rotated = self.position.rot_dim
         mark = ws.mark()
         lat = self.down.forward(h, ws=ws, stream=b.stream, out_dtype=torch.float32)
-        g = self.gate.forward(h, ws=ws, stream=b.stream) if self.gate is not None else None
-        cq = ws.take((T, s.q_rank), dt) if s.q_rank else None
-        if self.head_gate:
-            g = lat[:, s.q_rank + R + P:s.q_rank + R + P + H]
         if self.rider_rows:
             b.rider = lat[:, lat.shape[1] - self.rider_rows:]
-        per_head = (getattr(b, "fresh", False) and b.max_count >= PER_HEAD_PROMPT_TOKENS
-                    and ops.head_prompt_supported(dn, P, dv, dt))
+        cq = ws.take((T, s.q_rank), dt) if s.q_rank else None
+        fresh = getattr(b, "fresh", False) and b.max_count >= PER_HEAD_PROMPT_TOKENS
+        paged = fresh and self._prompt_takes_pages(b, T)
+        per_head = fresh and (paged or ops.head_prompt_supported(dn, P, dv, dt))
         c_out = ws.take((T, R), dt) if per_head else None
         k_out = ws.take((T, P), dt) if per_head else None
+        own = None
+        if paged:
+            shape = (ops.prompt_pages(T, b.n), H, 64, dn)
+            k_pages, v_pages = ws.take(shape, dt), ws.take(shape, dt)
+            own = (ws.take((b.n, -(-b.max_count // 64)), torch.int32), b.seq_start, v_pages)
         ops.latent_post(lat, self.q_gain, self.c_gain, cos, sin, cq, view.pool if view.writes else None, b.tok_seq,
-                        b.tok_pos, table, s.q_rank, R, P, rotated, s.norm_eps, b.stream, c_out, k_out, dtype=dt)
+                        b.tok_pos, table, s.q_rank, R, P, rotated, s.norm_eps, b.stream, c_out, k_out, dtype=dt, pages=own)
         q = self.uq.forward(cq if s.q_rank else h, ws=ws, stream=b.stream).view(T, H, dn + P)
+        if paged:
+            # the up-projection's epilogue puts every head's keys and values into pages of the step's own, and the tcgen05
+            # attention reads them there as it reads a key/value cache
+            ops.gemm_tc_qkv(c_out, self.ukv.weight, 0, H, dn, None, None, None, None, None, 1e-6, None, k_pages, v_pages,
+                            b.tok_seq, b.tok_pos, own[0], b.stream)
+            y = ws.take((T, H * dv), dt)
+            ops.attention_tc(q, k_pages, v_pages, y, b.seq_start, b.past, b.counts, own[0], b.max_count, H, H, dn, view.window,
+                             s.scale, b.stream, max_keys=b.max_count, sinks=self.sinks)
+            if self.gate is not None:
+                self.gate.gate_values(h, y, ws=ws, stream=b.stream)
+            self.o.forward(y, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None), **result_target(b, x))
+            ws.release(mark)
+            return
+        if self.head_gate:
+            g = lat[:, s.q_rank + R + P:s.q_rank + R + P + H]
+        else:
+            g = self.gate.forward(h, ws=ws, stream=b.stream) if self.gate is not None else None
         if per_head:
             kv = self.ukv.forward(c_out, ws=ws, stream=b.stream)
             val = ws.take((H, T, dv), dt)
@@ -177,6 +202,14 @@ class LatentAttention(Part):
         torch.bmm(o_lat, self.w_uv_t, out=val)
         self._gate_and_project(val, g, x, b, ws, T, H, dv, dt)
         ws.release(mark)
+
+    def _prompt_takes_pages(self, b, T: int) -> bool:
+        """Whether the step's whole prompts run on the tcgen05 attention: heads without a rotated part, keys and values of
+        the same width that kernel takes, sequences that fill its tiles."""
+        s = self.spec
+        return (s.rot_dim == 0 and s.plain_dim == s.value_dim and not self.head_gate
+                and use_tc_attention(s.heads, s.heads, s.plain_dim, self.ctx.dtype, b.max_count, s.scale)
+                and use_tc(T, 2 * s.heads * s.plain_dim, s.kv_rank))
 
     def _gate_and_project(self, val, g, x, b, ws, T, H, dv, dt):
         y = ws.take((T, H * dv), dt)

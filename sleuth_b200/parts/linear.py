@@ -10,7 +10,8 @@
   product (cuBLAS through ``torch.mm``, float32 accumulation), as the reference's ``nn.Linear`` always is
   (sleuth/forge/model/attention.py:106-108). The thresholds and what they were measured on stand below.
 
-``into`` adds the product to a float32 tensor (the residual stream) instead of returning it.
+``into`` adds the product to a float32 tensor (the residual stream) instead of returning it. ``gate_values`` multiplies values
+by the product's sigmoid (in the tcgen05 kernel's epilogue, or product, then the gate kernel).
 """
 
 from __future__ import annotations
@@ -215,3 +216,13 @@ class Linear:
         else:
             torch.mm(h, self._wt, out_dtype=want, out=out)
         return out
+
+    def gate_values(self, h: torch.Tensor, y: torch.Tensor, ws=None, stream=None) -> torch.Tensor:
+        """y <- y * sigmoid(h @ W^T), element by element, in place; ``y`` [rows, out] in the run dtype."""
+        if self.dtype == torch.bfloat16 and use_tc(h.shape[0], self.out_features, self.in_features):
+            ops.gemm_tc(h, self.weight, y, "gate", stream)
+            return y
+        mark = ws.mark()
+        ops.sigmoid_gate(y, self.forward(h, ws=ws, stream=stream, out_dtype=torch.float32), stream)
+        ws.release(mark)
+        return y

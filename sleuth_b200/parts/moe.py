@@ -89,9 +89,10 @@ class RoutedExperts(Part):
         self.w_shared_gate = t["shared_gate"].to(torch.float32).reshape(-1).contiguous() if s.shared_gate else None
         # A bfloat16 run whose router matrix is exactly representable in bfloat16 (a file that stores it so) forms the
         # logits as a product of its own: bfloat16 times bfloat16 is exact in float32 and the sums are float32, so these
-        # are the float32 logits of the same inputs, from the tensor cores instead of a lane per token.
+        # are the float32 logits of the same inputs, from the tensor cores instead of a lane per token; a bias joins in
+        # the choosing kernel.
         self.router_product = None
-        if (dt == torch.bfloat16 and self.bias is None and s.hidden % 32 == 0 and s.experts >= 8
+        if (dt == torch.bfloat16 and s.hidden % 32 == 0 and s.experts >= 8
                 and torch.equal(self.w_router.to(torch.bfloat16).to(torch.float32), self.w_router)):
             self.router_product = Linear(self.w_router.to(torch.bfloat16), dt)
 

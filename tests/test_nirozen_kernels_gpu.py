@@ -1,0 +1,329 @@
+"""Each mechanism of Nirozen alone, its kernel against the plain implementation's function: the position vector (alone and in
+the pass that forms token row and pair row), gains stored less one, attention without positions over the latent cache with a
+sink per head (every kernel form, slices, single tokens, loud keys far back and at page borders), whole prompts with per-head
+keys and values on both prompt kernels, the output gate in the product's epilogue, the router whose logits come from a
+product."""
+
+from __future__ import annotations
+
+import numpy as np
+import pytest
+import torch
+
+from plain import nirozen_plain as plain
+
+pytestmark = pytest.mark.gpu
+
+DEV = "cuda:0"
+DT = {"fp32": torch.float32, "bf16": torch.bfloat16}
+TOL = {"fp32": dict(rtol=2e-5, atol=2e-5), "bf16": dict(rtol=2e-2, atol=2e-2)}
+
+
+def ops():
+    from sleuth_b200.kernels import ops as o
+    return o
+
+
+def i32(v):
+    return torch.tensor(v, dtype=torch.int32, device=DEV)
+
+
+# ---- position vectors ----
+def place_vectors_at(positions, width):
+    """The plain position vectors of chosen positions, which may be far from 0."""
+    col = torch.arange(width)
+    freq = 10000.0 ** (-(2.0 * (col // 2).double()) / width)
+    a = torch.tensor(positions, dtype=torch.float64)[:, None] * freq[None, :]
+    return torch.where((col % 2 == 0)[None, :], torch.sin(a), torch.cos(a))
+
+
+@pytest.mark.parametrize("width", [1, 2, 75, 128, 1000, 2048])
+def test_position_vectors(width):
+    from sleuth_b200.parts.ends import sinusoid_turns
+    positions = [0, 1, 2, 63, 64, 1000, 16383, 131071, (1 << 20) - 1]
+    torch.testing.assert_close(place_vectors_at([0, 1, 2], width), plain.place_vectors(3, width, torch.float64))
+    x0 = torch.randn(len(positions), width, generator=torch.Generator().manual_seed(width))
+    x = x0.clone().to(DEV)
+    ops().sinusoid_add(x, i32(positions), sinusoid_turns(width, 10000.0, DEV))
+    torch.testing.assert_close(x.cpu().double(), x0.double() + place_vectors_at(positions, width), rtol=0, atol=2e-6)
+
+
+@pytest.mark.parametrize("dtype", ["fp32", "bf16"])
+@pytest.mark.parametrize("width", [75, 384])
+@pytest.mark.parametrize("one_pass", [True, False])
+def test_token_row_pair_row_and_position_vector(one_pass, width, dtype):
+    """Portions of unequal lengths, one sequence after another in a slot of its own, the previous token kept between steps."""
+    from sleuth_b200.parts.ends import sinusoid_turns
+    o = ops()
+    g = torch.Generator().manual_seed(width)
+    vocab, buckets, mp, mc = 300, 101, 7, 13
+    table = torch.randn(vocab, width, generator=g).to(DT[dtype])
+    pairs = torch.randn(buckets + 1, width, generator=g).to(DT[dtype])
+    w = {"embed": table.double(), "bigram": pairs.double()}
+    e = {"scale": 3.0, "bigram": {"buckets": buckets, "mul_prev": mp, "mul_cur": mc}}
+    seqs = [torch.randint(0, vocab, (n,), generator=g).tolist() for n in (9, 70, 4)]
+    slots, turns = [4, 0, 2], sinusoid_turns(width, 10000.0, DEV)
+    last = torch.full((6, 1), -1, dtype=torch.int32, device=DEV)
+    done, got = [0, 0, 0], [[], [], []]
+    for step in ([4, 1, 2], [1, 60, 2], [4, 9, 0]):
+        live = [k for k in range(3) if step[k]]
+        ids = sum((seqs[k][done[k]:done[k] + step[k]] for k in live), [])
+        c = [step[k] for k in live]
+        tok_seq = i32(sum(([n] * m for n, m in enumerate(c)), []))
+        tok_pos = i32(sum((list(range(done[k], done[k] + step[k])) for k in live), []))
+        x = torch.empty(len(ids), width, device=DEV)
+        starts, now = i32([0, *np.cumsum(c).tolist()]), i32([slots[k] for k in live])
+        if not one_pass:
+            o.embed(i32(ids), table.to(DEV), x, 3.0)
+        o.pair_embed(i32(ids), None, pairs.to(DEV), x, tok_seq, tok_pos, starts, now, last, vocab, buckets, mp, mc,
+                     table=table.to(DEV) if one_pass else None, scale=3.0, turns=turns)
+        at = 0
+        for k in live:
+            got[k].append(x[at:at + step[k]].cpu().double())
+            at += step[k]
+            done[k] += step[k]
+    for k in range(3):
+        torch.testing.assert_close(torch.cat(got[k]), plain.embedding(torch.tensor(seqs[k]), w, e), rtol=1e-6, atol=2e-6)
+    assert last.view(-1).cpu().tolist() == [seqs[1][-1], -1, seqs[2][-1], -1, seqs[0][-1], -1]
+
+
+# ---- gains stored less one ----
+@pytest.mark.parametrize("dtype", ["fp32", "bf16"])
+@pytest.mark.parametrize("d", [75, 384])
+def test_a_norm_whose_gain_is_stored_less_one(d, dtype):
+    from sleuth_b200.parts.base import BuildContext, build_norm
+    from sleuth_b200.parts.spec import NormSpec
+    x, gain = torch.randn(7, d), torch.randn(d) * 0.5
+    n = build_norm(NormSpec(d, 1e-3, gain_offset=1.0), BuildContext(torch.device(DEV), DT[dtype], 8))
+    n.bind({"weight": gain.to(DEV)})
+    out = torch.empty(7, d, dtype=DT[dtype], device=DEV)
+    n.forward(x.to(DEV), out)
+    torch.testing.assert_close(out.cpu().double(), plain.centred_norm(x.double(), gain.double(), 1e-3), **TOL[dtype])
+
+
+# ---- attention over the latent cache ----
+def paged(rows_per_seq, width, dtype, seed):
+    """A pool whose pages are handed out in a scrambled order, and the block table of the sequences."""
+    n_pages = sum(-(-len(r) // 64) for r in rows_per_seq) + 3
+    order = np.random.default_rng(seed).permutation(n_pages)
+    pool = torch.full((n_pages, 64, width), 7.0, dtype=dtype, device=DEV)      # stale contents must never be read
+    stride = max(-(-len(r) // 64) for r in rows_per_seq) + 1
+    table = torch.full((len(rows_per_seq), stride), -1, dtype=torch.int32)
+    k = 0
+    for s, rows in enumerate(rows_per_seq):
+        for p in range(-(-len(rows) // 64)):
+            table[s, p] = int(order[k])
+            part = rows[p * 64:(p + 1) * 64]
+            pool[order[k], :len(part)] = part.to(dtype).to(DEV)
+            k += 1
+    return pool, table.to(DEV)
+
+
+def case(H, dn, dv, R, lengths, seed, loud=()):
+    """Random latents, queries and up-projections. ``loud``: (sequence, query position, key position) triples whose score
+    is made to stand out, so that a key that is skipped or read from a wrong row changes the result."""
+    g = torch.Generator().manual_seed(seed)
+    w_uk = torch.randn(H * dn, R, generator=g, dtype=torch.float64) / R ** 0.5
+    w_uv = torch.randn(H * dv, R, generator=g, dtype=torch.float64) / R ** 0.5
+    seqs = [dict(c=torch.randn(n, R, generator=g, dtype=torch.float64), q=torch.randn(n, H, dn, generator=g, dtype=torch.float64))
+            for n in lengths]
+    for s, qi, ki in loud:
+        k = (seqs[s]["c"][ki] @ w_uk.T).reshape(H, dn)
+        seqs[s]["q"][qi] = 12.0 * k / k.norm(dim=-1, keepdim=True)
+    return w_uk, w_uv, seqs
+
+
+def sinks_for(H, kind):
+    if kind == "near":          # of the size of the scores: each head's differs
+        return torch.linspace(-1.0, 3.0, H, dtype=torch.float64) if H > 1 else torch.tensor([1.0], dtype=torch.float64)
+    return torch.full((H,), {"low": -60.0, "high": 40.0}[kind], dtype=torch.float64)
+
+
+def run(H, dn, dv, R, pasts, counts, dtype, seed, sinks="near", loud=(), splits=1, scale=0.3, general=False):
+    o, dt = ops(), DT[dtype]
+    lengths = [p + c for p, c in zip(pasts, counts)]
+    w_uk, w_uv, seqs = case(H, dn, dv, R, lengths, seed, loud)
+    if dtype == "bf16":     # both sides see the same rounded inputs
+        for s in seqs:
+            s["c"], s["q"] = s["c"].to(dt).double(), s["q"].to(dt).double()
+    sink = sinks_for(H, sinks) if sinks else None
+    pool, table = paged([s["c"] for s in seqs], R, dt, seed)
+    T = sum(counts)
+    q = torch.cat([s["q"][p:p + c] for s, p, c in zip(seqs, pasts, counts)])
+    q_lat = torch.einsum("thd,hdr->htr", q, w_uk.reshape(H, dn, R)).to(dt).to(DEV).contiguous()
+    out = torch.empty(H, T, R, dtype=dt, device=DEV)
+    scratch = torch.empty(max(1, o.latent_scratch_floats(T, H, R, splits)), dtype=torch.float32, device=DEV)
+    o.latent_attention_general_only(general)
+    try:
+        o.latent_attention(q_lat, q.to(dt).to(DEV).contiguous(), pool, out, None, None, i32([0, *np.cumsum(counts).tolist()]), i32(pasts),
+                           i32(counts), table, max(counts), H, R, 0, dn, 0, 0, scale, splits, scratch,
+                           sinks=None if sink is None else sink.float().to(DEV))
+        got = torch.einsum("htr,hvr->thv", out.cpu().double(), w_uv.reshape(H, dv, R))
+    finally:
+        o.latent_attention_general_only(False)
+    none = torch.full((H,), -1e9, dtype=torch.float64)
+    want = []
+    for s, p in zip(seqs, pasts):
+        n = len(s["c"])
+        k, v = (s["c"] @ w_uk.T).reshape(n, H, dn), (s["c"] @ w_uv.T).reshape(n, H, dv)
+        want.append(plain.causal_sink_attention(s["q"], k, v, scale, none if sink is None else sink)[p:])
+    return got, torch.cat(want)
+
+
+SIZES = [(3, 12, 20, 36), (8, 48, 64, 112), (1, 8, 8, 7), (40, 8, 8, 32), (5, 16, 16, 512), (70, 8, 8, 48), (16, 24, 16, 256),
+         (20, 16, 16, 272), (33, 8, 8, 64), (2, 16, 16, 528)]
+
+
+@pytest.mark.parametrize("dtype", ["fp32", "bf16"])
+@pytest.mark.parametrize("H, dn, dv, R", SIZES)
+def test_attention_with_sinks_prompts(H, dn, dv, R, dtype):
+    got, want = run(H, dn, dv, R, pasts=[0, 0, 0, 0, 70], counts=[1, 65, 130, 17, 9], dtype=dtype, seed=H)
+    torch.testing.assert_close(got, want, **TOL[dtype])
+
+
+@pytest.mark.parametrize("dtype", ["fp32", "bf16"])
+@pytest.mark.parametrize("splits", [1, 2, 7])
+@pytest.mark.parametrize("H, dn, dv, R", SIZES)
+def test_attention_with_sinks_single_tokens(H, dn, dv, R, splits, dtype):
+    """One token a sequence: the first of all, one that ends a page, one that begins one, far along; the far ones asking for
+    the first token, a page's last row and a page's first row."""
+    pasts = [0, 63, 64, 300, 447, 200]
+    loud = [(1, 63, 0), (2, 64, 63), (3, 300, 64), (4, 447, 1), (5, 200, 191)]
+    got, want = run(H, dn, dv, R, pasts, [1] * 6, dtype, seed=H + 1, loud=loud, splits=splits)
+    torch.testing.assert_close(got, want, **TOL[dtype])
+    assert float(want.abs().max()) > 0.5         # the loud keys carry the result
+
+
+@pytest.mark.parametrize("dtype", ["fp32", "bf16"])
+@pytest.mark.parametrize("general", [False, True])
+@pytest.mark.parametrize("counts, splits", [([1, 1, 1], 1), ([1, 1, 1], 5), ([33, 2, 65], 1), ([33, 2, 65], 3)])
+def test_the_sink_counts_once_and_is_not_scaled(counts, splits, general, dtype):
+    """A sink far below the scores is no sink; one far above takes everything; one between shares, the same whatever the
+    number of slices and the kernel."""
+    pasts = [200, 0, 64]
+    args = dict(H=6, dn=16, dv=16, R=64, pasts=pasts, counts=counts, dtype=dtype, seed=3, splits=splits, general=general)
+    bare = run(sinks=None, **args)[0]
+    torch.testing.assert_close(run(sinks="low", **args)[0], bare, rtol=1e-5, atol=1e-5)
+    assert float(run(sinks="high", **args)[0].abs().max()) < 1e-6
+    got, want = run(sinks="near", **args)
+    torch.testing.assert_close(got, want, **TOL[dtype])
+    assert float((got - bare).abs().max()) > 0.1
+
+
+@pytest.mark.parametrize("dtype", ["fp32", "bf16"])
+def test_attention_finds_far_keys_and_keys_at_page_borders(dtype):
+    loud = [(0, 299, 0), (0, 298, 63), (0, 297, 64), (0, 296, 127), (0, 295, 128), (0, 290, 5), (1, 200, 200), (1, 199, 191),
+            (2, 640, 1), (3, 130, 64), (4, 450, 3)]
+    pasts, counts = [250, 0, 640, 130, 450], [50, 201, 1, 1, 1]
+    got, want = run(4, 16, 12, 48, pasts, counts, dtype, seed=9, loud=loud)
+    torch.testing.assert_close(got, want, **TOL[dtype])
+    assert float(want.abs().max()) > 0.5
+
+
+# ---- whole prompts with per-head keys and values ----
+PROMPTS = [1, 65, 300, 64, 128, 191]
+LOUD = [(1, 64, 0), (1, 63, 62), (2, 299, 0), (2, 298, 63), (2, 297, 64), (2, 200, 128), (3, 63, 1), (4, 127, 0), (5, 190, 64)]
+
+
+@pytest.mark.parametrize("sinks", ["near", "low", "high"])
+@pytest.mark.parametrize("H, dn, dv, R", [(3, 16, 16, 40), (8, 48, 64, 80), (2, 128, 128, 72), (5, 32, 48, 24)])
+def test_whole_prompts_on_the_warp_level_kernel(H, dn, dv, R, sinks):
+    o, dt = ops(), torch.bfloat16
+    w_uk, w_uv, seqs = case(H, dn, dv, R, PROMPTS, seed=H + dn, loud=LOUD)
+    T, scale, sink = sum(PROMPTS), 0.3, sinks_for(H, sinks)
+    q = torch.cat([s["q"] for s in seqs]).to(dt)
+    c = torch.cat([s["c"] for s in seqs])
+    kv = torch.cat([c @ w_uk.T, c @ w_uv.T], dim=-1).to(dt)
+    out = torch.empty(H, T, dv, dtype=dt, device=DEV)
+    starts = [0, *np.cumsum(PROMPTS).tolist()]
+    o.head_prompt_attention(q.to(DEV), kv.to(DEV), torch.empty(T, 0, dtype=dt, device=DEV), out, None, None, i32(starts), i32(PROMPTS),
+                            max(PROMPTS), H, dn, 0, dv, 0, 0, scale, sinks=sink.float().to(DEV))
+    want = torch.cat([plain.causal_sink_attention(q[a:b].double(), kv[a:b, :H * dn].double().reshape(b - a, H, dn),
+                                                  kv[a:b, H * dn:].double().reshape(b - a, H, dv), scale, sink)
+                      for a, b in zip(starts, starts[1:])])
+    torch.testing.assert_close(out.cpu().double().transpose(0, 1), want, **TOL["bf16"])
+
+
+@pytest.mark.parametrize("lengths", [PROMPTS, [128], [1000, 3], [64, 64, 64, 256], [2, 1, 1, 130, 63]])
+@pytest.mark.parametrize("H, d, R", [(5, 64, 128), (3, 128, 272), (1, 64, 8), (16, 128, 64)])
+def test_whole_prompts_on_the_tensor_memory_kernel(H, d, R, lengths):
+    """Latents normed, keys and values formed into pages of the step's own, attention read from those pages: the pages' table,
+    the cleared rows behind every sequence's end (scratch memory full of NaN before), sinks, loud keys."""
+    o, dt = ops(), torch.bfloat16
+    loud = [(s, i, j) for s, i, j in LOUD if lengths is PROMPTS]
+    w_uk, w_uv, seqs = case(H, d, d, R, lengths, seed=H + d, loud=loud)
+    T, n, scale, sink = sum(lengths), len(lengths), 0.3, sinks_for(H, "near")
+    starts = [0, *np.cumsum(lengths).tolist()]
+    q = torch.cat([s["q"] for s in seqs]).to(dt)
+    lat = torch.cat([s["c"] for s in seqs]).float()
+    gain = 1.0 + 0.2 * torch.randn(R, generator=torch.Generator().manual_seed(R))
+    n_pages = o.prompt_pages(T, n)
+    k_pages, v_pages = (torch.full((n_pages, H, 64, d), float("nan"), dtype=dt, device=DEV) for _ in range(2))
+    table = torch.full((n, -(-max(lengths) // 64)), -1, dtype=torch.int32, device=DEV)
+    tok_seq = i32(sum(([s] * m for s, m in enumerate(lengths)), []))
+    tok_pos = i32(sum((list(range(m)) for m in lengths), []))
+    c_out, k_out = torch.empty(T, R, dtype=dt, device=DEV), torch.empty(T, 0, dtype=dt, device=DEV)
+    o.latent_post(lat.to(DEV), None, gain.to(DEV), None, None, None, None, tok_seq, tok_pos, None, 0, R, 0, 0, 1e-5, c_out=c_out,
+                  k_out=k_out, dtype=dt, pages=(table, i32(starts), v_pages))
+    torch.testing.assert_close(c_out.cpu().double(), plain.rms(lat.double(), 1e-5) * gain.double(), **TOL["bf16"])
+    pages = [table[s, p].item() for s, m in enumerate(lengths) for p in range(-(-m // 64))]
+    assert len(set(pages)) == len(pages) and min(pages) >= 0 and max(pages) < n_pages
+    w = torch.cat([w_uk, w_uv]).to(dt)
+    o.gemm_tc_qkv(c_out, w.to(DEV), 0, H, d, None, None, None, None, None, 1e-6, None, k_pages, v_pages, tok_seq, tok_pos, table)
+    c = c_out.cpu().double()
+    kv = (c @ w.double().T).to(dt)
+    for s, m in enumerate(lengths):       # the pages hold every head's rows, and zeros behind the last value row
+        for p in range(-(-m // 64)):
+            page, rows = table[s, p].item(), min(64, m - 64 * p)
+            mine = kv[starts[s] + 64 * p:starts[s] + 64 * p + rows].double()
+            torch.testing.assert_close(k_pages[page, :, :rows].cpu().double().transpose(0, 1), mine[:, :H * d].reshape(rows, H, d), rtol=1e-2, atol=1e-2)
+            torch.testing.assert_close(v_pages[page, :, :rows].cpu().double().transpose(0, 1), mine[:, H * d:].reshape(rows, H, d), rtol=1e-2, atol=1e-2)
+            assert bool((v_pages[page, :, rows:] == 0).all())
+    for wide in (None, False, True):
+        y = torch.empty(T, H * d, dtype=dt, device=DEV)
+        o.attention_tc(q.to(DEV), k_pages, v_pages, y, i32(starts), i32([0] * n), i32(lengths), table, max(lengths), H, H, d, 0, scale,
+                       max_keys=max(lengths), sinks=sink.float().to(DEV), wide=wide)
+        torch.cuda.synchronize()
+        o.gemm_tc_check(torch.device(DEV))
+        want = torch.cat([plain.causal_sink_attention(q[a:b].double(), kv[a:b, :H * d].double().reshape(b - a, H, d),
+                                                      kv[a:b, H * d:].double().reshape(b - a, H, d), scale, sink)
+                          for a, b in zip(starts, starts[1:])])
+        torch.testing.assert_close(y.view(T, H, d).cpu().double(), want, **TOL["bf16"])
+
+
+# ---- the output gate ----
+@pytest.mark.parametrize("dtype", ["fp32", "bf16"])
+@pytest.mark.parametrize("T, N, K", [(3, 60, 75), (40, 96, 64), (130, 320, 128), (300, 72, 104), (257, 1000, 192), (4100, 256, 64)])
+def test_gate_in_the_products_epilogue(T, N, K, dtype):
+    from sleuth_b200.parts.base import Workspace
+    from sleuth_b200.parts.linear import Linear
+    g = torch.Generator().manual_seed(T)
+    h, w, val = torch.randn(T, K, generator=g), torch.randn(N, K, generator=g) * (3.0 / K ** 0.5), torch.randn(T, N, generator=g)
+    h, w, val = (t.to(DT[dtype]) for t in (h, w, val))
+    y = val.clone().to(DEV)
+    Linear(w.to(DEV), DT[dtype]).gate_values(h.to(DEV), y, ws=Workspace(DEV))
+    torch.cuda.synchronize()
+    ops().gemm_tc_check(torch.device(DEV))
+    torch.testing.assert_close(y.cpu().double(), val.double() * torch.sigmoid(h.double() @ w.double().T), **TOL[dtype])
+
+
+# ---- the router ----
+@pytest.mark.parametrize("T", [1, 9, 300])
+@pytest.mark.parametrize("E, top, d", [(8, 3, 96), (12, 12, 64), (70, 2, 128)])
+def test_router_bias_joins_logits_that_a_product_formed(T, E, top, d):
+    o = ops()
+    g = torch.Generator().manual_seed(T + E)
+    h = torch.randn(T, d, generator=g).to(torch.bfloat16)
+    w = {"router": torch.randn(E, d, generator=g).to(torch.bfloat16).double(), "router.b": 5.0 * torch.randn(E, generator=g).double()}
+    idx, wt, margin = plain.expert_choice(h.double(), w, "", {"router": {"experts": E, "top": top}})
+    z = (h.double() @ w["router"].T).float().to(DEV).contiguous()
+    choice, rank, place, order = (torch.empty(T * top, dtype=torch.int32, device=DEV) for _ in range(4))
+    weight, counts = torch.empty(T * top, device=DEV), torch.empty(E, dtype=torch.int32, device=DEV)
+    o.moe_route(h.to(DEV), w["router"].float().to(DEV), w["router.b"].float().to(DEV), choice, weight, rank, counts, place, order, top,
+                logits=z, logits_ready=True)
+    clear = margin > 1e-4
+    assert torch.equal(choice.cpu().view(T, top).long()[clear], idx[clear]) and int(clear.sum()) >= T - 1
+    torch.testing.assert_close(weight.cpu().view(T, top).double()[clear], wt[clear], rtol=1e-4, atol=2e-5)
+    # the bias decides some of the choices
+    bare, _, _ = plain.expert_choice(h.double(), {**w, "router.b": w["router.b"] * 0}, "", {"router": {"experts": E, "top": top}})
+    assert top == E or T < 9 or not torch.equal(bare, idx)
