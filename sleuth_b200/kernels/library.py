@@ -165,6 +165,9 @@ _SIGNATURES = {
     "slb_latent_head_gate": [P, P, L, P, I, I, I, I, P],
     "slb_head_prompt_attention": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
     "slb_latent_attention": [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, I, P],
+    "slb_latent_decode_attention": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
+    "slb_latent_query": [P, L, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P],
+    "slb_latent_value": [P, P, P, P, P, L, I, P, I, I, I, I, I, P],
     "slb_latent_gate": [P, P, P, I, I, I, I, P],
     "slb_moe_route": [P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P],
     "slb_moe_experts_tc": [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, P, P],

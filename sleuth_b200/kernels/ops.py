@@ -1040,6 +1040,97 @@ def latent_head_gate(val, g, y, stream=None) -> None:
                stream if stream is not None else current_stream())
 
 
+# ---- the same attention in single-token steps of few sequences (csrc/latent_decode.cu, bfloat16) ----
+def latent_decode_supported(heads: int, rank: int, rot_dim: int, plain_dim: int, inner: int, dtype: torch.dtype) -> bool:
+    """Whether ``latent_query``, ``latent_decode_attention`` and ``latent_value`` take these sizes (``inner``: width of the
+    rows that the query up-projection reads)."""
+    if dtype != torch.bfloat16:
+        return False
+    return bool(_ints("slb_latent_decode_supported", heads, rank, rot_dim)) and bool(_ints("slb_latent_team_supported", inner, plain_dim, rank))
+
+
+def _ints(name: str, *values: int) -> int:
+    fn = getattr(lib().dll, name)
+    fn.argtypes, fn.restype = [ctypes.c_int] * len(values), ctypes.c_int
+    return int(fn(*(int(v) for v in values)))
+
+
+def latent_decode_splits(n_seqs: int, heads: int, rank: int, rot_dim: int, max_len: int) -> int:
+    """Into how many slices the keys of a single-token step are cut."""
+    return _ints("slb_latent_decode_splits", n_seqs, heads, rank, rot_dim, max_len)
+
+
+def latent_query(lat, q_gain, c_gain, h, w_uq, w_ukt, cos, sin, q_lat, q_raw, pool, tok_pos, block_table, q_rank: int, rank: int,
+                 rot_dim: int, plain_dim: int, rotated: int, eps: float, stream=None) -> None:
+    """From a single-token step's projections to the queries in the latent space and the cache rows, in one launch.
+    lat [n, >= q_rank + rank + rot_dim] float32 (rows may be part of wider ones): the query latent is RMS-normed (``q_gain``)
+    and up-projected by w_uq [heads * (plain_dim + rot_dim), q_rank] (``q_rank`` 0: the rows of ``h`` bfloat16 [n, inner] are
+    up-projected instead); each head's unrotated part goes on through w_ukt [heads, rank, plain_dim] into q_lat
+    [heads, n, rank], its rotated part, not yet turned, into q_raw [n, heads, plain_dim + rot_dim]; the normed key/value latent
+    (``c_gain``) and the turned key part go to the token's cache row (``pool`` None: nothing is stored)."""
+    _cuda(q_gain, c_gain, h, w_uq, w_ukt, cos, sin, q_lat, q_raw, pool, tok_pos, block_table)
+    heads, n = q_lat.shape[0], q_lat.shape[1]
+    inner = w_uq.shape[1]
+    _need(lat.is_cuda and lat.dtype == torch.float32 and lat.shape[0] == n and lat.stride(1) == 1 and lat.shape[1] >= q_rank + rank + rot_dim,
+          "latent_query: the projections' rows")
+    _need(w_uq.dtype == w_ukt.dtype == q_lat.dtype == torch.bfloat16 and w_uq.shape == (heads * (plain_dim + rot_dim), inner)
+          and w_ukt.shape == (heads, rank, plain_dim) and q_lat.shape == (heads, n, rank) and w_uq.is_contiguous() and w_ukt.is_contiguous(),
+          "latent_query: matrices or result")
+    _need((q_rank == inner and q_gain is not None) or (q_rank == 0 and h is not None and h.shape == (n, inner) and h.dtype == torch.bfloat16),
+          "latent_query: what the up-projection reads")
+    _need(rot_dim == 0 or (q_raw is not None and q_raw.shape == (n, heads, plain_dim + rot_dim) and q_raw.dtype == torch.bfloat16), "latent_query: rotated parts")
+    _need(not rotated or (cos is not None and cos.dtype == torch.float32 and cos.shape[1] == rotated // 2), "latent_query: rotation tables")
+    _need(pool is None or (pool.dtype == torch.bfloat16 and tuple(pool.shape[1:]) == (64, rank + rot_dim)), "latent_query: pool")
+    _need(tok_pos.dtype == torch.int32 and block_table.dtype == torch.int32, "latent_query: int32 tables")
+    lib().call("slb_latent_query", _p(lat), lat.stride(0) if n > 1 else lat.shape[1], _p(q_gain), _p(c_gain), _p(h) if q_rank == 0 else None,
+               _p(w_uq), _p(w_ukt), _p(cos), _p(sin), _p(q_lat), _p(q_raw), _p(pool), _p(tok_pos), _p(block_table), block_table.shape[1],
+               n, heads, inner, q_rank, rank, rot_dim, plain_dim, rotated, float(eps), stream if stream is not None else current_stream())
+
+
+def latent_decode_attention(q_lat, q_raw, pool, out, parts, cos, sin, past, block_table, rank: int, rot_dim: int, plain_dim: int,
+                            rotated: int, window: int, scale: float, splits: int, sinks=None, stream=None) -> None:
+    """``latent_attention`` for one token a sequence. With one slice the result, the sink included, goes to ``out``
+    [heads, n, rank]; with more, the slices' sums, maxima and masses go to ``parts`` (``latent_scratch_floats`` floats) for
+    ``latent_value`` to join, which then takes the sinks."""
+    _cuda(q_lat, q_raw, pool, out, parts, cos, sin, past, block_table)
+    _sinks_ok(sinks, q_lat.shape[0])
+    heads, n = q_lat.shape[0], q_lat.shape[1]
+    _need(q_lat.dtype == pool.dtype == torch.bfloat16 and q_lat.shape == (heads, n, rank) and tuple(pool.shape[1:]) == (64, rank + rot_dim),
+          "latent_decode_attention: shapes or dtypes")
+    _need(rot_dim == 0 or q_raw.shape == (n, heads, plain_dim + rot_dim), "latent_decode_attention: rotated parts")
+    _need(not rotated or (cos is not None and cos.shape[1] == rotated // 2), "latent_decode_attention: rotation tables")
+    _need(block_table.dtype == torch.int32 and block_table.shape[0] == n, "latent_decode_attention: block table")
+    if splits > 1:
+        _need(parts is not None and parts.dtype == torch.float32 and parts.numel() >= latent_scratch_floats(n, heads, rank, splits),
+              "latent_decode_attention: scratch for the slices")
+    else:
+        _need(out is not None and out.shape == (heads, n, rank) and out.dtype == torch.bfloat16, "latent_decode_attention: result")
+    lib().call("slb_latent_decode_attention", _p(q_lat), _p(q_raw), _p(pool), _p(out), _p(parts) if splits > 1 else None, _p(cos), _p(sin),
+               _p(past), _p(block_table), block_table.shape[1], n, heads, rank, rot_dim, plain_dim, rotated, int(window), float(scale),
+               int(splits), _p(sinks) if splits == 1 else None, stream if stream is not None else current_stream())
+
+
+def latent_value(parts, o_lat, w_uv, gate, y, splits: int, sinks=None, stream=None) -> None:
+    """y[t, h * width + j] = (w_uv[h, j] . o[t, h]) * sigmoid(gate), o the weighted sums of latents: o_lat [heads, n, rank], or with
+    ``splits`` > 1 the slices that ``latent_decode_attention`` left in ``parts``, joined here with the heads' ``sinks``. w_uv
+    [heads, width, rank]; ``gate`` float32 [n, heads * width] or [n, heads] (rows may be part of wider ones), or None."""
+    _cuda(o_lat, w_uv, y, parts)
+    heads, width, rank = w_uv.shape
+    n = y.shape[0]
+    _sinks_ok(sinks, heads)
+    _need(w_uv.dtype == y.dtype == torch.bfloat16 and w_uv.is_contiguous() and y.shape == (n, heads * width) and y.is_contiguous(),
+          "latent_value: matrix or result")
+    _need(splits > 1 or (o_lat is not None and o_lat.shape == (heads, n, rank) and o_lat.dtype == torch.bfloat16), "latent_value: weighted sums")
+    _need(splits == 1 or (parts is not None and parts.dtype == torch.float32 and parts.numel() >= latent_scratch_floats(n, heads, rank, splits)),
+          "latent_value: slices")
+    per_head = gate is not None and gate.shape[1] == heads and width != 1
+    _need(gate is None or (gate.is_cuda and gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[0] == n
+                           and gate.shape[1] in (heads, heads * width)), "latent_value: gate")
+    lib().call("slb_latent_value", _p(parts) if splits > 1 else None, _p(o_lat) if splits == 1 else None, _p(sinks) if splits > 1 else None,
+               _p(w_uv), _p(gate), 0 if gate is None else (gate.stride(0) if n > 1 else gate.shape[1]), 1 if per_head else 0, _p(y), n,
+               heads, rank, width, int(splits), stream if stream is not None else current_stream())
+
+
 # ---- routed experts (csrc/moe.cu) ----
 def moe_tile_words(tokens: int, top: int, experts: int) -> int:
     """int32 words of the row-tile table that ``moe_route`` writes for ``moe_experts_tc``."""

@@ -43,6 +43,8 @@ the per-head value up-projection (batched library product), ``latent_gate``, the
 
 from __future__ import annotations
 
+import os
+
 import torch
 
 from ..cache.paged import LatentRequest
@@ -59,8 +61,15 @@ from .spec import LatentAttentionSpec
 PER_HEAD_PROMPT_TOKENS = 64
 
 
+# Up to this many sequences a bfloat16 single-token step runs on the kernels of ``csrc/latent_decode.cu``: five launches a layer
+# (projections, queries and cache rows, attention, values with the gate, output product). SLEUTH_B200_LATENT_STEP=0 keeps
+# the launches that steps of many tokens take.
+STEP_ROWS = 32 if os.environ.get("SLEUTH_B200_LATENT_STEP", "1") != "0" else 0
+
+
 class LatentAttention(Part):
     stores_result = True
+    accepts_normed = True       # a single-token step normalises in the prologue of its first product
     accepts_rider = True        # a layer's own rows ride at the end of the stacked down-projection
 
     def __init__(self, spec: LatentAttentionSpec, ctx: BuildContext):
@@ -71,10 +80,11 @@ class LatentAttention(Part):
         if spec.q_rank < 0 or spec.window < 0:
             raise ValueError(f"latent_attention: q_rank {spec.q_rank}, window {spec.window}")
         self.spec, self.ctx = spec, ctx
+        self._step_ok = None            # whether the single-token kernels take these sizes (asked once)
         self.head_gate = spec.output_gate and spec.gate_span == "head"
         self.position = build_position(spec.position, ctx)
-        self.down = self.gate = self.uq = self.o = None
-        self.w_uk = self.w_uv_t = self.q_gain = self.c_gain = self.sinks = None
+        self.down = self.down_all = self.gate = self.uq = self.o = None
+        self.w_ukt = self.w_uv = self.q_gain = self.c_gain = self.sinks = None
 
     def declare(self):
         s = self.spec
@@ -119,13 +129,18 @@ class LatentAttention(Part):
         if t.get("rider.weight") is not None:
             stack.append(t["rider.weight"])
             self.rider_rows = t["rider.weight"].shape[0]
-        self.down = Linear(torch.cat(stack, dim=0) if len(stack) > 1 else stack[0], dt)     # one product, float32 result
-        self.gate = Linear(t["g.weight"], dt) if s.output_gate and not self.head_gate else None
+        # one product with a float32 result; a gate value per channel has a product of its own in steps of many tokens
+        # (behind the attention, which its epilogue then gates) and rides at the end of this one in single-token steps
+        rows = sum(w.shape[0] for w in stack)
+        channel_gate = s.output_gate and not self.head_gate
+        self.down_all = Linear(torch.cat(stack + ([t["g.weight"]] if channel_gate else []), dim=0), dt)
+        self.down = Linear(self.down_all.weight[:rows], dt)
+        self.gate = Linear(self.down_all.weight[rows:], dt) if channel_gate else None
         self.uq = Linear(self._paired_halves(t["uq.weight" if s.q_rank else "q.weight"], dn, dn + P, s.heads), dt)
         self.o = Linear(t["o.weight"], dt)
         self.ukv = Linear(torch.cat([t["uk.weight"], t["uv.weight"]], dim=0), dt)      # whole prompts: keys and values per head
-        self.w_uk = t["uk.weight"].to(dt).view(s.heads, s.plain_dim, s.kv_rank).contiguous()
-        self.w_uv_t = t["uv.weight"].to(dt).view(s.heads, s.value_dim, s.kv_rank).transpose(1, 2)   # [H, rank, value]
+        self.w_ukt = t["uk.weight"].to(dt).view(s.heads, s.plain_dim, s.kv_rank).transpose(1, 2).contiguous()   # [H, rank, plain]
+        self.w_uv = t["uv.weight"].to(dt).view(s.heads, s.value_dim, s.kv_rank).contiguous()
         self.q_gain, self.c_gain = t.get("dq_norm.weight"), t["dkv_norm.weight"]
         self.sinks = t["sinks"].to(torch.float32).contiguous() if s.sinks else None
 
@@ -134,10 +149,13 @@ class LatentAttention(Part):
         return LatentRequest(s.kv_rank + s.rot_dim, s.window)
 
     def lead_weight(self):
-        return self.down.weight if self.down is not None else None
+        return self.down_all.weight if self.down_all is not None else None
 
     def forward(self, h, x, b, view, ws):
         s, dt = self.spec, self.ctx.dtype
+        if b.max_count == 1 and b.T <= STEP_ROWS and self._step_takes(dt):
+            self._single_tokens(h, x, b, view, ws)
+            return
         if isinstance(h, Normed):
             h = h.tensor()
         T, H, R, P, dn, dv = h.shape[0], s.heads, s.kv_rank, s.rot_dim, s.plain_dim, s.value_dim
@@ -148,7 +166,7 @@ class LatentAttention(Part):
         mark = ws.mark()
         lat = self.down.forward(h, ws=ws, stream=b.stream, out_dtype=torch.float32)
         if self.rider_rows:
-            b.rider = lat[:, lat.shape[1] - self.rider_rows:]
+            b.rider = lat[:, lat.shape[1] - self.rider_rows:]        # (a channel gate's rows are not part of this product)
         cq = ws.take((T, s.q_rank), dt) if s.q_rank else None
         fresh = getattr(b, "fresh", False) and b.max_count >= PER_HEAD_PROMPT_TOKENS
         paged = fresh and self._prompt_takes_pages(b, T)
@@ -189,7 +207,7 @@ class LatentAttention(Part):
             ws.release(mark)
             return
         q_lat = ws.take((H, T, R), dt)
-        torch.bmm(q[:, :, :dn].transpose(0, 1), self.w_uk, out=q_lat)
+        torch.bmm(q[:, :, :dn].transpose(0, 1), self.w_ukt.transpose(1, 2), out=q_lat)
         o_lat = ws.take((H, T, R), dt)
         # the number of key slices follows the batch and the longest sequence allowed, never the lengths of the
         # moment: a recorded step stays valid as its sequences grow
@@ -199,7 +217,7 @@ class LatentAttention(Part):
         ops.latent_attention(q_lat, q, view.pool, o_lat, cos, sin, b.seq_start, b.past, b.counts, table, b.max_count,
                              H, R, P, dn, rotated, view.window, s.scale, splits, scratch, b.stream, sinks=self.sinks)
         val = ws.take((H, T, dv), dt)
-        torch.bmm(o_lat, self.w_uv_t, out=val)
+        torch.bmm(o_lat, self.w_uv.transpose(1, 2), out=val)
         self._gate_and_project(val, g, x, b, ws, T, H, dv, dt)
         ws.release(mark)
 
@@ -210,6 +228,50 @@ class LatentAttention(Part):
         return (s.rot_dim == 0 and s.plain_dim == s.value_dim and not self.head_gate
                 and use_tc_attention(s.heads, s.heads, s.plain_dim, self.ctx.dtype, b.max_count, s.scale)
                 and use_tc(T, 2 * s.heads * s.plain_dim, s.kv_rank))
+
+    def _step_takes(self, dt) -> bool:
+        s = self.spec
+        if self._step_ok is None:
+            self._step_ok = ops.latent_decode_supported(s.heads, s.kv_rank, s.rot_dim, s.plain_dim, s.q_rank or s.hidden, dt)
+        return self._step_ok
+
+    def _single_tokens(self, h, x, b, view, ws):
+        """A step that brings one token a sequence, few sequences: the down-projections with every gate row (the norm in
+        their prologue where that pays), queries into the latent space and cache rows, attention in slices, slices joined,
+        values up-projected and gated, output product."""
+        s, dt = self.spec, self.ctx.dtype
+        n, H, R, P, dn, dv = b.T, s.heads, s.kv_rank, s.rot_dim, s.plain_dim, s.value_dim
+        table = b.tables[view.group]
+        tables = self.position.tables()
+        cos, sin = tables if tables is not None else (None, None)
+        rotated = self.position.rot_dim
+        mark = ws.mark()
+        if isinstance(h, Normed) and not s.q_rank:
+            h = h.tensor()              # the queries read it too
+        lat = self.down_all.forward(h, ws=ws, stream=b.stream, out_dtype=torch.float32, next_read=self.uq.weight)
+        rows = self.down.out_features
+        if self.rider_rows:
+            b.rider = lat[:, rows - self.rider_rows:rows]
+        g = None
+        if self.head_gate:
+            g = lat[:, s.q_rank + R + P:s.q_rank + R + P + H]
+        elif self.gate is not None:
+            g = lat[:, rows:]
+        q_lat = ws.take((H, n, R), dt)
+        q_raw = ws.take((n, H, dn + P), dt) if P else None
+        ops.latent_query(lat, self.q_gain, self.c_gain, None if s.q_rank else h, self.uq.weight, self.w_ukt, cos, sin, q_lat, q_raw,
+                         view.pool if view.writes else None, b.tok_pos, table, s.q_rank, R, P, dn, rotated, s.norm_eps, b.stream)
+        # the number of slices follows the batch and the longest sequence allowed: a recorded step stays valid
+        splits = ops.latent_decode_splits(n, H, R, P, table.shape[1] * 64)
+        floats = ops.latent_scratch_floats(n, H, R, splits)
+        parts = ws.take((floats,), torch.float32) if floats else None
+        o_lat = ws.take((H, n, R), dt) if splits == 1 else None
+        ops.latent_decode_attention(q_lat, q_raw, view.pool, o_lat, parts, cos, sin, b.past, table, R, P, dn, rotated, view.window,
+                                    s.scale, splits, sinks=self.sinks, stream=b.stream)
+        y = ws.take((n, H * dv), dt)
+        ops.latent_value(parts, o_lat, self.w_uv, g, y, splits, sinks=self.sinks, stream=b.stream)
+        self.o.forward(y, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None), **result_target(b, x))
+        ws.release(mark)
 
     def _gate_and_project(self, val, g, x, b, ws, T, H, dv, dt):
         y = ws.take((T, H * dv), dt)

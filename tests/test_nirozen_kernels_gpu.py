@@ -327,3 +327,138 @@ def test_router_bias_joins_logits_that_a_product_formed(T, E, top, d):
     # the bias decides some of the choices
     bare, _, _ = plain.expert_choice(h.double(), {**w, "router.b": w["router.b"] * 0}, "", {"router": {"experts": E, "top": top}})
     assert top == E or T < 9 or not torch.equal(bare, idx)
+
+
+# ---- single-token steps of few sequences ----
+def turned(v, positions, dims, base=500.0):
+    """The first ``dims`` channels of the last axis turned, channel i with i + dims / 2, by position * base^(-2i / dims)."""
+    if not dims:
+        return v
+    half = dims // 2
+    ang = positions.double()[:, None] * base ** (-2.0 * torch.arange(half, dtype=torch.float64) / dims)[None, :]
+    shape = [v.shape[0]] + [1] * (v.dim() - 2) + [half]
+    c, s = ang.cos().reshape(shape), ang.sin().reshape(shape)
+    a, b = v[..., :half], v[..., half:dims]
+    return torch.cat([a * c - b * s, b * c + a * s, v[..., dims:]], dim=-1)
+
+
+def turn_tables(count, dims, base=500.0):
+    ang = torch.arange(count, dtype=torch.float64)[:, None] * base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)[None, :]
+    return ang.cos().float().to(DEV), ang.sin().float().to(DEV)
+
+
+@pytest.mark.parametrize("splits", [1, 2, 7, 64])
+@pytest.mark.parametrize("H, R, P, window", [(1, 16, 0, 0), (6, 64, 0, 0), (16, 512, 0, 0), (16, 256, 32, 0), (20, 272, 0, 0), (33, 112, 16, 100),
+                                             (70, 48, 0, 0), (16, 512, 64, 130), (5, 144, 16, 1), (64, 512, 0, 64)])
+def test_attention_of_single_tokens(H, R, P, window, splits):
+    """Scores, softmax and weighted sum over scattered pages, with sinks (joined in the kernel, or with the slices), windows,
+    a rotated part; the first token of all, a page's last and first places, far keys that stand out."""
+    o, dt = ops(), torch.bfloat16
+    g = torch.Generator().manual_seed(H + R)
+    pasts = [0, 63, 64, 300, 447, 200, 128]
+    loud = {1: 0, 2: 63, 3: 64, 4: 1, 5: 191, 6: 127}
+    n, scale, sink = len(pasts), 0.25, sinks_for(H, "near")
+    w_v = torch.randn(H, 8, R, generator=g, dtype=torch.float64) / R ** 0.5
+    rows = [torch.randn(p + 1, R + P, generator=g).to(dt).double() * 0.5 for p in pasts]
+    q = torch.randn(n, H, R + P, generator=g, dtype=torch.float64)
+    for s, k in loud.items():
+        key = turned(rows[s][:, R:], torch.arange(len(rows[s])), P)[k] if P else rows[s][k, :0]
+        near = torch.cat([rows[s][k, :R], turned(key[None], torch.tensor([-pasts[s]]), P)[0]]) if P else rows[s][k]
+        q[s] = 30.0 * near / near.norm()
+    q = q.to(dt).double()
+    cached = [torch.cat([r[:, :R], turned(r[:, R:], torch.arange(len(r)), P)], -1).to(dt).double() for r in rows]
+    pool, table = paged(cached, R + P, dt, H)
+    cos, sin = turn_tables(512, P) if P else (None, None)
+    q_raw = torch.cat([torch.randn(n, H, 8, generator=g, dtype=torch.float64), q[..., R:]], -1).to(dt).to(DEV).contiguous()
+    q_lat = q[..., :R].permute(1, 0, 2).to(dt).to(DEV).contiguous()
+    parts = torch.full((max(1, o.latent_scratch_floats(n, H, R, splits)),), float("nan"), device=DEV)
+    out = torch.empty(H, n, R, dtype=dt, device=DEV)
+    assert o.latent_decode_supported(H, R, P, 32, 32, dt) == (R % 32 == 0)
+    sinks = sink.float().to(DEV)
+    o.latent_decode_attention(q_lat, q_raw if P else None, pool, out if splits == 1 else None, parts, cos, sin, i32(pasts), table, R, P, 8, P,
+                              window, scale, splits, sinks=sinks)
+    want = []
+    for s, p in enumerate(pasts):
+        lo = max(0, p - window + 1) if window else 0
+        k = cached[s][lo:].unsqueeze(1).expand(-1, H, -1)
+        qq = torch.cat([q[s, :, :R], turned(q[s, :, R:][None], torch.tensor([p]), P)[0].to(dt).double()], -1)
+        sc = torch.einsum("hd,jhd->hj", qq, k) * scale
+        pr = plain.sink_softmax(sc[:, None, :], sink)[:, 0]
+        want.append(torch.einsum("hj,jr->hr", pr, cached[s][lo:, :R]))
+    want = torch.stack(want, 1)
+    if splits == 1:
+        got = out.cpu().double()
+    else:       # the slices as they are defined: sums, maxima and masses; an empty slice has mass 0
+        pt = parts.cpu().double().view(splits, n, H, R + 2)
+        m, mass = pt[..., R], pt[..., R + 1]
+        top = torch.maximum(m.amax(0), sink[None, :])
+        f = torch.where(mass > 0, torch.exp(m - top), torch.zeros_like(m))
+        total = (f * mass).sum(0) + torch.exp(sink[None, :] - top)
+        got = (torch.where((mass > 0)[..., None], pt[..., :R], torch.zeros_like(pt[..., :R])) * f[..., None]).sum(0) / total[..., None]
+        got = got.permute(1, 0, 2)
+    torch.testing.assert_close(got, want, rtol=2e-2, atol=1e-2)
+    if splits == 1 or R % 32:
+        return
+    # and joined, up-projected and gated (R a multiple of 32)
+    dv = 24
+    w = (torch.randn(H, dv, R, generator=g) / R ** 0.5).to(dt)
+    gate = 2.0 * torch.randn(n, 3 + H * dv, generator=g)
+    for view, per in ((gate[:, 3:], False), (gate[:, 3:3 + H], True), (None, False)):
+        y = torch.empty(n, H * dv, dtype=dt, device=DEV)
+        o.latent_value(parts, None, w.to(DEV), None if view is None else gate.to(DEV)[:, 3:3 + view.shape[1]], y, splits, sinks=sinks)
+        val = torch.einsum("hnr,hjr->nhj", want, w.double())
+        if view is not None:
+            z = torch.sigmoid(view.double())
+            val = val * (z[:, :, None] if per else z.reshape(n, H, dv))
+        torch.testing.assert_close(y.cpu().double(), val.reshape(n, -1), rtol=2e-2, atol=1e-2)
+
+
+@pytest.mark.parametrize("n", [1, 8, 9, 20])
+@pytest.mark.parametrize("H, dn, dv, R, P, q_rank", [(3, 32, 20, 64, 0, 96), (16, 64, 64, 256, 0, 384), (5, 96, 128, 96, 0, 32), (1, 32, 8, 32, 8, 64),
+                                                    (4, 128, 256, 512, 64, 0), (2, 160, 40, 1024, 16, 1536)])
+def test_queries_and_values_of_single_tokens(n, H, dn, dv, R, P, q_rank):
+    """Norms, both steps of the queries, the cache rows and nothing else in the pool; finished sums up-projected and gated."""
+    o, dt = ops(), torch.bfloat16
+    g = torch.Generator().manual_seed(n + R)
+    K = q_rank or 128
+    lat = torch.randn(n, q_rank + R + P + 11, generator=g)
+    h = torch.randn(n, K, generator=g).to(dt)
+    qg, cg = 1 + 0.2 * torch.randn(K, generator=g), 1 + 0.2 * torch.randn(R, generator=g)
+    w_uq = (torch.randn(H * (dn + P), K, generator=g) / K ** 0.5).to(dt)
+    w_uk = (torch.randn(H, dn, R, generator=g) / dn ** 0.5).to(dt)
+    pasts = [int(v) for v in torch.randint(0, 130, (n,), generator=g)]
+    pool, table = paged([torch.zeros(p + 1, R + P) for p in pasts], R + P, dt, n)
+    before = pool.clone()
+    cos, sin = turn_tables(140, P) if P else (None, None)
+    q_lat = torch.full((H, n, R), float("nan"), dtype=dt, device=DEV)
+    q_raw = torch.zeros(n, H, dn + P, dtype=dt, device=DEV) if P else None
+    assert o.latent_decode_supported(H, R, P, K, dn, dt) == (R <= 512 and (R + P) % 16 == 0)
+    o.latent_query(lat.to(DEV), qg.to(DEV) if q_rank else None, cg.to(DEV), None if q_rank else h.to(DEV), w_uq.to(DEV),
+                   w_uk.transpose(1, 2).contiguous().to(DEV), cos, sin, q_lat, q_raw, pool, i32(pasts), table, q_rank, R, P, dn, P, 1e-5)
+    x = (plain.rms(lat[:, :q_rank].double(), 1e-5) * qg.double()).to(dt).double() if q_rank else h.double()
+    q = (x @ w_uq.double().T).reshape(n, H, dn + P)
+    torch.testing.assert_close(q_lat.cpu().double(), torch.einsum("nhd,hdr->hnr", q[..., :dn].to(dt).double(), w_uk.double()), rtol=2e-2, atol=2e-2)
+    if P:
+        torch.testing.assert_close(q_raw[..., dn:].cpu().double(), q[..., dn:], rtol=1e-2, atol=1e-2)
+    want = torch.cat([plain.rms(lat[:, q_rank:q_rank + R].double(), 1e-5) * cg.double(),
+                      turned(lat[:, q_rank + R:q_rank + R + P].double(), torch.tensor(pasts), P)], -1)
+    for t, p in enumerate(pasts):
+        at = (table[t, p // 64].item(), p % 64)
+        torch.testing.assert_close(pool[at].cpu().double(), want[t], rtol=1e-2, atol=1e-2)
+        before[at] = pool[at]
+    assert torch.equal(pool, before)
+    o_lat = torch.randn(H, n, R, generator=g).to(dt)
+    w_uv = (torch.randn(H, dv, R, generator=g) / R ** 0.5).to(dt)
+    gate = 2.0 * torch.randn(n, 5 + H * dv, generator=g)
+    y = torch.empty(n, H * dv, dtype=dt, device=DEV)
+    o.latent_value(None, o_lat.to(DEV), w_uv.to(DEV), gate.to(DEV)[:, 5:], y, 1)
+    val = torch.einsum("hnr,hjr->nhj", o_lat.double(), w_uv.double()).reshape(n, -1) * torch.sigmoid(gate[:, 5:].double())
+    torch.testing.assert_close(y.cpu().double(), val, rtol=2e-2, atol=1e-2)
+
+
+def test_the_slices_follow_the_batch_and_the_longest_sequence():
+    o = ops()
+    one = o.latent_decode_splits(1, 16, 256, 0, 64 * 20)
+    assert one == 20 and o.latent_decode_splits(1, 16, 256, 0, 64) == 1 and o.latent_decode_splits(1000, 16, 256, 0, 4096) == 1
+    assert 1 < o.latent_decode_splits(8, 16, 512, 0, 4096) <= 64
+    assert not o.latent_decode_supported(16, 528, 0, 64, 64, torch.bfloat16) and not o.latent_decode_supported(16, 256, 0, 64, 64, torch.float32)
