@@ -587,7 +587,8 @@ __global__ void __launch_bounds__(256) moe_few_gate_up_kernel(const T* __restric
 template <typename T>
 __global__ void __launch_bounds__(256) moe_few_down_kernel(const T* __restrict__ act, const T* __restrict__ w_down,
                                                            const int* __restrict__ choice, const float* __restrict__ weight,
-                                                           float* __restrict__ x, int top, int dim, int ff) {
+                                                           float* __restrict__ x, const float* __restrict__ extra, int top, int dim,
+                                                           int ff) {
   pdl_enter();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = blockIdx.y * 8 + warp;
@@ -615,7 +616,7 @@ __global__ void __launch_bounds__(256) moe_few_down_kernel(const T* __restrict__
     }
     total = fmaf(weight[pair], warp_sum(s), total);
   }
-  if (lane == 0) x[(size_t)t * dim + n] += total;
+  if (lane == 0) x[(size_t)t * dim + n] += extra ? total + extra[(size_t)t * dim + n] : total;
 }
 
 __global__ void moe_combine_kernel(float* __restrict__ x, const float* __restrict__ y, int top, int dim, size_t total) {
@@ -755,13 +756,14 @@ extern "C" int slb_moe_route(const void* h, const float* w_router, const float* 
   return check_launch("moe_group");
 }
 
-// act: [tokens * top, ff] in the run dtype; y: float32 [tokens * top, dim]; x: the float32 stream [tokens, dim].
+// act: [tokens * top, ff] in the run dtype; y: float32 [tokens * top, dim]; x: the float32 stream [tokens, dim]; extra: null,
+// or float32 [tokens, dim] rows that the same kernel adds into the stream (steps of few pairs only).
 // choice (from slb_moe_route) serves steps of few pairs, which run a warp per output instead of tiles and need neither
 // the counts nor the expert-ordered list (`place` is accepted for callers that have it and is not read).
 extern "C" int slb_moe_experts(const void* h, const void* w_gu, const void* w_down, const int* counts, const int* list,
                                const int* choice, const int* place, const float* weight, void* act, float* y, float* x,
-                               int tokens, int dim, int ff, int E, int top, int act_kind, float act_limit, float act_alpha,
-                               int dtype, void* stream) {
+                               const float* extra, int tokens, int dim, int ff, int E, int top, int act_kind, float act_limit,
+                               float act_alpha, int dtype, void* stream) {
   SLB_REQUIRE(tokens >= 0 && dim > 0 && ff > 0 && E > 0 && top > 0, "moe_experts: tokens=%d dim=%d ff=%d experts=%d top=%d",
               tokens, dim, ff, E, top);
   SLB_REQUIRE(dtype == kF32 || dtype == kBF16, "moe_experts: unknown dtype %d", dtype);
@@ -780,15 +782,17 @@ extern "C" int slb_moe_experts(const void* h, const void* w_gu, const void* w_do
     const dim3 f1((unsigned)pairs, (ff + 7) / 8), f2((unsigned)tokens, (dim + 7) / 8);
     if (dtype == kF32) {
       launch(moe_few_gate_up_kernel<float>, f1, block, 0, s, (const float*)h, (const float*)w_gu, choice, (float*)act, top, dim, ff, gate);
-      launch(moe_few_down_kernel<float>, f2, block, 0, s, (const float*)act, (const float*)w_down, choice, weight, x, top, dim, ff);
+      launch(moe_few_down_kernel<float>, f2, block, 0, s, (const float*)act, (const float*)w_down, choice, weight, x, extra, top, dim, ff);
     } else {
       launch(moe_few_gate_up_kernel<__nv_bfloat16>, f1, block, 0, s, (const __nv_bfloat16*)h, (const __nv_bfloat16*)w_gu, choice,
              (__nv_bfloat16*)act, top, dim, ff, gate);
       launch(moe_few_down_kernel<__nv_bfloat16>, f2, block, 0, s, (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, choice,
-             weight, x, top, dim, ff);
+             weight, x, extra, top, dim, ff);
     }
     return check_launch("moe_experts");          // the down kernel has added into the stream already
-  } else if (dtype == kBF16 && dim % 8 == 0 && ff % 8 == 0 && aligned) {
+  }
+  SLB_REQUIRE(extra == nullptr, "moe_experts: further rows are added in steps of at most %d pairs only, this one has %lld", kMoeFewPairs, pairs);
+  if (dtype == kBF16 && dim % 8 == 0 && ff % 8 == 0 && aligned) {
     const long long tiles64 = pairs / kMmaRows + (pairs < E ? pairs : E);
     launch(moe_mma_kernel<true>, dim3((unsigned)tiles64, (ff + 63) / 64), dim3(128), 0, s, (const __nv_bfloat16*)h,
            (const __nv_bfloat16*)w_gu, counts, list, weight, (__nv_bfloat16*)act, (float*)nullptr, E, top, dim, ff, gate);

@@ -1177,11 +1177,14 @@ def moe_route(h, w_router, bias, choice, weight, rank, counts, place, order, top
 
 
 def moe_experts(h, w_gate_up, w_down, counts, order, weight, act, y, x, top: int, activation: str = "silu",
-                stream=None, choice=None, place=None, limit: float = 0.0, alpha: float = 1.0) -> None:
+                stream=None, choice=None, place=None, limit: float = 0.0, alpha: float = 1.0, extra=None) -> None:
     """x[t] += sum over the token's choices of weight * down_e(f(gate_e h) * (up_e h)). w_gate_up [experts, 2 * ff, d]
     (gate rows, then up rows), w_down [experts, d, ff]; act [T * top, ff] and y [T * top, d] float32 are scratch.
-    With ``choice`` and ``place`` (from ``moe_route``) a step of few pairs runs a warp per output instead of tiles."""
-    _cuda(h, w_gate_up, w_down, counts, order, weight, act, y, x, choice, place)
+    With ``choice`` and ``place`` (from ``moe_route``) a step of few pairs runs a warp per output instead of tiles, and then
+    adds the rows of ``extra`` (float32, the stream's shape) as well, if given."""
+    _cuda(h, w_gate_up, w_down, counts, order, weight, act, y, x, choice, place, extra)
+    _need(extra is None or (extra.dtype == torch.float32 and extra.shape == x.shape and h.shape[0] * top <= MOE_FEW_PAIRS),
+          "moe_experts: further rows go with steps of few pairs")
     for t in (choice, place):
         _need(t is None or (t.dtype == torch.int32 and t.numel() >= h.shape[0] * top), "moe_experts: choice and place tables")
     T, d = h.shape
@@ -1193,7 +1196,7 @@ def moe_experts(h, w_gate_up, w_down, counts, order, weight, act, y, x, top: int
     _need(x.shape == (T, d) and x.dtype == torch.float32, "moe_experts: the stream")
     _need(activation in ACTIVATIONS, f"moe_experts: activation {activation!r}")
     lib().call("slb_moe_experts", _p(h), _p(w_gate_up), _p(w_down), _p(counts), _p(order), _p(choice), _p(place), _p(weight), _p(act), _p(y),
-               _p(x), T, d, ff, E, int(top), ACTIVATIONS[activation], float(limit), float(alpha), DT[h.dtype],
+               _p(x), _p(extra), T, d, ff, E, int(top), ACTIVATIONS[activation], float(limit), float(alpha), DT[h.dtype],
                stream if stream is not None else current_stream())
 
 

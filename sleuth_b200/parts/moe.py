@@ -22,6 +22,7 @@ import torch
 
 from ..kernels import ops
 from .base import BuildContext, Normed, ParamDecl, Part, build_ffn, register_ffn
+from .layer import BRANCH, _side_stream
 from .linear import Linear
 from .spec import RoutedExpertsSpec
 
@@ -106,7 +107,12 @@ class RoutedExperts(Part):
         if isinstance(h, Normed):
             h = h.tensor()
         mark = ws.mark()
-        if self.shared is not None:       # the shared expert first: its weights are what the layer in front asked L2 for
+        T = h.shape[0]
+        pairs = T * s.top
+        extra = side = None
+        if self._shared_beside(b, pairs, x.device):
+            extra, side = self._start_shared(h, x, b, ws)
+        elif self.shared is not None:     # the shared expert first: its weights are what the layer in front asked L2 for
             after = getattr(b, "next_read", None)
             b.next_read = None
             if self.w_shared_gate is None:
@@ -122,8 +128,6 @@ class RoutedExperts(Part):
                 self.shared.forward(h, own, b, ws)
                 ops.row_gate(h, self.w_shared_gate, own, x, accumulate=not store, stream=b.stream)
             b.next_read = after
-        T = h.shape[0]
-        pairs = T * s.top
         choice, rank, place, order = (ws.take((pairs,), torch.int32) for _ in range(4))
         counts = ws.take((s.experts,), torch.int32)
         weight = ws.take((pairs,), torch.float32)
@@ -148,9 +152,39 @@ class RoutedExperts(Part):
             ops.moe_experts_tc(h, self.w_gate_up, self.w_down, order, place, weight, tiles, xs, act, y, x, s.top, b.stream,
                                activation=s.activation, limit=s.limit, alpha=s.alpha)
         else:
+            if side is not None:
+                torch.cuda.current_stream().wait_stream(side)
             ops.moe_experts(h, self.w_gate_up, self.w_down, counts, order, weight, act, y, x, s.top, s.activation, b.stream,
-                            choice, place, limit=s.limit, alpha=s.alpha)
+                            choice, place, limit=s.limit, alpha=s.alpha, extra=extra)
         ws.release(mark)
+
+    def _shared_beside(self, b, pairs: int, device) -> bool:
+        """Whether the shared expert runs on a second stream beside the router: in steps that bring one token a sequence and
+        few pairs, whose kernels each wait for the one before. Not inside a branch that is on that stream already."""
+        return (BRANCH and self.shared is not None and self.w_shared_gate is None and getattr(self.shared, "stores_result", False)
+                and b.max_count == 1 and pairs <= ops.MOE_FEW_PAIRS
+                and torch.cuda.current_stream().cuda_stream != _side_stream(device).cuda_stream)
+
+    def _start_shared(self, h, x, b, ws):
+        """The shared expert on the second stream, into an empty target (``b.store_first``) or into rows of its own that the
+        experts' last kernel adds. Its scratch memory is taken first, and what follows begins above the highest address it
+        used. Returns (those rows or None, the stream to wait for)."""
+        main, side = torch.cuda.current_stream(), _side_stream(x.device)
+        own = None
+        if not getattr(b, "store_first", False):
+            own = ws.take(x.shape, torch.float32)
+            b.store_first = True
+        after, seen, ws.high = getattr(b, "next_read", None), ws.high, ws.top
+        b.next_read = None
+        side.wait_stream(main)              # the normed input is ready
+        with torch.cuda.stream(side):
+            b.stream = side.cuda_stream
+            self.shared.forward(h, x if own is None else own, b, ws)
+        b.stream = main.cuda_stream
+        b.next_read = after
+        ws.top = max(ws.top, ws.high)
+        ws.high = max(seen, ws.high)
+        return own, side
 
 
 register_ffn("routed_experts", RoutedExperts)
