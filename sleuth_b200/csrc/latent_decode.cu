@@ -3,9 +3,9 @@
 // and long caches, so each kernel here spreads one step over all SMs and does in one launch what would be several.
 //
 //   latent_decode_attn_kernel   scores, online softmax and weighted sum of latents for all heads of a sequence over a slice
-//                               of its cache rows. Eight warps share a chunk of 64 rows: for the scores a warp takes eight of
-//                               the keys, for the weighted sum a share of the latent's columns, so that all of them work
-//                               although a sequence brings no more rows than it has heads
+//                               of its cache rows. Sixteen warps share a chunk of 64 rows: for the scores a warp takes eight
+//                               of the keys and half of the columns, for the weighted sum a share of the latent's columns,
+//                               so that all of them work although a sequence brings no more rows than it has heads
 //   latent_query_kernel         norm of the query latent, query up-projection, the step into the latent space, norm of the
 //                               key/value latent, rotation of the key part and the cache write; a cluster of blocks a head
 //   latent_value_kernel         joining of the slices with the head's sink, value up-projection, output gate; a cluster of
@@ -33,24 +33,28 @@ struct LatentDecodeArgs {
   float scale;
 };
 
-// Shared memory of a block: queries [16 MT][ks], `buffers` chunks of 64 cache rows [64][ks], scores float [16 MT][68],
-// weights bfloat16 [16 MT][72], the rows' factors float [16 MT].
+constexpr int kLdWarps = 16, kLdThreads = kLdWarps * 32;
+
+// Shared memory of a block: queries [16 MT][ks], `buffers` chunks of 64 cache rows [64][ks], the scores of each half of the
+// columns float [2][16 MT][68], weights bfloat16 [16 MT][72], the rows' factors float [16 MT].
 __host__ __device__ inline size_t latent_decode_smem(int mt, int W, int buffers) {
   const size_t rows = 16 * mt;
-  return (rows + (size_t)64 * buffers) * (W + 8) * 2 + rows * 68 * 4 + rows * 72 * 2 + rows * 4;
+  return (rows + (size_t)64 * buffers) * (W + 8) * 2 + 2 * rows * 68 * 4 + rows * 72 * 2 + rows * 4;
 }
 
-// Grid: (slice, sequence, tile of 16 MT heads). NP: pairs of 8-column tiles of the latent that a warp owns (R <= 128 NP).
-template <int MT, int NP>
-__global__ void __launch_bounds__(256) latent_decode_attn_kernel(const LatentDecodeArgs a) {
+// Grid: (slice, sequence, tile of 16 MT heads). NP: pairs of 8-column tiles of the latent that a warp owns (R <= 256 NP).
+// KQ > 0 (one row tile, R + P = 32 KQ): a warp keeps the queries of its half of the columns, KQ steps of 16, in registers; read
+// from shared memory by sixteen warps at every chunk they would be two fifths of all that is read there.
+template <int MT, int NP, int KQ>
+__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_attn_kernel(const LatentDecodeArgs a) {
   pdl_enter();
   extern __shared__ __align__(16) unsigned char ld_raw[];
-  constexpr int ROWS = 16 * MT, TPR = 256 / ROWS, KPT = 64 / TPR;      // threads a row, keys a thread in the softmax
+  constexpr int ROWS = 16 * MT, TPR = kLdThreads / ROWS, KPT = 64 / TPR;      // threads a row, keys a thread in the softmax
   const int W = a.R + a.P, ks = W + 8;
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(ld_raw);
   __nv_bfloat16* Ks = Qs + ROWS * ks;
   float* Ss = reinterpret_cast<float*>(Ks + (size_t)a.buffers * 64 * ks);
-  __nv_bfloat16* Ps = reinterpret_cast<__nv_bfloat16*>(Ss + ROWS * 68);
+  __nv_bfloat16* Ps = reinterpret_cast<__nv_bfloat16*>(Ss + 2 * ROWS * 68);
   float* As = reinterpret_cast<float*>(Ps + ROWS * 72);
   const int slice = blockIdx.x, seq = blockIdx.y, h0 = blockIdx.z * ROWS, nh = min(ROWS, a.H - h0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
@@ -63,12 +67,14 @@ __global__ void __launch_bounds__(256) latent_decode_attn_kernel(const LatentDec
   const int* trow = a.table + (size_t)seq * a.stride;
   const int pieces = W / 8;
 
-  // a chunk of 64 cache rows (a page) into buffer `buf`; rows past the token become zeros, never stale values
-  auto load_chunk = [&](int c, int buf) {
+  // a chunk of 64 cache rows (a page, whose number was looked up a chunk earlier) into buffer `buf`; rows past the token
+  // become zeros, never stale values
+  auto page_of = [&](int c) { return c < c_hi ? trow[first / 64 + c] : 0; };
+  auto load_chunk = [&](int c, int page, int buf) {
     const int k0 = first + c * 64, nk = min(64, pos - k0 + 1);
-    const __nv_bfloat16* src = a.pool + (size_t)trow[k0 / 64] * 64 * W;
+    const __nv_bfloat16* src = a.pool + (size_t)page * 64 * W;
     __nv_bfloat16* base = Ks + (size_t)buf * 64 * ks;
-    for (int j = warp; j < 64; j += 8)
+    for (int j = warp; j < 64; j += kLdWarps)
       for (int p = lane; p < pieces; p += 32) {
         __nv_bfloat16* dst = base + (size_t)j * ks + p * 8;
         if (j < nk) cp_async16(smem_u32(dst), src + (size_t)j * W + p * 8);
@@ -78,12 +84,13 @@ __global__ void __launch_bounds__(256) latent_decode_attn_kernel(const LatentDec
   // one group of copies per chunk, empty past the end, so that "all but the newest groups" always means the same chunks
   const int ahead = a.buffers - 1;
   for (int i = 0; i < ahead; ++i) {
-    if (c_lo + i < c_hi) load_chunk(c_lo + i, i);
+    if (c_lo + i < c_hi) load_chunk(c_lo + i, page_of(c_lo + i), i);
     cp_async_commit();
   }
+  int next_page = page_of(c_lo + ahead);
   // queries: the latent part as it is, the rotated part turned by the token's angle
   const int half = a.rot / 2;
-  for (int r = warp; r < ROWS; r += 8) {
+  for (int r = warp; r < ROWS; r += kLdWarps) {
     __nv_bfloat16* qs = Qs + (size_t)r * ks;
     if (r >= nh) {
       for (int i = lane * 8; i < W; i += 256) *reinterpret_cast<uint4*>(qs + i) = make_uint4(0, 0, 0, 0);
@@ -114,41 +121,60 @@ __global__ void __launch_bounds__(256) latent_decode_attn_kernel(const LatentDec
   float m = -INFINITY, l = 0.f;
   const float scale_log2 = a.scale * 1.4426950408889634f;
   const uint32_t q_base = smem_u32(Qs), p_base = smem_u32(Ps);
-  const int k16 = W / 16;
+  const int k16 = W / 16, k_mid = (k16 + 1) / 2;            // the columns' halves, in steps of 16
+  const int kt = warp & 7, kb_lo = warp < 8 ? 0 : k_mid, kb_hi = warp < 8 ? min(k_mid, k16) : k16;
+  uint32_t qr[KQ > 0 ? KQ : 1][4];
+  if constexpr (KQ > 0) {
+    __syncthreads();           // the queries are in shared memory
+#pragma unroll
+    for (int i = 0; i < KQ; ++i) ldmatrix_x4(qr[i], q_base + 2 * ((lane & 15) * ks + (kb_lo + i) * 16 + ((lane >> 4) << 3)));
+  }
+  int buf = 0, fill = ahead;      // the buffer of this chunk, and the one that the next load fills
   for (int c = c_lo; c < c_hi; ++c) {
-    const int buf = (c - c_lo) % a.buffers;
-    if (a.buffers == 3) cp_async_wait<1>();
+    if (a.buffers == 4) cp_async_wait<2>();
+    else if (a.buffers == 3) cp_async_wait<1>();
     else cp_async_wait<0>();
     __syncthreads();           // this chunk has arrived, and the one before is no longer read
-    if (c + ahead < c_hi) load_chunk(c + ahead, (c - c_lo + ahead) % a.buffers);
+    if (c + ahead < c_hi) load_chunk(c + ahead, next_page, fill);
     cp_async_commit();
+    next_page = page_of(c + ahead + 1);
     const uint32_t k_base = smem_u32(Ks + (size_t)buf * 64 * ks);
-    // scores of this warp's eight keys, two sums a row tile so that products do not wait for one another
+    // scores of this warp's eight keys over its half of the columns, two sums a row tile so that products do not wait for one another
     float s[MT][2][4];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[mt][0][e] = s[mt][1][e] = 0.f;
-    const uint32_t k_at = k_base + 2 * ((warp * 8 + (lane & 7)) * ks + (lane >> 3) * 8);
+    const uint32_t k_at = k_base + 2 * ((kt * 8 + (lane & 7)) * ks + (lane >> 3) * 8);
     const uint32_t q_at = q_base + 2 * ((lane & 15) * ks + ((lane >> 4) << 3));
-#pragma unroll 4
-    for (int kb = 0; kb < k16; kb += 2) {
-      uint32_t kf[4];          // two steps of 16 columns; behind an odd last step lies padding or the next row, not used
-      ldmatrix_x4(kf, k_at + 2 * kb * 16);
+    if constexpr (KQ > 0) {
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) {
-        uint32_t qf[4];
-        ldmatrix_x4(qf, q_at + 2 * (mt * 16 * ks + kb * 16));
-        mma_bf16(s[mt][0], qf, kf[0], kf[1]);
-        if (kb + 1 < k16) {
-          ldmatrix_x4(qf, q_at + 2 * (mt * 16 * ks + kb * 16 + 16));
-          mma_bf16(s[mt][1], qf, kf[2], kf[3]);
+      for (int i = 0; i < KQ; i += 2) {
+        uint32_t kf[4];
+        ldmatrix_x4(kf, k_at + 2 * (kb_lo + i) * 16);
+        mma_bf16(s[0][0], qr[i], kf[0], kf[1]);
+        if (i + 1 < KQ) mma_bf16(s[0][1], qr[i + 1 < KQ ? i + 1 : i], kf[2], kf[3]);
+      }
+    } else {
+#pragma unroll 4
+      for (int kb = kb_lo; kb < kb_hi; kb += 2) {
+        uint32_t kf[4];          // two steps of 16 columns; behind an odd last step lies padding or the next row, not used
+        ldmatrix_x4(kf, k_at + 2 * kb * 16);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+          uint32_t qf[4];
+          ldmatrix_x4(qf, q_at + 2 * (mt * 16 * ks + kb * 16));
+          mma_bf16(s[mt][0], qf, kf[0], kf[1]);
+          if (kb + 1 < kb_hi) {
+            ldmatrix_x4(qf, q_at + 2 * (mt * 16 * ks + kb * 16 + 16));
+            mma_bf16(s[mt][1], qf, kf[2], kf[3]);
+          }
         }
       }
     }
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
-      float* at = Ss + (mt * 16 + g) * 68 + warp * 8 + 2 * t4;
+      float* at = Ss + ((warp >> 3) * ROWS + mt * 16 + g) * 68 + kt * 8 + 2 * t4;
       *reinterpret_cast<float2*>(at) = make_float2(s[mt][0][0] + s[mt][1][0], s[mt][0][1] + s[mt][1][1]);
       *reinterpret_cast<float2*>(at + 8 * 68) = make_float2(s[mt][0][2] + s[mt][1][2], s[mt][0][3] + s[mt][1][3]);
     }
@@ -159,7 +185,7 @@ __global__ void __launch_bounds__(256) latent_decode_attn_kernel(const LatentDec
 #pragma unroll
       for (int i = 0; i < KPT; ++i) {
         const int key = k0 + my_key + TPR * i;
-        v[i] = Ss[my_row * 68 + my_key + TPR * i] * scale_log2;
+        v[i] = (Ss[my_row * 68 + my_key + TPR * i] + Ss[(ROWS + my_row) * 68 + my_key + TPR * i]) * scale_log2;
         if (key > pos || key < key_lo) v[i] = -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
@@ -196,7 +222,7 @@ __global__ void __launch_bounds__(256) latent_decode_attn_kernel(const LatentDec
       for (int mt = 0; mt < MT; ++mt) ldmatrix_x4(pf[mt], p_base + 2 * ((mt * 16 + (lane & 15)) * 72 + kk * 16 + ((lane >> 4) << 3)));
 #pragma unroll
       for (int i = 0; i < NP; ++i) {
-        const int col = (warp + 8 * i) * 16;
+        const int col = (warp + kLdWarps * i) * 16;
         if (col < a.R) {
           uint32_t vf[4];
           ldmatrix_x4_trans(vf, k_base + 2 * ((kk * 16 + (lane & 15)) * ks + col + ((lane >> 4) << 3)));
@@ -208,6 +234,8 @@ __global__ void __launch_bounds__(256) latent_decode_attn_kernel(const LatentDec
         }
       }
     }
+    buf = buf + 1 == a.buffers ? 0 : buf + 1;
+    fill = fill + 1 == a.buffers ? 0 : fill + 1;
   }
   cp_async_wait<0>();
   __syncthreads();             // the last chunk's factors have been read
@@ -240,8 +268,8 @@ __global__ void __launch_bounds__(256) latent_decode_attn_kernel(const LatentDec
       const int h = h0 + r;
 #pragma unroll
       for (int i = 0; i < NP; ++i) {
-        const int col = (warp + 8 * i) * 16 + 2 * t4;
-        if ((warp + 8 * i) * 16 >= a.R) continue;
+        const int col = (warp + kLdWarps * i) * 16 + 2 * t4;
+        if ((warp + kLdWarps * i) * 16 >= a.R) continue;
         if (a.splits == 1) {
           const float f = As[r];
           __nv_bfloat16* dst = a.out + ((size_t)h * a.n + seq) * a.R + col;
@@ -524,12 +552,18 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentValueArgs
       if (t < nt) {
         const float* src = a.parts + ((size_t)(t0 + t) * a.H + head) * (a.R + 2) + 2 * p;
         const size_t step = rows * (a.R + 2);
-#pragma unroll 8
-        for (int s = 0; s < a.splits; ++s) {
-          const float f = factor[t][s];
-          const float2 v = f != 0.f ? *reinterpret_cast<const float2*>(src + s * step) : make_float2(0.f, 0.f);
-          vx = fmaf(v.x, f, vx);
-          vy = fmaf(v.y, f, vy);
+        constexpr int kBatch = 12;                // loads in flight; a slice without keys left zeros
+        for (int s0 = 0; s0 < a.splits; s0 += kBatch) {
+          float2 v[kBatch];
+#pragma unroll
+          for (int u = 0; u < kBatch; ++u)
+            v[u] = s0 + u < a.splits ? *reinterpret_cast<const float2*>(src + (size_t)(s0 + u) * step) : make_float2(0.f, 0.f);
+#pragma unroll
+          for (int u = 0; u < kBatch; ++u) {
+            const float f = factor[t][min(s0 + u, 63)];
+            vx = fmaf(v[u].x, f, vx);
+            vy = fmaf(v[u].y, f, vy);
+          }
         }
       }
       const uint32_t at = smem_addr(os + t * ostride + 2 * p), two = pack_bf16(vx, vy);
@@ -560,19 +594,17 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentValueArgs
 
 using namespace slb;
 
-// How the attention kernel is launched for these sizes: row tiles of 16 heads a block, chunks in flight, blocks an SM holds.
-// Two blocks an SM where two chunks each fit, else three chunks in flight where they fit, else two. false: not taken.
+// How the attention kernel is launched for these sizes: row tiles of 16 heads a block, chunks in shared memory (as many of
+// four as fit). false: not taken.
 struct DecodeShape {
-  int mt, buffers, per_sm;
+  int mt, buffers;
 };
 static bool decode_shape(int H, int R, int P, DecodeShape& s) {
   const int W = R + P;
   if (H <= 0 || R <= 0 || P < 0 || R % 16 != 0 || W % 16 != 0 || R > 512) return false;
   for (int mt = H <= 16 ? 1 : (H <= 32 ? 2 : 4); mt >= 1; mt /= 2) {
-    const size_t two = latent_decode_smem(mt, W, 2), three = latent_decode_smem(mt, W, 3);
-    if (2 * (two + 1024) <= kLdMaxSmem) { s = {mt, 2, 2}; return true; }
-    if (three <= kLdMaxSmem) { s = {mt, 3, 1}; return true; }
-    if (two <= kLdMaxSmem) { s = {mt, 2, 1}; return true; }
+    for (int buffers = 4; buffers >= 2; --buffers)
+      if (latent_decode_smem(mt, W, buffers) <= kLdMaxSmem) { s = {mt, buffers}; return true; }
   }
   return false;
 }
@@ -587,9 +619,8 @@ extern "C" int slb_latent_decode_supported(int H, int R, int P) {
 extern "C" int slb_latent_decode_splits(int n, int H, int R, int P, int max_len) {
   DecodeShape s;
   if (n <= 0 || !decode_shape(H, R, P, s)) return 1;
-  const int blocks = n * ((H + 16 * s.mt - 1) / (16 * s.mt));
-  int splits = sm_count() * s.per_sm / blocks;
-  const int pages = (max_len + 63) / 64;
+  const int blocks = n * ((H + 16 * s.mt - 1) / (16 * s.mt)), pages = (max_len + 63) / 64;
+  int splits = sm_count() / blocks;
   if (splits > pages) splits = pages;
   if (splits > 64) splits = 64;
   return splits < 1 ? 1 : splits;
@@ -614,21 +645,27 @@ extern "C" int slb_latent_decode_attention(const void* q_lat, const void* q_raw,
   a.stride = stride; a.n = n; a.H = H; a.R = R; a.P = P; a.dn = dn; a.rot = rot; a.window = window; a.splits = splits;
   a.buffers = shape.buffers; a.scale = scale;
   const size_t smem = latent_decode_smem(shape.mt, R + P, shape.buffers);
-  const dim3 grid(splits, n, (H + 16 * shape.mt - 1) / (16 * shape.mt)), block(256);
+  const dim3 grid(splits, n, (H + 16 * shape.mt - 1) / (16 * shape.mt)), block(kLdThreads);
   cudaStream_t s = (cudaStream_t)stream;
-  const int np = R <= 128 ? 1 : (R <= 256 ? 2 : 4);
-#define SLB_LD(MT, NP)                                                                                                       \
+  const bool one = R <= 256;
+#define SLB_LD(MT, NP, KQ)                                                                                                   \
   do {                                                                                                                       \
     static bool raised = false;                                                                                              \
     if (!raised) {                                                                                                           \
-      cudaFuncSetAttribute(latent_decode_attn_kernel<MT, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLdMaxSmem); \
+      cudaFuncSetAttribute(latent_decode_attn_kernel<MT, NP, KQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLdMaxSmem); \
       raised = true;                                                                                                         \
     }                                                                                                                        \
-    launch(latent_decode_attn_kernel<MT, NP>, grid, block, smem, s, a);                                                      \
+    launch(latent_decode_attn_kernel<MT, NP, KQ>, grid, block, smem, s, a);                                                      \
   } while (0)
 #define SLB_LD_NP(MT) \
-  do { if (np == 1) SLB_LD(MT, 1); else if (np == 2) SLB_LD(MT, 2); else SLB_LD(MT, 4); } while (0)
-  if (shape.mt == 1) SLB_LD_NP(1); else if (shape.mt == 2) SLB_LD_NP(2); else SLB_LD_NP(4);
+  do { if (one) SLB_LD(MT, 1, 0); else SLB_LD(MT, 2, 0); } while (0)
+  if (shape.mt == 1) {
+    const int width = R + P;
+    if (one && width == 64) SLB_LD(1, 1, 2); else if (one && width == 128) SLB_LD(1, 1, 4);
+    else if (one && width == 256) SLB_LD(1, 1, 8); else if (one && width == 288) SLB_LD(1, 1, 9);
+    else if (!one && width == 512) SLB_LD(1, 2, 16); else if (!one && width == 576) SLB_LD(1, 2, 18);
+    else SLB_LD_NP(1);
+  } else if (shape.mt == 2) SLB_LD_NP(2); else SLB_LD_NP(4);
 #undef SLB_LD_NP
 #undef SLB_LD
   return check_launch("latent_decode_attention");
