@@ -462,3 +462,32 @@ def test_the_slices_follow_the_batch_and_the_longest_sequence():
     assert one == 20 and o.latent_decode_splits(1, 16, 256, 0, 64) == 1 and o.latent_decode_splits(1000, 16, 256, 0, 4096) == 1
     assert 1 < o.latent_decode_splits(8, 16, 512, 0, 4096) <= 64
     assert not o.latent_decode_supported(16, 528, 0, 64, 64, torch.bfloat16) and not o.latent_decode_supported(16, 256, 0, 64, 64, torch.float32)
+
+
+@pytest.mark.parametrize("dtype", ["fp32", "bf16"])
+@pytest.mark.parametrize("T, top", [(1, 3), (5, 2)])
+def test_further_rows_join_the_experts_sum(T, top, dtype):
+    """The rows of a shared expert that ran beside the router are added by the experts' last kernel."""
+    o, dt = ops(), DT[dtype]
+    g = torch.Generator().manual_seed(T)
+    E, d, ff = 6, 72, 40
+    h = torch.randn(T, d, generator=g).to(dt)
+    gu, dn = (torch.randn(E, 2 * ff, d, generator=g) / d ** 0.5).to(dt), (torch.randn(E, d, ff, generator=g) / ff ** 0.5).to(dt)
+    choice = torch.stack([torch.randperm(E, generator=g)[:top] for _ in range(T)]).view(-1)
+    weight, x, extra = torch.rand(T * top, generator=g), torch.randn(T, d, generator=g), torch.randn(T, d, generator=g)
+    junk = torch.zeros(max(E, T * top), dtype=torch.int32, device=DEV)
+    got = []
+    for more in (None, extra.to(DEV)):
+        y = x.clone().to(DEV)
+        o.moe_experts(h.to(DEV), gu.to(DEV), dn.to(DEV), junk, junk, weight.to(DEV), torch.empty(T * top, ff, dtype=dt, device=DEV),
+                      torch.empty(T * top, d, device=DEV), y, top, choice=choice.int().to(DEV), extra=more)
+        got.append(y.cpu())
+    torch.testing.assert_close(got[1], got[0] + extra, rtol=1e-5, atol=1e-5)
+    want = x.double()
+    for p, e in enumerate(choice.tolist()):
+        w = {"gate": gu[e, :ff].double(), "up": gu[e, ff:].double(), "down": dn[e].double()}
+        want[p // top] += weight[p].double() * plain.gated_mlp(h[p // top:p // top + 1].double(), w, "")[0]
+    torch.testing.assert_close(got[0].double(), want, **TOL[dtype])
+    with pytest.raises(Exception):
+        o.moe_experts(h.to(DEV), gu.to(DEV), dn.to(DEV), junk, junk, weight.to(DEV), torch.empty(T * top, ff, dtype=dt, device=DEV),
+                      torch.empty(T * top, d, device=DEV), x.to(DEV), top, choice=choice.int().to(DEV), extra=extra[:, :8].to(DEV))
