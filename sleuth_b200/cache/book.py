@@ -10,7 +10,9 @@ kept here.
   group's **block table**: entry ``i`` of the row is the page that holds positions ``64*i .. 64*i+63``.
 * A group with a **window** gives pages back as soon as every position on them has fallen out of the
   window of all future queries, so such a group holds about ``window`` tokens per sequence however
-  long the sequence grows. Positions still map to table entries the same way.
+  long the sequence grows. Positions still map to table entries the same way. Windows are signed numbers: w > 0 means the
+  w most recent positions, w < 0 chunks of -w positions counted from position 0 (a query sees its own chunk only), 0 every
+  earlier position (``first_visible``; csrc/common.cuh first_key is the same rule for the kernels).
 * ``lengths[slot]`` is the number of tokens the sequence holds. Stale contents of a reused page are
   never read: every kernel reads positions below the length only (the reference relies on the same
   idea: entries past ``pos`` are simply overwritten, sleuth/forge/infer/kv_cache.py:52-64).
@@ -41,6 +43,15 @@ class CacheMisuse(RuntimeError):
 
 def pages_for(tokens: int) -> int:
     return (tokens + PAGE_TOKENS - 1) // PAGE_TOKENS
+
+
+def first_visible(position: int, window: int) -> int:
+    """The first position that a query at ``position`` can see under a signed ``window``."""
+    if window > 0:
+        return max(0, position - window + 1)
+    if window < 0:
+        return position // -window * -window
+    return 0
 
 
 class PagePool:
@@ -75,7 +86,7 @@ class PagePool:
 
 @dataclass
 class GroupBook:
-    window: int                 # 0 = keep every position
+    window: int                 # signed, see above; 0 = keep every position
     pool: PagePool
     table: np.ndarray           # [max_slots, stride] int32, -1 = no page
     first_page: np.ndarray      # [max_slots] index of the first table entry still held
@@ -84,7 +95,7 @@ class GroupBook:
 class CacheBook:
     """Slots, lengths and per-group block tables.
 
-    windows: the window of each group (0 = none). n_pages: pages of each group's pool.
+    windows: the signed window of each group (0 = none). n_pages: pages of each group's pool.
     stride: entries per block-table row = pages of the longest sequence allowed.
     """
 
@@ -165,7 +176,7 @@ class CacheBook:
                 peak = max(peak, out)
                 if g.window:
                     for s, n in zip(slots, new_lengths):
-                        keep_from = max(0, n - g.window + 1) // PAGE_TOKENS
+                        keep_from = first_visible(n, g.window) // PAGE_TOKENS
                         if keep_from > first[s]:
                             back = min(have[s], keep_from - first[s])
                             have[s] -= back
@@ -200,8 +211,8 @@ class CacheBook:
             self.lengths[s] = n
             for g in self.groups:
                 if g.window:
-                    # the next query sits at position >= n and sees keys >= n - window + 1
-                    keep_from = max(0, n - g.window + 1) // PAGE_TOKENS
+                    # the next query sits at position >= n; what it sees never begins earlier for later ones
+                    keep_from = first_visible(n, g.window) // PAGE_TOKENS
                     lo = int(g.first_page[s])
                     if keep_from > lo:
                         row = g.table[s]

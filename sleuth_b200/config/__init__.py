@@ -2,6 +2,7 @@
 
 from .base import ConfigError, read_config_json, read_fields
 from .fekitar import FekitarConfig, fekitar_model_spec
+from .levolix import LevolixConfig, levolix_model_spec
 from .lezepel import LezepelConfig, lezepel_model_spec
 from .movalorn import MovalornConfig, movalorn_model_spec
 from .nirozen import NirozenConfig, nirozen_model_spec
@@ -16,7 +17,8 @@ register_architecture("Rabadra", RabadraConfig, rabadra_model_spec, model_types=
 register_architecture("Movalorn", MovalornConfig, movalorn_model_spec, model_types=("movalorn",))
 register_architecture("Nirozen", NirozenConfig, nirozen_model_spec, model_types=("nirozen",))
 register_architecture("Fekitar", FekitarConfig, fekitar_model_spec, model_types=("fekitar",))
+register_architecture("Levolix", LevolixConfig, levolix_model_spec, model_types=("levolix",))
 
-__all__ = ["ConfigError", "read_config_json", "read_fields", "Qwen3Config", "qwen3_model_spec", "LezepelConfig", "lezepel_model_spec", "RabadraConfig", "rabadra_model_spec", "MovalornConfig", "movalorn_model_spec", "NirozenConfig", "nirozen_model_spec", "FekitarConfig", "fekitar_model_spec", "Architecture",
+__all__ = ["ConfigError", "read_config_json", "read_fields", "Qwen3Config", "qwen3_model_spec", "LezepelConfig", "lezepel_model_spec", "RabadraConfig", "rabadra_model_spec", "MovalornConfig", "movalorn_model_spec", "NirozenConfig", "nirozen_model_spec", "FekitarConfig", "fekitar_model_spec", "LevolixConfig", "levolix_model_spec", "Architecture",
            "find_architecture", "parse_config", "register_architecture", "registered_architectures",
            "unregister_architecture"]

@@ -1,7 +1,7 @@
 // Causal grouped-query attention over the paged cache on the tensor cores (bfloat16, head sizes 64 and 128).
 //
 // Same contract as the general kernel (attention_generic.cu): a step has written its keys and values to the
-// cache; a query at position p of sequence s sees keys lo..p of s (lo = max(0, p - window + 1) with a window).
+// cache; a query at position p of sequence s sees keys lo..p of s (lo from common.cuh first_key: window, chunk or 0).
 // Formulas: sleuth/forge/model/attention.py:160-206 (mask, 1/sqrt(head_dim) scale, GQA head mapping, float32
 // softmax); the reference itself calls a library kernel here (F.scaled_dot_product_attention, attention.py:171-193).
 //
@@ -114,7 +114,7 @@ __global__ void __launch_bounds__(kFlashThreads) attn_prefill_kernel(FlashArgs a
   const int t_first = r0 / G;
   const int t_last = min(rows_total - 1, r0 + 63) / G;
   const int p_hi = past + t_last;
-  const int key_lo = a.window > 0 ? max(0, past + t_first - a.window + 1) : 0;
+  const int key_lo = first_key(past + t_first, a.window);
   const int page_lo = key_lo / 64, page_hi = p_hi / 64;
   const int* table = a.block_table + (size_t)seq * a.table_stride;
 
@@ -154,13 +154,13 @@ __global__ void __launch_bounds__(kFlashThreads) attn_prefill_kernel(FlashArgs a
     const int R = r0 + warp * 16 + g + 8 * h;
     const int p = R < rows_total ? past + R / G : -1;      // -1: a padding row sees nothing
     pos_r[h] = p;
-    lo_r[h] = a.window > 0 ? max(0, p - a.window + 1) : 0;
+    lo_r[h] = first_key(p, a.window);
     slope_r[h] = a.slopes != nullptr && R < rows_total ? a.slopes[kh * G + R % G] * kLog2e : 0.0f;
   }
   const int warp_p_min = past + min(rows_total - 1, r0 + warp * 16) / G;
   const int warp_R_last = min(rows_total - 1, r0 + warp * 16 + 15);
   const bool warp_active = r0 + warp * 16 < rows_total;
-  const int warp_lo_max = a.window > 0 ? max(0, past + warp_R_last / G - a.window + 1) : 0;
+  const int warp_lo_max = first_key(past + warp_R_last / G, a.window);
 
   float o[HD / 8][4];
 #pragma unroll
@@ -181,7 +181,7 @@ __global__ void __launch_bounds__(kFlashThreads) attn_prefill_kernel(FlashArgs a
     __syncthreads();
     const int key0 = page * 64;
     // skip pages that lie wholly after this warp's last row or before its first row's window
-    if (warp_active && key0 <= past + warp_R_last / G && key0 + 63 >= (a.window > 0 ? max(0, warp_p_min - a.window + 1) : 0)) {
+    if (warp_active && key0 <= past + warp_R_last / G && key0 + 63 >= first_key(warp_p_min, a.window)) {
       const uint32_t kS = sK + stage * TILE, vS = sV + stage * TILE;
       float s[8][4];
 #pragma unroll
@@ -373,7 +373,7 @@ __global__ void __launch_bounds__(kFlashThreads) attn_decode_kernel(FlashArgs a)
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t4 = lane & 3;
   const int pos = a.past[seq], tok = a.seq_start[seq];
-  const int key_lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int key_lo = first_key(pos, a.window);
   const int page_lo = key_lo / 64, page_hi = pos / 64;
   const int n_pages = page_hi - page_lo + 1;
   const int per = (n_pages + a.splits - 1) / a.splits;
@@ -736,7 +736,7 @@ static int attention_prefill_any(const void* q, const void* k_pool, const void* 
   SLB_REQUIRE(n_seqs >= 0 && max_count >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
               "attention (prefill): seqs=%d max_count=%d heads=%d kv_heads=%d", n_seqs, max_count, heads, kv_heads);
   SLB_REQUIRE(head_dim == 64 || head_dim == 128, "attention (prefill): the tensor-core kernel takes head_dim 64 or 128, got %d", head_dim);
-  SLB_REQUIRE(window >= 0 && table_stride > 0 && n_seqs < 65536 && kv_heads < 65536, "attention (prefill): window=%d table_stride=%d", window, table_stride);
+  SLB_REQUIRE(window > -(1 << 30) && table_stride > 0 && n_seqs < 65536 && kv_heads < 65536, "attention (prefill): window=%d table_stride=%d", window, table_stride);
   if (n_seqs == 0 || max_count == 0) return 0;
   FlashArgs a{};
   a.q = (const __nv_bfloat16*)q; a.k_pool = (const __nv_bfloat16*)k_pool; a.v_pool = (const __nv_bfloat16*)v_pool;
@@ -786,7 +786,7 @@ static int attention_decode_any(const void* q, const void* k_pool, const void* v
   SLB_REQUIRE(n_seqs >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
               "attention (decode): seqs=%d heads=%d kv_heads=%d", n_seqs, heads, kv_heads);
   SLB_REQUIRE(head_dim == 64 || head_dim == 128, "attention (decode): the tensor-core kernel takes head_dim 64 or 128, got %d", head_dim);
-  SLB_REQUIRE(window >= 0 && table_stride > 0 && splits >= 1 && n_seqs < 65536 && kv_heads < 65536,
+  SLB_REQUIRE(window > -(1 << 30) && table_stride > 0 && splits >= 1 && n_seqs < 65536 && kv_heads < 65536,
               "attention (decode): window=%d table_stride=%d splits=%d", window, table_stride, splits);
   const long long need = slb_attention_decode_scratch_floats(n_seqs, heads, head_dim, splits);
   SLB_REQUIRE(need == 0 || (scratch != nullptr && scratch_floats >= need),

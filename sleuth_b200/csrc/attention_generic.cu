@@ -3,7 +3,8 @@
 // It serves every head size (even, up to 256), both dtypes, prompts, single decoded tokens and anything between,
 // because a step first writes its keys and values to the cache and then every query reads all its keys from there.
 // A query at position p of sequence s sees the keys at positions lo..p of s, lo = max(0, p - window + 1) with a
-// window and 0 without (sleuth/forge/model/attention.py:160-169); query head h reads key/value head h / (H / K)
+// window, the start of p's own chunk with chunks (a negative window, common.cuh first_key) and 0 without
+// (sleuth/forge/model/attention.py:160-169); query head h reads key/value head h / (H / K)
 // (attention.py:197-199); scores are (q . k) * scale, softmax and the weighted sum run in float32
 // (attention.py:200-206).
 //
@@ -103,7 +104,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32) attn_generic_kernel(AttnArgs 
   const float slope = a.slopes ? a.slopes[h / maps] : 0.0f;
   const int pos = a.tok_pos[t];
   const int* table = a.block_table + (size_t)a.tok_seq[t] * a.table_stride;
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int lo = first_key(pos, a.window);
 
   const T* qrow = (const T*)a.q + ((size_t)t * a.heads + h) * hd;
   for (int c = threadIdx.x; c < hd; c += kAttnWarps * 32) qs[c] = to_f32(qrow[c]);
@@ -205,7 +206,7 @@ extern "C" int slb_attention_generic(const void* q, const void* k_pool, const vo
               "attention: tokens=%d heads=%d kv_heads=%d", tokens, heads, kv_heads);
   SLB_REQUIRE(head_dim > 0 && head_dim <= 256 && head_dim % 2 == 0,
               "attention: head_dim %d is not supported (even, at most 256)", head_dim);
-  SLB_REQUIRE(window >= 0 && table_stride > 0, "attention: window=%d table_stride=%d", window, table_stride);
+  SLB_REQUIRE(window > -(1 << 30) && table_stride > 0, "attention: window=%d table_stride=%d", window, table_stride);
   if (value_dim == 0) value_dim = head_dim;
   SLB_REQUIRE(value_dim > 0 && value_dim <= 256, "attention: value size %d is not supported (at most 256)", value_dim);
   if (tokens == 0) return 0;
@@ -232,7 +233,7 @@ extern "C" int slb_attention_scored(const void* q, const void* k_pool, const voi
               "attention: tokens=%d heads=%d kv_heads=%d", tokens, heads, kv_heads);
   SLB_REQUIRE(head_dim > 0 && head_dim <= 256 && head_dim % 2 == 0,
               "attention: head_dim %d is not supported (even, at most 256)", head_dim);
-  SLB_REQUIRE(window >= 0 && table_stride > 0, "attention: window=%d table_stride=%d", window, table_stride);
+  SLB_REQUIRE(window > -(1 << 30) && table_stride > 0, "attention: window=%d table_stride=%d", window, table_stride);
   SLB_REQUIRE(maps >= 1 && maps <= 8 && softcap >= 0.0f, "attention: maps=%d softcap=%g", maps, (double)softcap);
   SLB_REQUIRE(gate == nullptr || gate_stride >= (long long)heads * maps * value_dim, "attention: gate rows are too short");
   if (value_dim == 0) value_dim = head_dim;

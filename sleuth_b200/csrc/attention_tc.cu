@@ -1,7 +1,7 @@
 // Attention over the paged cache for steps that bring many tokens (prompts), on the fifth-generation tensor cores.
 //
 // The step has already written its keys and values into the cache; every query row reads the cache
-// (scores = q k^T * scale, causal mask with an optional window, softmax in float32, weighted sum of values:
+// (scores = q k^T * scale, causal mask with an optional window or chunks (common.cuh first_key), softmax in float32, weighted sum of values:
 // sleuth/forge/model/attention.py:131-141, mask sleuth/forge/model/attention.py:57-68). Rows of one
 // (sequence, kv head) are (token, head of the group): row r is token r / G, head kv * G + r % G, so a page of keys
 // serves all G heads of the group.
@@ -158,7 +158,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
   const int r0 = tile * kAtRows;
   const int t_first = r0 / G;
   const int t_last = min(rows_total - 1, r0 + kAtRows - 1) / G;
-  const int key_lo = a.window > 0 ? max(0, past + t_first - a.window + 1) : 0;
+  const int key_lo = first_key(past + t_first, a.window);
   const int page_lo = key_lo / 64, page_hi = (past + t_last) / 64;
   const int n_pages = page_hi - page_lo + 1;
   const int seq_len = past + count;
@@ -275,7 +275,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     const int r = quad * 32 + lane;
     const int R = r0 + r;
     const int pos = R < rows_total ? past + R / G : -1;        // -1: a padding row sees nothing
-    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const int lo = first_key(pos, a.window);
     const uint32_t lane_addr = tmem + ((uint32_t)(quad * 32) << 16);
     unsigned short* xch = reinterpret_cast<unsigned short*>(smem + L::XCH_OFF);     // [2 pages][2 halves][128 rows]
     float m_used = -INFINITY, l = 0.0f;
@@ -475,7 +475,7 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   const int r0 = tile * kAtRows;
   const int t_first = r0 / G;
   const int t_last = min(rows_total - 1, r0 + kAtRows - 1) / G;
-  const int key_lo = a.window > 0 ? max(0, past + t_first - a.window + 1) : 0;
+  const int key_lo = first_key(past + t_first, a.window);
   const int page_lo = key_lo / 64, page_hi = (past + t_last) / 64;
   const int n_pages = page_hi - page_lo + 1;
   const int n_steps = (n_pages + 1) >> 1;
@@ -605,7 +605,7 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int r = quad * 32 + lane;
     const int R = r0 + r;
     const int pos = R < rows_total ? past + R / G : -1;        // -1: a padding row sees nothing
-    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const int lo = first_key(pos, a.window);
     const uint32_t lane_addr = tmem + ((uint32_t)(quad * 32) << 16);
     unsigned short* xch = reinterpret_cast<unsigned short*>(smem + L::XCH_OFF);     // [2 steps][4 parts][128 rows]
     float m_used = -INFINITY, l = 0.0f;
@@ -761,8 +761,8 @@ static bool wide_pays(int n_seqs, int max_count, int max_keys, int heads, int kv
   if (max_keys < max_count) max_keys = max_count;
   int longest = (max_keys + 63) / 64;      // pages of the last tile
   int mean = longest - (max_count / 64) / 2;      // tiles of a prompt grow from its first page to its last
-  if (window > 0) {
-    const int seen = (window + kAtRows / G + 63) / 64 + 1;
+  if (window != 0) {            // a window, or (negative) chunks
+    const int seen = (abs(window) + kAtRows / G + 63) / 64 + 1;
     longest = min(longest, seen);
     mean = min(mean, seen);
   }
@@ -820,7 +820,7 @@ static int attention_tc_any(const void* q, const void* k_pool, const void* v_poo
               "attention (tcgen05): heads=%d kv_heads=%d head_dim=%d is not taken (head size 64 or 128, group size a divisor of 128)",
               heads, kv_heads, head_dim);
   SLB_REQUIRE(scale > 0.0f, "attention (tcgen05): the kernel takes a positive scale, got %g", (double)scale);
-  SLB_REQUIRE(n_seqs >= 0 && max_count >= 0 && window >= 0 && table_stride > 0 && n_seqs < 65536 && kv_heads < 65536 &&
+  SLB_REQUIRE(n_seqs >= 0 && max_count >= 0 && window > -(1 << 30) && table_stride > 0 && n_seqs < 65536 && kv_heads < 65536 &&
               tokens >= 0 && pool_pages > 0 && status != nullptr,
               "attention (tcgen05): seqs=%d max_count=%d window=%d table_stride=%d", n_seqs, max_count, window, table_stride);
   SLB_REQUIRE(pool_pages * kv_heads * 64 < (1ll << 31), "attention (tcgen05): the pool has too many rows for one tensor map");

@@ -39,6 +39,15 @@ __device__ __forceinline__ void pdl_enter() {
   pdl_wait();
 }
 
+// Which keys a query sees. `window` w > 0: the w most recent positions, the query's own included. w < 0: the positions of
+// the query's own chunk of -w, chunks being counted from position 0 of the sequence. 0: every earlier position. All
+// attention kernels and the cache's book (cache/book.py) share this convention; never decreasing in the position.
+__host__ __device__ __forceinline__ int first_key(int pos, int window) {
+  if (window > 0) return pos - window + 1 > 0 ? pos - window + 1 : 0;
+  if (window < 0) return pos / -window * -window;
+  return 0;
+}
+
 // A range of memory that the kernel after this one will read and that no kernel writes (the next weight matrix).
 // The blocks of a kernel that is given one ask the L2 cache for it, a share each, so that the next kernel finds its
 // weights on the chip: a single-token step leaves the memory system idle more than half of the time, and a kernel
@@ -82,7 +91,7 @@ __device__ __forceinline__ void prefetch_page_item(const NextPages& p, int item,
   const int slice = rest % p.splits, seq = rest / p.splits;
   if (seq >= p.n_seqs) return;
   const int pos = p.past[seq];
-  const int key_lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int key_lo = first_key(pos, p.window);
   const int page_lo = key_lo / 64, page_hi = pos / 64;
   const int per = (page_hi - page_lo + 1 + p.splits - 1) / p.splits;
   const int my_lo = page_lo + slice * per, my_hi = min(page_hi, my_lo + per - 1);

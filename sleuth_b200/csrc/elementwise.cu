@@ -339,18 +339,28 @@ __global__ void pair_embed_kernel(const int* __restrict__ ids, const int* __rest
 // The end of a sublayer that is gated and normalised before it joins the stream:
 //   v = y * sigmoid(g + b) (g absent: v = y);  x += v / sqrt(mean(v^2) + eps) * w
 // y [T, dim] float32 (rows too wide for a thread's registers are overwritten with v), g [T, dim] float32 with row stride
-// g_stride, b and w [dim] float32.
+// g_stride, b and w [dim] float32. With y2 [T, dim] (two results side by side, not together with g) v = s1 * y + s2 * y2. With
+// `rounded` [T, dim] the new row of x is also stored there as bfloat16 (what a sublayer that reads the stream itself reads).
+struct SecondResult {
+  const float* y2;
+  float s1, s2;
+  __nv_bfloat16* rounded;
+};
+
 __global__ void gated_norm_add_kernel(float* __restrict__ x, float* __restrict__ y, const float* __restrict__ g,
                                       long long g_stride, const float* __restrict__ b, const float* __restrict__ w, int dim,
-                                      float eps) {
+                                      float eps, SecondResult two) {
   pdl_enter();
   __shared__ float scratch[33];
   constexpr int kKeep = 8;      // values a thread keeps between the two passes; rows wider than that park the rest in y
   const int r = blockIdx.x;
   float* yr = y + (size_t)r * dim;
   const float* gr = g ? g + (size_t)r * g_stride : nullptr;
+  const float* yr2 = two.y2 ? two.y2 + (size_t)r * dim : nullptr;
+  __nv_bfloat16* rr = two.rounded ? two.rounded + (size_t)r * dim : nullptr;
   auto gated = [&](int i) {
     float v = yr[i];
+    if (yr2) v = two.s1 * v + two.s2 * yr2[i];
     if (gr) {
       const float z = gr[i] + (b ? b[i] : 0.0f);
       v = v * (1.0f / (1.0f + expf(-z)));
@@ -378,9 +388,17 @@ __global__ void gated_norm_add_kernel(float* __restrict__ x, float* __restrict__
 #pragma unroll
   for (int k = 0; k < kKeep; ++k) {
     const int i = threadIdx.x + k * blockDim.x;
-    if (i < dim) xr[i] += (keep[k] * inv) * w[i];
+    if (i < dim) {
+      const float v = xr[i] + (keep[k] * inv) * w[i];
+      xr[i] = v;
+      if (rr) rr[i] = __float2bfloat16_rn(v);
+    }
   }
-  for (int i = threadIdx.x + kKeep * blockDim.x; i < dim; i += blockDim.x) xr[i] += (yr[i] * inv) * w[i];
+  for (int i = threadIdx.x + kKeep * blockDim.x; i < dim; i += blockDim.x) {
+    const float v = xr[i] + (yr[i] * inv) * w[i];
+    xr[i] = v;
+    if (rr) rr[i] = __float2bfloat16_rn(v);
+  }
 }
 
 // The same for rows of whole float4s that fit a block's registers (PER float4s a thread): every load of the row, its gate,
@@ -389,11 +407,12 @@ template <int PER>
 __global__ void __launch_bounds__(256) gated_norm_add_vec_kernel(float* __restrict__ x, const float* __restrict__ y,
                                                                  const float* __restrict__ g, long long g_stride,
                                                                  const float* __restrict__ b, const float* __restrict__ w, int dim,
-                                                                 float eps) {
+                                                                 float eps, SecondResult two) {
   pdl_enter();
   __shared__ float scratch[33];
   const int r = blockIdx.x, n4 = dim >> 2;
   const float4* yr = reinterpret_cast<const float4*>(y + (size_t)r * dim);
+  const float4* yr2 = two.y2 ? reinterpret_cast<const float4*>(two.y2 + (size_t)r * dim) : nullptr;
   const float4* gr = g ? reinterpret_cast<const float4*>(g + (size_t)r * g_stride) : nullptr;
   const float4* b4 = reinterpret_cast<const float4*>(b);
   const float4* w4 = reinterpret_cast<const float4*>(w);
@@ -405,7 +424,7 @@ __global__ void __launch_bounds__(256) gated_norm_add_vec_kernel(float* __restri
     const int c = threadIdx.x + k * blockDim.x;
     const bool in = c < n4;
     v[k] = in ? yr[c] : zero;
-    z[k] = in && gr ? gr[c] : zero;
+    z[k] = in && gr ? gr[c] : (in && yr2 ? yr2[c] : zero);       // the gate's row or the second result's
     bias[k] = in && gr && b ? b4[c] : zero;
     xv[k] = in ? xr[c] : zero;
     gains[k] = in ? w4[c] : zero;
@@ -413,6 +432,10 @@ __global__ void __launch_bounds__(256) gated_norm_add_vec_kernel(float* __restri
   float ss = 0.0f;
 #pragma unroll
   for (int k = 0; k < PER; ++k) {
+    if (yr2) {
+      v[k] = make_float4(two.s1 * v[k].x + two.s2 * z[k].x, two.s1 * v[k].y + two.s2 * z[k].y, two.s1 * v[k].z + two.s2 * z[k].z,
+                         two.s1 * v[k].w + two.s2 * z[k].w);
+    }
     if (gr) {
       v[k].x = v[k].x * (1.0f / (1.0f + expf(-(z[k].x + bias[k].x))));
       v[k].y = v[k].y * (1.0f / (1.0f + expf(-(z[k].y + bias[k].y))));
@@ -430,8 +453,14 @@ __global__ void __launch_bounds__(256) gated_norm_add_vec_kernel(float* __restri
   for (int k = 0; k < PER; ++k) {
     const int c = threadIdx.x + k * blockDim.x;
     if (c >= n4) continue;
-    xr[c] = make_float4(xv[k].x + (v[k].x * inv) * gains[k].x, xv[k].y + (v[k].y * inv) * gains[k].y,
-                        xv[k].z + (v[k].z * inv) * gains[k].z, xv[k].w + (v[k].w * inv) * gains[k].w);
+    const float4 sum = make_float4(xv[k].x + (v[k].x * inv) * gains[k].x, xv[k].y + (v[k].y * inv) * gains[k].y,
+                                   xv[k].z + (v[k].z * inv) * gains[k].z, xv[k].w + (v[k].w * inv) * gains[k].w);
+    xr[c] = sum;
+    if (two.rounded) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(sum.x, sum.y), hi = __floats2bfloat162_rn(sum.z, sum.w);
+      reinterpret_cast<uint2*>(two.rounded + (size_t)r * dim)[c] =
+          make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
   }
 }
 
@@ -689,26 +718,29 @@ extern "C" int slb_sinusoid_add(float* x, const int* tok_pos, const double* turn
 }
 
 extern "C" int slb_gated_norm_add(float* x, float* y, const float* g, long long g_stride, const float* b, const float* w,
-                                  int rows, int dim, float eps, void* stream) {
+                                  int rows, int dim, float eps, const float* y2, float s1, float s2, void* rounded, void* stream) {
+  SLB_REQUIRE(g == nullptr || y2 == nullptr, "gated_norm_add: a gate and a second result do not go together");
+  const SecondResult two{y2, s1, s2, (__nv_bfloat16*)rounded};
   SLB_REQUIRE(rows >= 0 && dim > 0 && eps > 0.0f && (g == nullptr || g_stride >= dim), "gated_norm_add: rows=%d dim=%d eps=%g", rows,
               dim, (double)eps);
   if (rows == 0) return 0;
   auto aligned = [](const void* p) { return (uintptr_t)p % 16 == 0; };
   // one block shape for a width whatever the row count, so that a row's sum is formed in the same order in every step
-  if (dim % 4 == 0 && dim <= 4096 && g_stride % 4 == 0 && aligned(x) && aligned(y) && aligned(g) && aligned(b) && aligned(w)) {
+  if (dim % 4 == 0 && dim <= 4096 && g_stride % 4 == 0 && aligned(x) && aligned(y) && aligned(g) && aligned(b) && aligned(w) &&
+      aligned(y2) && aligned(rounded)) {
     const int n4 = dim / 4;
     const int threads = n4 <= 64 ? 64 : (n4 <= 128 ? 128 : 256);
     const int per = (n4 + threads - 1) / threads;      // at most 4
     const float* yc = y;
     if (per <= 1)
-      launch(gated_norm_add_vec_kernel<1>, dim3(rows), dim3(threads), 0, (cudaStream_t)stream, x, yc, g, g_stride, b, w, dim, eps);
+      launch(gated_norm_add_vec_kernel<1>, dim3(rows), dim3(threads), 0, (cudaStream_t)stream, x, yc, g, g_stride, b, w, dim, eps, two);
     else if (per <= 2)
-      launch(gated_norm_add_vec_kernel<2>, dim3(rows), dim3(threads), 0, (cudaStream_t)stream, x, yc, g, g_stride, b, w, dim, eps);
+      launch(gated_norm_add_vec_kernel<2>, dim3(rows), dim3(threads), 0, (cudaStream_t)stream, x, yc, g, g_stride, b, w, dim, eps, two);
     else
-      launch(gated_norm_add_vec_kernel<4>, dim3(rows), dim3(threads), 0, (cudaStream_t)stream, x, yc, g, g_stride, b, w, dim, eps);
+      launch(gated_norm_add_vec_kernel<4>, dim3(rows), dim3(threads), 0, (cudaStream_t)stream, x, yc, g, g_stride, b, w, dim, eps, two);
     return check_launch("gated_norm_add");
   }
-  launch(gated_norm_add_kernel, dim3(rows), dim3(norm_threads(dim)), 0, (cudaStream_t)stream, x, y, g, g_stride, b, w, dim, eps);
+  launch(gated_norm_add_kernel, dim3(rows), dim3(norm_threads(dim)), 0, (cudaStream_t)stream, x, y, g, g_stride, b, w, dim, eps, two);
   return check_launch("gated_norm_add");
 }
 

@@ -326,7 +326,7 @@ static int take_pages(SkinnyArgs& a, const NextPages* pages) {
   if (pages == nullptr || pages->k_pool == nullptr) return 0;
   SLB_REQUIRE(pages->v_pool && pages->block_table && pages->past && pages->page_bytes > 0 && pages->page_bytes % 16 == 0 &&
               (uintptr_t)pages->k_pool % 16 == 0 && (uintptr_t)pages->v_pool % 16 == 0 && pages->table_stride > 0 &&
-              pages->n_seqs > 0 && pages->splits > 0 && pages->depth > 0 && pages->window >= 0 &&
+              pages->n_seqs > 0 && pages->splits > 0 && pages->depth > 0 && pages->window > -(1 << 30) &&
               pages->page_bytes <= 32 * 32768,
               "gemm_skinny: the description of the pages to prefetch is incomplete");
   a.pages = *pages;

@@ -12,7 +12,10 @@
 //                        expert-ordered list, list[place] = pair
 //   moe_gate_up_kernel   act[place, j] = f(gate_e[j] . h, up_e[j] . h), f one of the gated activations of common.cuh
 //   moe_down_kernel      y[pair, :] = weight[pair] * (down_e act[place])   (float32)
-//   moe_combine_kernel   x[t, :] += sum over the token's choices of y, in the order of the choices
+//   moe_combine_kernel   x[t, :] += sum over the token's choices of y, in the order of the choices (or = , into an empty row)
+// The last experts of the router may be identity experts: they have no matrices and return the token's own input row. They
+// come last in the expert order too, so the product kernels, which are given the number of experts that have matrices, never
+// meet their pairs; the kernels that sum a token's choices add weight * h for them.
 // In bfloat16 with inner sizes that are multiples of 8 the two products run on the tensor cores (moe_mma_kernel);
 // the kernels above then serve float32 and odd sizes.
 #include "mma_sync.cuh"
@@ -250,10 +253,10 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ h,
 // pair's turn there, and list[place] = pair. The turns come from shared-memory counters, so which of an expert's rows
 // a pair gets may differ from run to run; every pair's result is computed from its own row alone, so nothing else does.
 // With `tiles`: also the experts' row tiles of `tile_rows` rows for the grouped product: [0] = their number, then
-// (expert, first row, rows) each.
+// (expert, first row, rows) each, for the first `tiled` experts (those that have matrices).
 __global__ void __launch_bounds__(1024) moe_group_kernel(const int* __restrict__ choice, int* __restrict__ counts,
                                                          int* __restrict__ place, int* __restrict__ list, int pairs, int E,
-                                                         int* __restrict__ tiles, int tile_rows) {
+                                                         int tiled, int* __restrict__ tiles, int tile_rows) {
   pdl_enter();
   extern __shared__ int sh[];          // [E] counts, then [E] first rows / cursors
   int* cnt = sh;
@@ -279,7 +282,7 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int* __restrict__
     __syncwarp();
     if (tiles != nullptr && threadIdx.x == 0) {
       int n = 0;
-      for (int e = 0; e < E; ++e)
+      for (int e = 0; e < tiled; ++e)        // identity experts have no product and no tiles
         for (int r = 0; r < cnt[e]; r += tile_rows) {
           tiles[1 + 3 * n] = e;
           tiles[2 + 3 * n] = cur[e] + r;
@@ -538,12 +541,13 @@ __global__ void __launch_bounds__(128) moe_mma_kernel(const __nv_bfloat16* __res
 template <typename T>
 __global__ void __launch_bounds__(256) moe_few_gate_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gu,
                                                               const int* __restrict__ choice, T* __restrict__ act, int top,
-                                                              int dim, int ff, GateAct gate) {
+                                                              int dim, int ff, int E, GateAct gate) {
   pdl_enter();
   const int pair = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int j = blockIdx.y * 8 + warp;
   if (j >= ff) return;
   const int e = choice[pair];
+  if (e >= E) return;                  // an identity expert
   const T* x = h + (size_t)(pair / top) * dim;
   const T* wg = w_gu + ((size_t)e * 2 * ff + j) * dim;
   const T* wu = wg + (size_t)ff * dim;
@@ -582,13 +586,13 @@ __global__ void __launch_bounds__(256) moe_few_gate_up_kernel(const T* __restric
   }
 }
 
-// grid (tokens, column groups of 8): x[t, n] += sum over the token's choices, in their order, of
-// weight[pair] * (down_e[n] . act[pair]).
+// grid (tokens, column groups of 8): x[t, n] += (store: =) sum over the token's choices, in their order, of
+// weight[pair] * (down_e[n] . act[pair]), or weight[pair] * h[t, n] for an identity expert (e >= E).
 template <typename T>
-__global__ void __launch_bounds__(256) moe_few_down_kernel(const T* __restrict__ act, const T* __restrict__ w_down,
+__global__ void __launch_bounds__(256) moe_few_down_kernel(const T* __restrict__ h, const T* __restrict__ act, const T* __restrict__ w_down,
                                                            const int* __restrict__ choice, const float* __restrict__ weight,
                                                            float* __restrict__ x, const float* __restrict__ extra, int top, int dim,
-                                                           int ff) {
+                                                           int ff, int E, int store) {
   pdl_enter();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = blockIdx.y * 8 + warp;
@@ -596,6 +600,10 @@ __global__ void __launch_bounds__(256) moe_few_down_kernel(const T* __restrict__
   float total = 0.f;
   for (int k = 0; k < top; ++k) {
     const int pair = t * top + k;
+    if (choice[pair] >= E) {
+      total = fmaf(weight[pair], to_f32(h[(size_t)t * dim + n]), total);
+      continue;
+    }
     const T* a = act + (size_t)pair * ff;
     const T* w = w_down + ((size_t)choice[pair] * dim + n) * ff;
     float s = 0.f;
@@ -616,18 +624,37 @@ __global__ void __launch_bounds__(256) moe_few_down_kernel(const T* __restrict__
     }
     total = fmaf(weight[pair], warp_sum(s), total);
   }
-  if (lane == 0) x[(size_t)t * dim + n] += extra ? total + extra[(size_t)t * dim + n] : total;
+  if (lane == 0) {
+    if (extra) total += extra[(size_t)t * dim + n];
+    float* dst = x + (size_t)t * dim + n;
+    *dst = store ? total : *dst + total;
+  }
 }
 
-__global__ void moe_combine_kernel(float* __restrict__ x, const float* __restrict__ y, int top, int dim, size_t total) {
+// What the kernels that sum a token's choices need to know of identity experts: the choices, the number of experts that
+// have matrices and the tokens' input rows (all unused when `choice` is null).
+struct IdentityRows {
+  const int* choice;
+  const float* weight;
+  const void* h;
+  int E;
+};
+
+template <typename T>
+__global__ void moe_combine_kernel(float* __restrict__ x, const float* __restrict__ y, int top, int dim, size_t total,
+                                   IdentityRows same, int store) {
   pdl_enter();
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t step = (size_t)gridDim.x * blockDim.x;
   for (; i < total; i += step) {
     const size_t t = i / dim, d = i - t * dim;
     float s = 0.f;
-    for (int k = 0; k < top; ++k) s += y[(t * top + k) * dim + d];
-    x[i] += s;
+    for (int k = 0; k < top; ++k) {
+      const size_t pair = t * top + k;
+      if (same.choice && same.choice[pair] >= same.E) s = fmaf(same.weight[pair], to_f32(((const T*)same.h)[i]), s);
+      else s += y[pair * dim + d];
+    }
+    x[i] = store ? s : x[i] + s;
   }
 }
 
@@ -644,16 +671,53 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ h, const int
 
 // x[t, :] += sum over the token's choices, in their order, of weight[pair] * y[place[pair], :] (y in the expert order).
 __global__ void moe_combine_sorted_kernel(float* __restrict__ x, const float* __restrict__ y, const int* __restrict__ place,
-                                          const float* __restrict__ weight, int top, int dim, size_t total) {
+                                          const float* __restrict__ weight, int top, int dim, size_t total,
+                                          IdentityRows same, int store) {
   pdl_enter();
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t step = (size_t)gridDim.x * blockDim.x;
   for (; i < total; i += step) {
     const size_t t = i / dim, d = i - t * dim;
     float s = 0.f;
-    for (int k = 0; k < top; ++k) s = fmaf(weight[t * top + k], y[(size_t)place[t * top + k] * dim + d], s);
-    x[i] += s;
+    for (int k = 0; k < top; ++k) {
+      const size_t pair = t * top + k;
+      const float v = same.choice && same.choice[pair] >= same.E ? to_f32(((const __nv_bfloat16*)same.h)[i]) : y[(size_t)place[pair] * dim + d];
+      s = fmaf(weight[pair], v, s);
+    }
+    x[i] = store ? s : x[i] + s;
   }
+}
+
+// The same in pieces of four columns (dim a multiple of 4): one index computation and `top` 16-byte loads a piece.
+__global__ void __launch_bounds__(256) moe_combine_sorted_vec_kernel(float4* __restrict__ x, const float4* __restrict__ y,
+                                                                     const int* __restrict__ place, const float* __restrict__ weight,
+                                                                     int top, int dim4, size_t total4, IdentityRows same, int store) {
+  pdl_enter();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total4) return;
+  const size_t t = i / dim4, d = i - t * dim4;
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int k = 0; k < top; ++k) {
+    const size_t pair = t * top + k;
+    const float w = weight[pair];
+    float4 v;
+    if (same.choice && same.choice[pair] >= same.E) {
+      const uint2 p = reinterpret_cast<const uint2*>(same.h)[i];
+      const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&p.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&p.y));
+      v = make_float4(lo.x, lo.y, hi.x, hi.y);
+    } else {
+      v = y[(size_t)place[pair] * dim4 + d];
+    }
+    s.x = fmaf(w, v.x, s.x);
+    s.y = fmaf(w, v.y, s.y);
+    s.z = fmaf(w, v.z, s.z);
+    s.w = fmaf(w, v.w, s.w);
+  }
+  if (!store) {
+    const float4 old = x[i];
+    s = make_float4(old.x + s.x, old.y + s.y, old.z + s.z, old.w + s.w);
+  }
+  x[i] = s;
 }
 
 }  // namespace slb
@@ -670,7 +734,7 @@ extern "C" int slb_gemm_tc_grouped_gated(const void* X, const void* W, void* C, 
 extern "C" int slb_moe_experts_tc(const void* h, const void* w_gu, const void* w_down, const int* list, const int* place,
                                   const float* weight, const int* tiles, void* xs, void* act, float* y, float* x, int tokens,
                                   int dim, int ff, int E, int top, int act_kind, float act_limit, float act_alpha,
-                                  int* status, void* stream) {
+                                  const int* choice, int store, int* status, void* stream) {
   SLB_REQUIRE(tokens > 0 && dim > 0 && ff > 0 && E > 0 && top > 0 && dim % 8 == 0 && ff % 8 == 0,
               "moe_experts_tc: tokens=%d dim=%d ff=%d experts=%d top=%d (inner sizes must be multiples of 8)", tokens, dim, ff, E, top);
   SLB_REQUIRE(tiles != nullptr && status != nullptr, "moe_experts_tc: the row tiles and the status word are needed");
@@ -689,23 +753,31 @@ extern "C" int slb_moe_experts_tc(const void* h, const void* w_gu, const void* w
                                  stream);
   if (rc) return rc;
   const size_t total = (size_t)tokens * dim;
+  const IdentityRows same{choice, weight, h, E};
+  if (dim % 4 == 0 && ((uintptr_t)x | (uintptr_t)y | (uintptr_t)h) % 16 == 0) {
+    launch(moe_combine_sorted_vec_kernel, dim3((unsigned)((total / 4 + 255) / 256)), dim3(256), 0, s, (float4*)x, (const float4*)y, place, weight,
+           top, dim / 4, total / 4, same, store);
+    return check_launch("moe_combine");
+  }
   size_t blocks = (total + 255) / 256;
   if (blocks > (size_t)sm_count() * 16) blocks = (size_t)sm_count() * 16;
-  launch(moe_combine_sorted_kernel, dim3((unsigned)blocks), dim3(256), 0, s, x, (const float*)y, place, weight, top, dim, total);
+  launch(moe_combine_sorted_kernel, dim3((unsigned)blocks), dim3(256), 0, s, x, (const float*)y, place, weight, top, dim, total, same, store);
   return check_launch("moe_combine");
 }
 
+// E counts all experts of the router, of which the last `identity` have no matrices.
 // choice, place, list: int32 [tokens * top]; weight: float32 [tokens * top]; counts: int32 [E] (written here).
 // logits: float32 scratch [tokens, E], or null (then every token's block forms its own logits); with logits_ready they
 // hold the logits already (a matrix product formed them) and nothing is computed from h. tiles: int32
 // [1 + 3 * (tokens * top / 128 + min(tokens * top, E))] for the grouped tensor-memory product, or null.
 extern "C" int slb_moe_route(const void* h, const float* w_router, const float* bias, const float* pick_bias, int* choice, float* weight,
                              int* rank, int* counts, int* place, int* list, float* logits, int* tiles, int layout,
-                             int tokens, int dim, int E, int top, int scoring, int groups, int keep, float route_scale,
+                             int tokens, int dim, int E, int identity, int top, int scoring, int groups, int keep, float route_scale,
                              int logits_ready, int dtype, void* stream) {
   SLB_REQUIRE(tokens >= 0 && dim > 0 && E > 0 && top > 0 && top <= E, "moe_route: tokens=%d dim=%d experts=%d top=%d",
               tokens, dim, E, top);
   SLB_REQUIRE(E <= 4096, "moe_route: at most 4096 experts, got %d", E);
+  SLB_REQUIRE(identity >= 0 && identity <= E, "moe_route: %d identity experts of %d", identity, E);
   SLB_REQUIRE(dtype == kF32 || dtype == kBF16, "moe_route: unknown dtype %d", dtype);
   SLB_REQUIRE(scoring >= 0 && scoring <= 3, "moe_route: unknown scoring %d", scoring);
   SLB_REQUIRE(pick_bias == nullptr || scoring >= 2, "moe_route: a choice correction goes with the softmax scoring over all experts");
@@ -752,10 +824,11 @@ extern "C" int slb_moe_route(const void* h, const float* w_router, const float* 
   if (rc || !layout) return rc;        // a step of few pairs needs no counts and no expert order
   const int pairs = tokens * top;
   launch(moe_group_kernel, dim3(1), dim3(pairs >= 1024 ? 1024 : 256), 2 * sizeof(int) * E, s, (const int*)choice, counts, place, list,
-         pairs, E, tiles, 128);
+         pairs, E, E - identity, tiles, 128);
   return check_launch("moe_group");
 }
 
+// E: the experts that have matrices; `identity` more may be among the choices (numbers E ..). store: x = the sum instead of x += .
 // act: [tokens * top, ff] in the run dtype; y: float32 [tokens * top, dim]; x: the float32 stream [tokens, dim]; extra: null,
 // or float32 [tokens, dim] rows that the same kernel adds into the stream (steps of few pairs only).
 // choice (from slb_moe_route) serves steps of few pairs, which run a warp per output instead of tiles and need neither
@@ -763,11 +836,12 @@ extern "C" int slb_moe_route(const void* h, const float* w_router, const float* 
 extern "C" int slb_moe_experts(const void* h, const void* w_gu, const void* w_down, const int* counts, const int* list,
                                const int* choice, const int* place, const float* weight, void* act, float* y, float* x,
                                const float* extra, int tokens, int dim, int ff, int E, int top, int act_kind, float act_limit,
-                               float act_alpha, int dtype, void* stream) {
+                               float act_alpha, int identity, int store, int dtype, void* stream) {
   SLB_REQUIRE(tokens >= 0 && dim > 0 && ff > 0 && E > 0 && top > 0, "moe_experts: tokens=%d dim=%d ff=%d experts=%d top=%d",
               tokens, dim, ff, E, top);
   SLB_REQUIRE(dtype == kF32 || dtype == kBF16, "moe_experts: unknown dtype %d", dtype);
   SLB_REQUIRE(act_kind >= kGateSilu && act_kind <= kGateLast, "moe_experts: unknown activation %d", act_kind);
+  SLB_REQUIRE(identity == 0 || choice != nullptr, "moe_experts: identity experts need the choices");
   if (tokens == 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   const GateAct gate{act_kind, act_limit, act_alpha};
@@ -781,13 +855,13 @@ extern "C" int slb_moe_experts(const void* h, const void* w_gu, const void* w_do
   if (pairs <= kMoeFewPairs && choice != nullptr && (dtype == kF32 || aligned)) {
     const dim3 f1((unsigned)pairs, (ff + 7) / 8), f2((unsigned)tokens, (dim + 7) / 8);
     if (dtype == kF32) {
-      launch(moe_few_gate_up_kernel<float>, f1, block, 0, s, (const float*)h, (const float*)w_gu, choice, (float*)act, top, dim, ff, gate);
-      launch(moe_few_down_kernel<float>, f2, block, 0, s, (const float*)act, (const float*)w_down, choice, weight, x, extra, top, dim, ff);
+      launch(moe_few_gate_up_kernel<float>, f1, block, 0, s, (const float*)h, (const float*)w_gu, choice, (float*)act, top, dim, ff, E, gate);
+      launch(moe_few_down_kernel<float>, f2, block, 0, s, (const float*)h, (const float*)act, (const float*)w_down, choice, weight, x, extra, top, dim, ff, E, store);
     } else {
       launch(moe_few_gate_up_kernel<__nv_bfloat16>, f1, block, 0, s, (const __nv_bfloat16*)h, (const __nv_bfloat16*)w_gu, choice,
-             (__nv_bfloat16*)act, top, dim, ff, gate);
-      launch(moe_few_down_kernel<__nv_bfloat16>, f2, block, 0, s, (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, choice,
-             weight, x, extra, top, dim, ff);
+             (__nv_bfloat16*)act, top, dim, ff, E, gate);
+      launch(moe_few_down_kernel<__nv_bfloat16>, f2, block, 0, s, (const __nv_bfloat16*)h, (const __nv_bfloat16*)act, (const __nv_bfloat16*)w_down, choice,
+             weight, x, extra, top, dim, ff, E, store);
     }
     return check_launch("moe_experts");          // the down kernel has added into the stream already
   }
@@ -813,6 +887,8 @@ extern "C" int slb_moe_experts(const void* h, const void* w_gu, const void* w_do
   const size_t total = (size_t)tokens * dim;
   size_t blocks = (total + 255) / 256;
   if (blocks > (size_t)sm_count() * 16) blocks = (size_t)sm_count() * 16;
-  launch(moe_combine_kernel, dim3((unsigned)blocks), block, 0, s, x, (const float*)y, top, dim, total);
+  const IdentityRows same{identity ? choice : nullptr, weight, h, E};
+  if (dtype == kF32) launch(moe_combine_kernel<float>, dim3((unsigned)blocks), block, 0, s, x, (const float*)y, top, dim, total, same, store);
+  else launch(moe_combine_kernel<__nv_bfloat16>, dim3((unsigned)blocks), block, 0, s, x, (const float*)y, top, dim, total, same, store);
   return check_launch("moe_combine");
 }

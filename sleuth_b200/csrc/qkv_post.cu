@@ -227,7 +227,9 @@ static int launch_qkv_post(const QkvPostArgs& a, cudaStream_t s) {
 // the sums of squares are formed in an order that the row's layout alone fixes, so a token's result depends on nothing
 // but its own row.
 struct QkvSpanArgs {
-  const float* qkv;         // [tokens, H * dk + G * dk + G * dv]
+  const float* qkv;         // [tokens, row_stride], of which H * dk + G * dk + G * dv values count
+  long long row_stride;
+  const float* bias;        // [H * dk + G * dk + G * dv] or null: added to the row first
   const float* q_gain;      // null: no norm
   const float* k_gain;
   const float* cos_table;   // [positions, rot / 2] or null
@@ -258,8 +260,8 @@ __global__ void __launch_bounds__(256) qkv_post_span_kernel(QkvSpanArgs a) {
   __shared__ float scratch[33];
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int H = a.heads, G = a.kv_heads, dk = a.key_dim, dv = a.value_dim;
-  const size_t row_len = (size_t)(H + G) * dk + (size_t)G * dv;
-  const float* row = a.qkv + (size_t)t * row_len;
+  const float* row = a.qkv + (size_t)t * a.row_stride;
+  auto at = [&](int i) { return a.bias ? row[i] + a.bias[i] : row[i]; };
   const bool normed = a.q_gain != nullptr;
   // the token's place in the cache is looked up first: these dependent loads then overlap the row's
   const int pos = a.tok_pos[t];
@@ -271,17 +273,17 @@ __global__ void __launch_bounds__(256) qkv_post_span_kernel(QkvSpanArgs a) {
   if (normed && a.whole) {
     const int nq = H * dk, nk = G * dk;
     float sq = 0.0f, sk = 0.0f;
-    for (int i = threadIdx.x; i < nq; i += nthreads) sq = fmaf(row[i], row[i], sq);
-    for (int i = threadIdx.x; i < nk; i += nthreads) sk = fmaf(row[nq + i], row[nq + i], sk);
+    for (int i = threadIdx.x; i < nq; i += nthreads) { const float x = at(i); sq = fmaf(x, x, sq); }
+    for (int i = threadIdx.x; i < nk; i += nthreads) { const float x = at(nq + i); sk = fmaf(x, x, sk); }
     sq = block_sum(sq, scratch);
     sk = block_sum(sk, scratch);
     inv_q = 1.0f / sqrtf(sq / (float)(H * a.norm_dim) + a.eps);
     inv_k = 1.0f / sqrtf(sk / (float)(G * a.norm_dim) + a.eps);
   } else if (normed) {
     for (int hh = hh0 + warp; hh < hh1; hh += nwarps) {
-      const float* src = row + (size_t)hh * dk;
+      const int at0 = hh * dk;
       float ss = 0.0f;
-      for (int c = lane; c < dk; c += 32) ss = fmaf(src[c], src[c], ss);
+      for (int c = lane; c < dk; c += 32) { const float x = at(at0 + c); ss = fmaf(x, x, ss); }
       ss = warp_sum(ss);
       if (lane == 0) head_ss[hh] = ss;
     }
@@ -311,8 +313,7 @@ __global__ void __launch_bounds__(256) qkv_post_span_kernel(QkvSpanArgs a) {
       c0 = 2 * half_rot + 2 * (pi - half_rot);
       c1 = c0 + 1;
     }
-    const float* src = row + (size_t)hh * dk;
-    float x0 = src[c0], x1 = src[c1];
+    float x0 = at(hh * dk + c0), x1 = at(hh * dk + c1);
     if (normed) {
       const float inv = a.whole ? (is_q ? inv_q : inv_k) : 1.0f / sqrtf(head_ss[hh] / (float)a.norm_dim + a.eps);
       const float* gain = is_q ? a.q_gain : a.k_gain;
@@ -331,11 +332,10 @@ __global__ void __launch_bounds__(256) qkv_post_span_kernel(QkvSpanArgs a) {
     dst[c1] = from_f32<T>(x1);
   }
   if (vdst != nullptr) {      // the values of the kv heads among this slice's heads (kv head g rides with head H + g)
-    const float* src = row + (size_t)(H + G) * dk;
     const int g0 = max(hh0, H) - H, g1 = hh1 - H;
     for (int i = g0 * dv + threadIdx.x; i < g1 * dv; i += nthreads) {
       const int g = i / dv, c = i - g * dv;
-      vdst[(size_t)g * kPageTokens * dv + c] = from_f32<T>(src[i]);
+      vdst[(size_t)g * kPageTokens * dv + c] = from_f32<T>(at((H + G) * dk + i));
     }
   }
 }
@@ -365,9 +365,18 @@ __global__ void __launch_bounds__(256) qkv_post_span_quad_kernel(QkvSpanArgs a) 
   __shared__ float scratch[33];
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int H = a.heads, G = a.kv_heads, dk = a.key_dim, dv = a.value_dim;
-  const size_t row_len = (size_t)(H + G) * dk + (size_t)G * dv;
-  const float* row = a.qkv + (size_t)t * row_len;
+  const float* row = a.qkv + (size_t)t * a.row_stride;
   const float4* row4 = reinterpret_cast<const float4*>(row);
+  const float4* bias4 = reinterpret_cast<const float4*>(a.bias);
+  auto at = [&](int i) { return a.bias ? row[i] + a.bias[i] : row[i]; };
+  auto at4 = [&](int i) {
+    float4 x = row4[i];
+    if (bias4) {
+      const float4 b = bias4[i];
+      x = make_float4(x.x + b.x, x.y + b.y, x.z + b.z, x.w + b.w);
+    }
+    return x;
+  };
   const bool normed = a.q_gain != nullptr;
   const int pos = a.tok_pos[t];
   const int page = a.k_pool != nullptr ? a.block_table[(size_t)a.tok_seq[t] * a.table_stride + pos / kPageTokens] : 0;
@@ -390,7 +399,7 @@ __global__ void __launch_bounds__(256) qkv_post_span_quad_kernel(QkvSpanArgs a) 
     si[i] = make_float2(0.f, 0.f);
     if (item < n_items) {
       const int hh = hh0 + item / quads, c = (item % quads) * 4;
-      v[i] = row4[hh0 * quads + item];
+      v[i] = at4(hh0 * quads + item);
       if (normed) {
         const bool is_q = hh < H;
         const float* gain = (is_q ? a.q_gain : a.k_gain) + (a.whole ? (is_q ? hh : hh - H) * dk : 0);
@@ -408,11 +417,11 @@ __global__ void __launch_bounds__(256) qkv_post_span_quad_kernel(QkvSpanArgs a) 
     kdst = (T*)a.k_pool + slot * dk;
     // the values of the kv heads among this slice's heads (kv head g rides with head H + g): nothing to wait for
     T* vdst = (T*)a.v_pool + slot * dv;
-    const float4* src4 = reinterpret_cast<const float4*>(row + (size_t)(H + G) * dk);
+    const int v0 = (H + G) * quads;
     const int vq = dv >> 2, g0 = max(hh0, H) - H, g1 = hh1 - H;
     for (int i = g0 * vq + threadIdx.x; i < g1 * vq; i += nthreads) {
       const int gh = i / vq, c = (i - gh * vq) * 4;
-      store4<T>(vdst + (size_t)gh * kPageTokens * dv + c, src4[i]);
+      store4<T>(vdst + (size_t)gh * kPageTokens * dv + c, at4(v0 + i));
     }
   }
   float inv_q = 1.0f, inv_k = 1.0f;
@@ -428,7 +437,7 @@ __global__ void __launch_bounds__(256) qkv_post_span_quad_kernel(QkvSpanArgs a) 
       }
     } else {
       for (int i = threadIdx.x; i < nq4 + nk4; i += nthreads) {      // the same values to the same threads as above
-        const float4 x = row4[i];
+        const float4 x = at4(i);
         const float ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w)));
         if (i < nq4) sq += ss; else sk += ss;
       }
@@ -439,9 +448,9 @@ __global__ void __launch_bounds__(256) qkv_post_span_quad_kernel(QkvSpanArgs a) 
     inv_k = 1.0f / sqrtf(sk / (float)(G * a.norm_dim) + a.eps);
   } else if (normed) {
     for (int hh = hh0 + warp; hh < hh1; hh += nwarps) {
-      const float* src = row + (size_t)hh * dk;
+      const int at0 = hh * dk;
       float ss = 0.0f;
-      for (int c = lane; c < dk; c += 32) ss = fmaf(src[c], src[c], ss);
+      for (int c = lane; c < dk; c += 32) { const float x = at(at0 + c); ss = fmaf(x, x, ss); }
       ss = warp_sum(ss);
       if (lane == 0) head_ss[hh] = ss;
     }
@@ -501,7 +510,7 @@ extern "C" int slb_qkv_post(const void* qkv, const float* bias, const float* q_g
   return fail(1, "qkv_post: unknown dtype %d", dtype);
 }
 
-extern "C" int slb_qkv_post_span(const float* qkv, const float* q_gain, const float* k_gain, const float* cos_table,
+extern "C" int slb_qkv_post_span(const float* qkv, long long row_stride, const float* bias, const float* q_gain, const float* k_gain, const float* cos_table,
                                  const float* sin_table, void* q_out, void* k_pool, void* v_pool, const int* tok_seq,
                                  const int* tok_pos, const int* block_table, int table_stride, int tokens, int heads,
                                  int kv_heads, int key_dim, int value_dim, int rot_dim, int neighbours, int whole, float eps,
@@ -516,6 +525,8 @@ extern "C" int slb_qkv_post_span(const float* qkv, const float* q_gain, const fl
   SLB_REQUIRE(k_pool == nullptr || (v_pool && block_table && table_stride > 0), "qkv_post_span: a cache write needs both pools and a block table");
   if (tokens == 0) return 0;
   QkvSpanArgs a;
+  SLB_REQUIRE(row_stride >= (long long)(heads + kv_heads) * key_dim + (long long)kv_heads * value_dim, "qkv_post_span: rows of %lld values are too short", row_stride);
+  a.row_stride = row_stride; a.bias = bias;
   a.qkv = qkv; a.q_gain = q_gain; a.k_gain = k_gain;
   a.cos_table = rot_dim > 0 ? cos_table : nullptr; a.sin_table = sin_table;
   a.q_out = q_out; a.k_pool = k_pool; a.v_pool = v_pool;
@@ -530,7 +541,7 @@ extern "C" int slb_qkv_post_span(const float* qkv, const float* q_gain, const fl
   int slices = (2 * sm_count() + tokens - 1) / tokens;
   slices = slices < 1 ? 1 : (slices > 16 ? 16 : slices);
   if (slices > heads + kv_heads) slices = heads + kv_heads;
-  const bool aligned = ((uintptr_t)qkv | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)q_out | (uintptr_t)k_pool |
+  const bool aligned = row_stride % 4 == 0 && ((uintptr_t)qkv | (uintptr_t)bias | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)q_out | (uintptr_t)k_pool |
                         (uintptr_t)v_pool) % 16 == 0 && ((uintptr_t)cos_table | (uintptr_t)sin_table) % 8 == 0;
   // many tokens: smaller blocks, so that all of them are resident at once (the float32 run keeps one block shape, so
   // that a row's sums are formed in the same order in every step)

@@ -294,7 +294,7 @@ struct GroupNormArgs {
   int head_width;
   const float* gate;     // [tokens, gate_stride] pre-activations of the silu gate
   long long gate_stride;
-  const float* gain;     // [gain_len]; channel c reads gain[c % gain_len]
+  const float* gain;     // [gain_len] or null (ones); channel c reads gain[c % gain_len]
   int gain_len;
   void* out;             // [tokens, inner] in the run dtype
   int tokens, inner, groups;
@@ -324,7 +324,8 @@ __global__ void __launch_bounds__(128) gated_group_norm_kernel(GroupNormArgs a) 
     float v = y[c];
     if (a.skip) v = fmaf(a.skip_gain[c / a.head_width], a.skip[(size_t)t * a.skip_stride + c], v);
     if (a.gate_first) v *= silu_f(gate[c]);
-    v = v * r * a.gain[c % a.gain_len];
+    v = v * r;
+    if (a.gain) v *= a.gain[c % a.gain_len];
     if (!a.gate_first) v *= silu_f(gate[c]);
     out[c] = from_f32<T>(v);
   }

@@ -53,6 +53,7 @@ class Model:
         if request is not None:
             self.embedding_entry = len(self.cache_requests)
             self.cache_requests.append(request)
+        self.reads_stream = any(getattr(layer, "reads_stream", False) for layer in self.layers)
         self.pass_mix = None            # the product W [x; x0] of schedule entries that mix the embedding into the stream
         self._programs: dict = {}       # per cache: the runs of the schedule prepared for the persistent kernel
         self.pass_rows = None           # [rows, hidden] float32: vectors that schedule entries add to the stream
@@ -118,6 +119,9 @@ class Model:
             self.embedding.forward(b, x, cache.view(self.embedding_entry, writes=True))
         else:
             self.embedding.forward(b, x)
+        b.rounded, b.rounded_ok = None, False
+        if self.reads_stream and self.ctx.dtype != torch.float32:      # layers without front norms read the stream in the run dtype
+            b.rounded = ws.take((b.T, self.hidden), self.ctx.dtype)
         xs = None
         if self.spec.streams > 1:           # several copies of the stream: all start as the embedding's output
             from ..kernels import ops
@@ -135,6 +139,8 @@ class Model:
                 i = self._run_fused(fused[i], x, b, ws)
                 continue
             e = schedule[i]
+            if e.mix_embedding or e.add_embedding or e.add_row >= 0:
+                b.rounded_ok = False
             if e.mix_embedding:          # x <- W [x; x0]
                 from ..kernels import ops
                 m = ws.mark()
@@ -152,7 +158,10 @@ class Model:
                 view["borrowed"] = cache.view(e.borrow, writes=False)
             following = self.layers[schedule[i + 1].layer] if i + 1 < len(schedule) and (i + 1) not in fused else None
             b.next_read = lead_weight_of(following)
-            self.layers[e.layer].forward(x if xs is None else xs, b, view, ws)
+            layer = self.layers[e.layer]
+            layer.forward(x if xs is None else xs, b, view, ws)
+            if not getattr(layer, "reads_stream", False):
+                b.rounded_ok = False        # it has written the stream alone
             if self.observe is not None:
                 if xs is not None:
                     ops.streams_sum(xs, x, b.stream)

@@ -153,11 +153,11 @@ _SIGNATURES = {
     "slb_gated_act": [P, P, I, I, I, I, F, F, P],
     "slb_layernorm": [P, P, P, P, P, I, P, I, I, F, P],
     "slb_softcap": [P, L, I, I, F, P],
-    "slb_qkv_post_span": [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P],
+    "slb_qkv_post_span": [P, L, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P],
     "slb_stream_inject": [P, P, P, I, I, P],
     "slb_pair_embed": [P, P, P, I, P, P, P, P, P, P, I, I, I, I, L, L, P, F, P, P],
     "slb_sinusoid_add": [P, P, P, I, I, P],
-    "slb_gated_norm_add": [P, P, P, L, P, P, I, I, F, P],
+    "slb_gated_norm_add": [P, P, P, L, P, P, I, I, F, P, F, F, P, P],
     "slb_stream_pair": [P, P, P, I, I, I, P],
     "slb_scale": [P, L, I, I, F, P, P],
     "slb_mingru": [P, L, P, P, P, P, P, P, P, I, I, I, I, P],
@@ -169,11 +169,11 @@ _SIGNATURES = {
     "slb_latent_query": [P, L, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P],
     "slb_latent_value": [P, P, P, P, P, L, I, P, I, I, I, I, I, P],
     "slb_latent_gate": [P, P, P, I, I, I, I, P],
-    "slb_moe_route": [P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P],
-    "slb_moe_experts_tc": [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, P, P],
+    "slb_moe_route": [P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P],
+    "slb_moe_experts_tc": [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, P, I, P, P],
     "slb_gemm_skinny_gated": [P, P, P, I, I, I, I, I, F, F, P, L, P, I, P],
     "slb_gemm_tc_gated": [P, P, P, I, I, I, I, I, F, F, P, P],
-    "slb_moe_experts": [P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, P],
+    "slb_moe_experts": [P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, I, I, P],
     "slb_attention_scored": [P, P, P, P, P, P, P, I, I, I, I, I, I, F, P, F, I, I, P, L, I, I, P],
     "slb_attention_tc_scored": [P, P, P, P, P, P, P, P, I, I, I, L, L, I, I, I, I, F, P, I, I, P, F, P],
     "slb_attention_prefill_scored": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, P, F, I, P],
@@ -184,6 +184,10 @@ _SIGNATURES = {
     "slb_step_decay": [P, L, P, P, P, P, I, I, P],
     "slb_channel_decay": [P, P, I, I, F, P],
     "slb_gated_group_norm": [P, P, L, P, I, P, L, P, I, P, I, I, I, I, F, I, P],
+    "slb_rotate_rows": [P, L, P, P, P, I, I, I, I, I, P],
+    "slb_delta_prep": [P, L, I, I, F, F, P, P, L, P, P, P, P, I, I, P],
+    "slb_delta_scan": [P, L, P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, P],
+    "slb_state_token": [P, L, P, L, P, L, P, L, P, P, P, L, P, P, P, P, P, I, I, P, P, P, P, I, I, I, I, I, F, F, F, I, P],
     "slb_unit_post": [P, L, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P],
     "slb_diff_combine": [P, P, L, P, I, I, I, F, F, F, I, I, P],
     "slb_streams_fill": [P, P, L, I, I, P],

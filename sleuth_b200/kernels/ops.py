@@ -168,10 +168,15 @@ def sinusoid_add(x, tok_pos, turns, stream=None) -> None:
     lib().call("slb_sinusoid_add", _p(x), _p(tok_pos), _p(turns), T, d, stream if stream is not None else current_stream())
 
 
-def gated_norm_add(x, y, g, bias, gain, eps: float, stream=None) -> None:
+def gated_norm_add(x, y, g, bias, gain, eps: float, stream=None, second=None, rounded=None) -> None:
     """x += rmsnorm(y * sigmoid(g + bias)) * gain, row by row in float32; without ``g``: x += rmsnorm(y) * gain. ``y`` may be
-    overwritten. ``g`` may be a view of a wider float32 matrix (unit column stride)."""
-    _cuda(x, y, bias, gain)
+    overwritten. ``g`` may be a view of a wider float32 matrix (unit column stride). ``second`` = (y2, s1, s2), not together
+    with ``g``: s1 * y + s2 * y2 stands for y. ``rounded``: a bfloat16 tensor of the stream's shape that receives the new rows."""
+    _cuda(x, y, bias, gain, rounded)
+    y2, s1, s2 = second if second is not None else (None, 1.0, 1.0)
+    _need(y2 is None or (g is None and y2.is_cuda and y2.is_contiguous() and y2.dtype == torch.float32 and y2.shape == x.shape),
+          "gated_norm_add: the second result is float32, of the stream's shape, and without a gate")
+    _need(rounded is None or (rounded.dtype == torch.bfloat16 and rounded.shape == x.shape), "gated_norm_add: the rounded rows")
     T, d = x.shape
     _need(x.dtype == torch.float32 and y.dtype == torch.float32 and y.shape == x.shape, "gated_norm_add: the stream and the sublayer's result are float32")
     _need(gain.dtype == torch.float32 and gain.numel() == d, "gated_norm_add: gain")
@@ -182,7 +187,7 @@ def gated_norm_add(x, y, g, bias, gain, eps: float, stream=None) -> None:
         stride = g.stride(0) if T > 1 else d
         _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == d), "gated_norm_add: bias")
     lib().call("slb_gated_norm_add", _p(x), _p(y), _p(g), stride, _p(bias) if g is not None else None, _p(gain), T, d, float(eps),
-               stream if stream is not None else current_stream())
+               _p(y2), float(s1), float(s2), _p(rounded), stream if stream is not None else current_stream())
 
 
 def stream_pair(a, b, out, stream=None) -> None:
@@ -254,18 +259,20 @@ def qkv_post(qkv, bias, q_gain, k_gain, cos, sin, q_out, k_pool, v_pool, tok_seq
 
 def qkv_post_span(qkv, q_gain, k_gain, cos, sin, q_out, k_pool, v_pool, tok_seq, tok_pos, block_table, heads: int,
                   kv_heads: int, key_dim: int, value_dim: int, rot_dim: int, neighbours: bool, whole: bool, eps: float,
-                  stream=None, norm_dim: int = 0) -> None:
+                  stream=None, norm_dim: int = 0, bias=None) -> None:
     """What follows separate q, k and v projections whose float32 results lie side by side in ``qkv``
     [T, heads * key_dim + kv_heads * key_dim + kv_heads * value_dim]: RMS norm of q and k (``whole``: over the whole
     projection with gains of that length; else per head with gains [key_dim]; no gains: none), rotation of each head's
     first ``rot_dim`` channels (``neighbours``: pairs (2i, 2i + 1); else (i, i + rot_dim / 2)), q into ``q_out``
     [T, heads, key_dim], k and v into the token's cache row (pools [pages, kv_heads, 64, key_dim | value_dim]).
     ``norm_dim``: how many channels of a head count in the norms' means, when the heads end in zero channels that only
-    pad them (0 = ``key_dim``)."""
-    _cuda(qkv, q_gain, k_gain, cos, sin, q_out, k_pool, v_pool, tok_seq, tok_pos, block_table)
+    pad them (0 = ``key_dim``). ``qkv`` may be a view of wider rows; ``bias``: float32 values added to the rows first."""
+    _cuda(bias, q_gain, k_gain, cos, sin, q_out, k_pool, v_pool, tok_seq, tok_pos, block_table)
     T = q_out.shape[0]
-    _need(qkv.dtype == torch.float32 and qkv.shape == (T, (heads + kv_heads) * key_dim + kv_heads * value_dim),
-          "qkv_post_span: the projections' float32 rows")
+    width = (heads + kv_heads) * key_dim + kv_heads * value_dim
+    _need(qkv.shape[0] == T, "qkv_post_span: the projections' float32 rows")
+    row_stride = _rows_f32(qkv, width, "qkv_post_span")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == width), "qkv_post_span: bias")
     _need(q_out.shape[1:] == (heads, key_dim) and q_out.dtype in DT, "qkv_post_span: q_out")
     n_q, n_k = (heads * key_dim, kv_heads * key_dim) if whole else (key_dim, key_dim)
     for g, n in ((q_gain, n_q), (k_gain, n_k)):
@@ -281,7 +288,7 @@ def qkv_post_span(qkv, q_gain, k_gain, cos, sin, q_out, k_pool, v_pool, tok_seq,
         _need(block_table.dtype == torch.int32 and block_table.dim() == 2, "qkv_post_span: block table")
         stride = block_table.shape[1]
     _need(tok_seq.dtype == torch.int32 and tok_pos.dtype == torch.int32, "qkv_post_span: token tables are int32")
-    lib().call("slb_qkv_post_span", _p(qkv), _p(q_gain), _p(k_gain), _p(cos), _p(sin), _p(q_out), _p(k_pool), _p(v_pool),
+    lib().call("slb_qkv_post_span", qkv.data_ptr(), row_stride, _p(bias), _p(q_gain), _p(k_gain), _p(cos), _p(sin), _p(q_out), _p(k_pool), _p(v_pool),
                _p(tok_seq), _p(tok_pos), _p(block_table), stride, T, heads, kv_heads, key_dim, value_dim, rot_dim,
                1 if neighbours else 0, 1 if whole else 0, float(eps), int(norm_dim), DT[q_out.dtype],
                stream if stream is not None else current_stream())
@@ -1143,7 +1150,7 @@ MOE_FEW_PAIRS = 64      # up to this many (token, choice) pairs ``moe_experts`` 
 
 def moe_route(h, w_router, bias, choice, weight, rank, counts, place, order, top: int, stream=None, logits=None,
               tiles=None, layout: bool = True, scoring: str = "softmax_top", groups: int = 1, keep: int = 1,
-              scale: float = 1.0, logits_ready: bool = False, pick_bias=None) -> None:
+              scale: float = 1.0, logits_ready: bool = False, pick_bias=None, identity: int = 0) -> None:
     """Router logits in float32, then the choice. ``scoring="softmax_top"``: the ``top`` largest logits, weights =
     softmax over those. ``scoring="sigmoid"``: scores = sigmoid(logits); the experts form ``groups`` equal groups of
     neighbours, a group scores the sum of its two largest scores, only experts of the ``keep`` best groups can be
@@ -1155,6 +1162,7 @@ def moe_route(h, w_router, bias, choice, weight, rank, counts, place, order, top
     [T * top] (the pair at each row). choice, rank int32 [T * top]; weight float32 [T * top]. ``logits``: float32
     scratch [T, experts]; with it, steps of many tokens form their logits 32 tokens at a time (the same sums, k
     ascending). ``logits_ready``: ``logits`` holds the router's logits already (a product formed them, without the bias, which is added here).
+    ``identity``: the last so many of the router's experts have no matrices (``tiles`` then holds none of their pairs).
     ``layout=False`` leaves counts, place and order unwritten: ``moe_experts`` with ``choice`` does not read
     them for steps of at most ``MOE_FEW_PAIRS`` pairs."""
     _cuda(h, w_router, bias, choice, weight, rank, counts, place, order, logits, tiles, pick_bias)
@@ -1172,16 +1180,18 @@ def moe_route(h, w_router, bias, choice, weight, rank, counts, place, order, top
     _need(logits is None or (logits.dtype == torch.float32 and logits.numel() >= T * E), "moe_route: scratch for the logits")
     _need(tiles is None or (tiles.dtype == torch.int32 and tiles.numel() >= moe_tile_words(T, top, E)), "moe_route: row-tile table")
     lib().call("slb_moe_route", _p(h), _p(w_router), _p(bias), _p(pick_bias), _p(choice), _p(weight), _p(rank), _p(counts), _p(place),
-               _p(order), _p(logits), _p(tiles), 1 if layout else 0, T, d, E, int(top), ROUTE_SCORINGS[scoring], int(groups),
+               _p(order), _p(logits), _p(tiles), 1 if layout else 0, T, d, E, int(identity), int(top), ROUTE_SCORINGS[scoring], int(groups),
                int(keep), float(scale), 1 if logits_ready else 0, DT[h.dtype], stream if stream is not None else current_stream())
 
 
 def moe_experts(h, w_gate_up, w_down, counts, order, weight, act, y, x, top: int, activation: str = "silu",
-                stream=None, choice=None, place=None, limit: float = 0.0, alpha: float = 1.0, extra=None) -> None:
+                stream=None, choice=None, place=None, limit: float = 0.0, alpha: float = 1.0, extra=None, identity: int = 0,
+                store: bool = False) -> None:
     """x[t] += sum over the token's choices of weight * down_e(f(gate_e h) * (up_e h)). w_gate_up [experts, 2 * ff, d]
     (gate rows, then up rows), w_down [experts, d, ff]; act [T * top, ff] and y [T * top, d] float32 are scratch.
     With ``choice`` and ``place`` (from ``moe_route``) a step of few pairs runs a warp per output instead of tiles, and then
-    adds the rows of ``extra`` (float32, the stream's shape) as well, if given."""
+    adds the rows of ``extra`` (float32, the stream's shape) as well, if given. ``identity``: so many experts behind the ones
+    with matrices may be among the choices; they return h. ``store``: x = the sum instead of x += the sum."""
     _cuda(h, w_gate_up, w_down, counts, order, weight, act, y, x, choice, place, extra)
     _need(extra is None or (extra.dtype == torch.float32 and extra.shape == x.shape and h.shape[0] * top <= MOE_FEW_PAIRS),
           "moe_experts: further rows go with steps of few pairs")
@@ -1196,16 +1206,17 @@ def moe_experts(h, w_gate_up, w_down, counts, order, weight, act, y, x, top: int
     _need(x.shape == (T, d) and x.dtype == torch.float32, "moe_experts: the stream")
     _need(activation in ACTIVATIONS, f"moe_experts: activation {activation!r}")
     lib().call("slb_moe_experts", _p(h), _p(w_gate_up), _p(w_down), _p(counts), _p(order), _p(choice), _p(place), _p(weight), _p(act), _p(y),
-               _p(x), _p(extra), T, d, ff, E, int(top), ACTIVATIONS[activation], float(limit), float(alpha), DT[h.dtype],
-               stream if stream is not None else current_stream())
+               _p(x), _p(extra), T, d, ff, E, int(top), ACTIVATIONS[activation], float(limit), float(alpha), int(identity),
+               1 if store else 0, DT[h.dtype], stream if stream is not None else current_stream())
 
 
 def moe_experts_tc(h, w_gate_up, w_down, order, place, weight, tiles, xs, act, y, x, top: int, stream=None,
-                   activation: str = "silu", limit: float = 0.0, alpha: float = 1.0) -> None:
+                   activation: str = "silu", limit: float = 0.0, alpha: float = 1.0, choice=None, store: bool = False) -> None:
     """The same sum as ``moe_experts`` for steps of many pairs in bfloat16: the tokens' rows gathered into the
     expert order (``xs`` [T * top, d]) and both products as grouped tcgen05 products over the row tiles that
-    ``moe_route`` wrote into ``tiles``; ``y`` [T * top, d] float32 comes out in the expert order."""
-    _cuda(h, w_gate_up, w_down, order, place, weight, tiles, xs, act, y, x)
+    ``moe_route`` wrote into ``tiles``; ``y`` [T * top, d] float32 comes out in the expert order. ``choice``: the router's
+    choices, needed when identity experts (numbers from ``w_down.shape[0]`` on) are among them."""
+    _cuda(h, w_gate_up, w_down, order, place, weight, tiles, xs, act, y, x, choice)
     T, d = h.shape
     E, ff2, _ = w_gate_up.shape
     ff = ff2 // 2
@@ -1218,7 +1229,7 @@ def moe_experts_tc(h, w_gate_up, w_down, order, place, weight, tiles, xs, act, y
     _need(tiles.dtype == torch.int32 and tiles.numel() >= moe_tile_words(T, top, E), "moe_experts_tc: row-tile table")
     lib().call("slb_moe_experts_tc", _p(h), _p(w_gate_up), _p(w_down), _p(order), _p(place), _p(weight), _p(tiles), _p(xs),
                _p(act), _p(y), _p(x), T, d, ff, E, int(top), ACTIVATIONS[activation], float(limit), float(alpha),
-               _p(_tc_status(h.device)), stream if stream is not None else current_stream())
+               _p(choice), 1 if store else 0, _p(_tc_status(h.device)), stream if stream is not None else current_stream())
 
 
 # ---- other score rules, short convolutions, recurrences with a matrix state, several copies of the stream ----
@@ -1326,20 +1337,99 @@ def channel_decay(z, bias, tau: float, stream=None) -> None:
     lib().call("slb_channel_decay", _p(z), _p(bias), T, C, float(tau), _st(stream))
 
 
+# ---- the gated delta rule, linear attention with a fixed decay (csrc/delta_rule.cu) ----
+
+def rotate_rows(rows, cos, sin, tok_pos, units: int, dim: int, rot: int, neighbours: bool = False, stream=None) -> None:
+    """In place: the first ``rot`` channels of each of a row's first ``units`` units of ``dim`` values turn in pairs by the
+    token's position (``neighbours``: channels 2i and 2i + 1, else i and i + rot / 2). ``rows``: float32, possibly a view."""
+    _cuda(cos, sin, tok_pos)
+    stride = _rows_f32(rows, units * dim, "rotate_rows")
+    _need(rot == 0 or (cos.dtype == torch.float32 and cos.shape[1] == rot // 2 and sin.shape == cos.shape), "rotate_rows: tables")
+    _need(tok_pos.dtype == torch.int32 and tok_pos.numel() >= rows.shape[0], "rotate_rows: positions")
+    lib().call("slb_rotate_rows", rows.data_ptr(), stride, _p(cos), _p(sin), _p(tok_pos), rows.shape[0], int(units), int(dim), int(rot),
+               1 if neighbours else 0, _st(stream))
+
+
+def delta_prep(rows, raw_beta, raw_step, dt_bias, a_log, beta, log_decay, groups: int, dim: int, q_scale: float, unit_eps: float,
+               stream=None) -> None:
+    """In place: the ``groups`` query units and then the ``groups`` key units at the start of each float32 row become x / sqrt(sum x^2
+    + unit_eps), queries times ``q_scale``. beta [T, H] = sigmoid(raw_beta), log_decay [T, H] = -exp(a_log) softplus(raw_step +
+    dt_bias); the raw values are rows of H (views of one wider matrix)."""
+    _cuda(dt_bias, a_log, beta, log_decay)
+    T, H = beta.shape
+    stride = _rows_f32(rows, 2 * groups * dim, "delta_prep")
+    rs = _rows_f32(raw_beta, H, "delta_prep strengths")
+    _need(_rows_f32(raw_step, H, "delta_prep steps") == rs and rows.shape[0] == T and log_decay.shape == (T, H), "delta_prep: shapes disagree")
+    _need(all(t.dtype == torch.float32 for t in (dt_bias, a_log, beta, log_decay)) and dt_bias.numel() == a_log.numel() == H, "delta_prep: float32, one value a head")
+    lib().call("slb_delta_prep", rows.data_ptr(), stride, int(groups), int(dim), float(q_scale), float(unit_eps), raw_beta.data_ptr(),
+               raw_step.data_ptr(), rs, _p(dt_bias), _p(a_log), _p(beta), _p(log_decay), T, H, _st(stream))
+
+
+def _state_ok(state, heads: int, groups: int, what: str):
+    _cuda(state)
+    _need(state.dtype == torch.float32 and state.dim() == 4 and state.shape[1] == heads and heads % groups == 0, f"{what}: the state is float32 [slots, heads, N, P]")
+    return int(state.shape[2]), int(state.shape[3])
+
+
+def delta_scan(q, k, v, log_decay, beta, state, slots, seq_start, out, heads: int, groups: int, stream=None) -> None:
+    """The gated delta rule over each sequence's tokens of the step, from and back into ``state`` float32 [slots, heads, N, P]:
+    S <- exp(log_decay) S, u = beta (v - S^T k), S <- S + k u^T, out = S^T q. q, k: float32 rows of groups * N values (head h
+    reads group h // (heads / groups)); v: rows of heads * P; log_decay, beta, [T, heads]; out float32 [T, heads * P]."""
+    N, P = _state_ok(state, heads, groups, "delta_scan")
+    _cuda(log_decay, beta, slots, seq_start, out)
+    T = out.shape[0]
+    _need(out.dtype == torch.float32 and out.shape == (T, heads * P) and log_decay.shape == beta.shape == (T, heads), "delta_scan: shapes disagree")
+    _need(slots.dtype == torch.int32 and seq_start.dtype == torch.int32 and seq_start.numel() >= slots.numel() + 1, "delta_scan: tables")
+    lib().call("slb_delta_scan", q.data_ptr(), _rows_f32(q, groups * N, "delta_scan q"), k.data_ptr(), _rows_f32(k, groups * N, "delta_scan k"),
+               v.data_ptr(), _rows_f32(v, heads * P, "delta_scan v"), _p(log_decay), _p(beta), _p(state), _p(slots), _p(seq_start), _p(out),
+               slots.numel(), heads, groups, N, P, _st(stream))
+
+
+def state_token_supported(N: int, P: int) -> bool:
+    """Whether ``state_token`` takes heads of N key and P value channels."""
+    return lib().dll.slb_state_token_supported(int(N), int(P)) != 0
+
+
+def state_token(q, k, v, gate, state, slots, out, heads: int, groups: int, eps: float, gain=None, q_scale: float = 1.0, decay=None,
+                raw_beta=None, raw_step=None, dt_bias=None, a_log=None, unit_eps: float = 0.0, cos=None, sin=None, tok_pos=None,
+                rot: int = 0, neighbours: bool = False, stream=None) -> None:
+    """A step of one token a sequence of a recurrence with a matrix state, from the projections' float32 rows to what the output
+    product reads: out[i, h] = o / rms(o) * gain * silu(gate), o = S^T q after the token's update of ``state``. With ``decay``
+    [heads]: q and k turn (``rot`` channels, tables, ``tok_pos``), S <- decay S + k v^T. Without: q and k become unit vectors
+    (``unit_eps``) and the gated delta rule with the token's own strength and decay runs (``raw_beta``, ``raw_step``, ``dt_bias``,
+    ``a_log`` as in ``delta_prep``). ``q_scale`` multiplies q. ``gain`` [P] or None."""
+    N, P = _state_ok(state, heads, groups, "state_token")
+    _cuda(slots, out, gain, decay, dt_bias, a_log, cos, sin, tok_pos)
+    n = slots.numel()
+    _need(out.shape == (n, heads * P) and out.dtype in DT and q.shape[0] == n, "state_token: one row a sequence")
+    _need(slots.dtype == torch.int32 and (decay is None or (decay.dtype == torch.float32 and decay.numel() == heads)), "state_token: tables")
+    _need(gain is None or (gain.dtype == torch.float32 and gain.numel() == P), "state_token: gain")
+    _need(rot == 0 or (cos.dtype == torch.float32 and cos.shape[1] == rot // 2 and sin.shape == cos.shape and tok_pos.dtype == torch.int32), "state_token: rotation")
+    rs = 0
+    if decay is None:
+        rs = _rows_f32(raw_beta, heads, "state_token strengths")
+        _need(_rows_f32(raw_step, heads, "state_token steps") == rs and dt_bias.numel() == a_log.numel() == heads, "state_token: one value a head")
+    lib().call("slb_state_token", q.data_ptr(), _rows_f32(q, groups * N, "state_token q"), k.data_ptr(), _rows_f32(k, groups * N, "state_token k"),
+               v.data_ptr(), _rows_f32(v, heads * P, "state_token v"), gate.data_ptr(), _rows_f32(gate, heads * P, "state_token gate"), _p(decay),
+               _p(raw_beta), _p(raw_step), rs, _p(dt_bias), _p(a_log), _p(cos), _p(sin), _p(tok_pos), int(rot), 1 if neighbours else 0,
+               _p(state), _p(slots), _p(gain), _p(out), n, heads, groups, N, P, float(q_scale), float(unit_eps), float(eps), DT[out.dtype],
+               _st(stream))
+
+
 def gated_group_norm(y, gate, gain, out, groups: int, eps: float, gate_first: bool, skip=None, skip_gain=None,
                      head_width: int = 1, stream=None) -> None:
     """Rows of ``y`` float32 [T, inner] in ``groups`` equal parts, each divided by its root mean square, times
-    gain[c % len(gain)]; silu(gate) multiplies the row before the norm (``gate_first``) or after it. With ``skip``:
+    gain[c % len(gain)] (``gain`` None: ones); silu(gate) multiplies the row before the norm (``gate_first``) or after it. With ``skip``:
     skip_gain[c // head_width] * skip[t, c] is added to y first. ``out`` [T, inner] in the run dtype."""
     _cuda(y, gain, out, skip_gain)
     T, inner = y.shape
     gs = _rows_f32(gate, inner, "gated_group_norm gate")
     ks = _rows_f32(skip, inner, "gated_group_norm skip") if skip is not None else 0
-    _need(y.dtype == torch.float32 and gain.dtype == torch.float32 and out.shape == (T, inner) and out.dtype in DT and inner % groups == 0,
+    _need(y.dtype == torch.float32 and (gain is None or gain.dtype == torch.float32) and out.shape == (T, inner) and out.dtype in DT and inner % groups == 0,
           "gated_group_norm: shapes or dtypes")
     _need(skip is None or (skip_gain is not None and skip_gain.dtype == torch.float32 and skip_gain.numel() * head_width == inner),
           "gated_group_norm: the skip term's gains")
-    lib().call("slb_gated_group_norm", _p(y), _p(skip), ks, _p(skip_gain), int(head_width), _p(gate), gs, _p(gain), gain.numel(),
+    lib().call("slb_gated_group_norm", _p(y), _p(skip), ks, _p(skip_gain), int(head_width), _p(gate), gs, _p(gain), 1 if gain is None else gain.numel(),
                _p(out), T, inner, int(groups), 1 if gate_first else 0, float(eps), DT[out.dtype], _st(stream))
 
 

@@ -13,8 +13,11 @@ application wrote.
 Options that another design may set (``AttentionSpec``): values of another width than the keys (``value_dim``), one
 RMSNorm over the whole q projection and one over the whole k projection instead of one per head
 (``qk_norm_span="projection"``), rotation of neighbouring channels (the position's ``pairing``), and a learned sink per
-head in the softmax denominator (``sinks``). Any of the first three sends a step through the *wide* form: the stacked
-projection with a float32 result, ``qkv_post_span`` (norms, rotation, cache write) and the attention kernel.
+head in the softmax denominator (``sinks``, or ``unit_sink``: one whose score is 0). ``chunk`` limits a query to the keys of its
+own chunk of positions; ``gate`` multiplies the heads' outputs by sigmoid(W_g h). Values of another width, whole-projection
+norms, neighbouring channels and a gate send a step through the *wide* form: the stacked projection (the gate's rows behind
+q, k and v) with a float32 result, ``qkv_post_span`` (biases, norms, rotation, cache write), the attention kernel, and the
+gate in place.
 """
 
 from __future__ import annotations
@@ -26,8 +29,7 @@ import torch
 
 from ..cache.paged import KVRequest
 from ..kernels import ops
-from .base import BuildContext, ParamDecl, Part, build_position, register_mixer
-from .base import Normed
+from .base import BuildContext, Normed, ParamDecl, Part, build_position, register_mixer, result_target
 from .linear import Linear, use_tc
 from .spec import AttentionSpec
 
@@ -46,6 +48,7 @@ def use_tc_attention(heads: int, kv_heads: int, head_dim: int, dtype, max_count:
 
 class GQAAttention(Part):
     accepts_normed = True
+    stores_result = True
 
     def __init__(self, spec: AttentionSpec, ctx: BuildContext):
         if spec.heads % spec.kv_heads:
@@ -65,7 +68,13 @@ class GQAAttention(Part):
             raise ValueError(f"value_dim {self.value_dim} is not supported: at most 256")
         self.whole_norm = spec.qk_norm and spec.qk_norm_span == "projection"
         # the wide form: what the per-head kernels (equal widths, per-head norms, halves turned together) do not take
-        self.wide = (self.value_dim != spec.head_dim or self.whole_norm or getattr(self.position, "neighbours", False))
+        if spec.gate not in ("none", "channel"):
+            raise ValueError(f"attention: gate {spec.gate!r} is not 'none' or 'channel'")
+        if spec.chunk < 0 or spec.chunk and spec.window or spec.sinks and spec.unit_sink:
+            raise ValueError(f"attention: chunk {spec.chunk} and window {spec.window} (one of them), learned sinks or a unit sink (one of them)")
+        self.reach = -spec.chunk if spec.chunk else spec.window         # the signed window of the cache and the kernels
+        self.gated = spec.gate == "channel"
+        self.wide = (self.value_dim != spec.head_dim or self.whole_norm or getattr(self.position, "neighbours", False) or self.gated)
         # The tensor-core attention kernels take keys and values of one width, 64 or 128. A bfloat16 run of the wide form
         # with other widths up to 128 gives every head zero channels at its end until it has such a width (zero rows in
         # the projections, zero columns in the output matrix): scores and outputs are the same numbers, the cache rows are
@@ -73,9 +82,9 @@ class GQAAttention(Part):
         self.key_run, self.value_run = spec.head_dim, self.value_dim
         if self.wide and ctx.dtype == torch.bfloat16 and max(spec.head_dim, self.value_dim) <= 128:
             self.key_run = self.value_run = 64 if max(spec.head_dim, self.value_dim) <= 64 else 128
-        if self.wide and (spec.qkv_bias or spec.reads_shared_kv):
-            raise ValueError("attention: biases and a borrowed cache entry are not built for values of another width, "
-                             "whole-projection norms or neighbour pairing")
+        if self.wide and spec.reads_shared_kv:
+            raise ValueError("attention: a borrowed cache entry is not built for values of another width, whole-projection "
+                             "norms, neighbour pairing or a gate")
 
     # ---- weights ----
     def declare(self):
@@ -89,22 +98,26 @@ class GQAAttention(Part):
             d["q_proj.bias"] = ParamDecl((s.heads * s.head_dim,), "vector")
             if not s.reads_shared_kv:
                 d["k_proj.bias"] = ParamDecl((s.kv_heads * s.head_dim,), "vector")
-                d["v_proj.bias"] = ParamDecl((s.kv_heads * s.head_dim,), "vector")
+                d["v_proj.bias"] = ParamDecl((s.kv_heads * self.value_dim,), "vector")
         if s.qk_norm:
             d["q_norm.weight"] = ParamDecl(((s.heads if self.whole_norm else 1) * s.head_dim,), "vector", init="gain")
             if not s.reads_shared_kv:
                 d["k_norm.weight"] = ParamDecl(((s.kv_heads if self.whole_norm else 1) * s.head_dim,), "vector", init="gain")
         if s.sinks:
             d["sinks"] = ParamDecl((s.heads,), "vector")
+        if self.gated:
+            d["g_proj.weight"] = ParamDecl((s.heads * self.value_dim, s.hidden))
         return d
 
     def bind(self, t):
         s = self.spec
         names = ["q_proj"] if s.reads_shared_kv else ["q_proj", "k_proj", "v_proj"]
+        if s.unit_sink:
+            self.sinks = torch.zeros(s.heads, dtype=torch.float32, device=t["q_proj.weight"].device)
         if (self.key_run, self.value_run) != (s.head_dim, self.value_dim):
             self._bind_padded(t)
             return
-        self.qkv = Linear(torch.cat([t[n + ".weight"] for n in names], dim=0), self.ctx.dtype)
+        self.qkv = Linear(torch.cat([t[n + ".weight"] for n in names + (["g_proj"] if self.gated else [])], dim=0), self.ctx.dtype)
         self.o = Linear(t["o_proj.weight"], self.ctx.dtype)
         if s.qkv_bias:
             self.bias = torch.cat([t[n + ".bias"] for n in names]).contiguous()
@@ -127,7 +140,12 @@ class GQAAttention(Part):
         q = heads_padded(t["q_proj.weight"], s.heads, s.head_dim, self.key_run)
         k = heads_padded(t["k_proj.weight"], s.kv_heads, s.head_dim, self.key_run)
         v = heads_padded(t["v_proj.weight"], s.kv_heads, self.value_dim, self.value_run)
-        self.qkv = Linear(torch.cat([q, k, v], dim=0), dt)
+        g = [heads_padded(t["g_proj.weight"], s.heads, self.value_dim, self.value_run)] if self.gated else []
+        self.qkv = Linear(torch.cat([q, k, v, *g], dim=0), dt)
+        if s.qkv_bias:
+            self.bias = torch.cat([heads_padded(t["q_proj.bias"], s.heads, s.head_dim, self.key_run),
+                                   heads_padded(t["k_proj.bias"], s.kv_heads, s.head_dim, self.key_run),
+                                   heads_padded(t["v_proj.bias"], s.kv_heads, self.value_dim, self.value_run)]).to(torch.float32).contiguous()
         o = t["o_proj.weight"]                        # [hidden, heads * value_dim]: zero columns behind each head
         self.o = Linear(heads_padded(o.t().contiguous(), s.heads, self.value_dim, self.value_run).t().contiguous(), dt)
         if s.qk_norm:
@@ -142,7 +160,7 @@ class GQAAttention(Part):
 
     def cache_request(self):
         s = self.spec
-        return KVRequest(s.kv_heads, self.key_run, s.window, 0 if self.value_run == self.key_run else self.value_run)
+        return KVRequest(s.kv_heads, self.key_run, self.reach, 0 if self.value_run == self.key_run else self.value_run)
 
     # ---- one step ----
     def _attend(self, q, y, b, view, table, ws):
@@ -174,7 +192,7 @@ class GQAAttention(Part):
     def fused_decode(self):
         s = self.spec
         rot = self.position.rot_dim
-        if (self.wide or self.sinks is not None or self.ctx.dtype != torch.bfloat16 or self.qkv is None or s.reads_shared_kv or s.head_dim not in (64, 128)
+        if (self.wide or self.sinks is not None or s.chunk or self.ctx.dtype != torch.bfloat16 or self.qkv is None or s.reads_shared_kv or s.head_dim not in (64, 128)
                 or rot not in (0, s.head_dim) or s.heads // s.kv_heads > 8 or s.hidden % 128
                 or (s.qk_norm and (self.q_gain is None or self.k_gain is None))):
             return None
@@ -211,7 +229,7 @@ class GQAAttention(Part):
                             b.stream)
             y = ws.take((T, s.heads * s.head_dim), self.ctx.dtype)
             self._attend(q, y, b, view, table, ws)
-            self.o.forward(y, into=x, ws=ws, stream=b.stream)
+            self.o.forward(y, ws=ws, stream=b.stream, **result_target(b, x))
             ws.release(mark)
             return
         single = flash and b.max_count == 1 and rot in (0, s.head_dim) and (writes or s.reads_shared_kv)
@@ -231,7 +249,7 @@ class GQAAttention(Part):
                                  qkv_kv_heads=kvh, bias=self.bias, q_gain=self.q_gain, k_gain=self.k_gain,
                                  cos=cos if rot else None, sin=sin if rot else None, eps=s.qk_norm_eps,
                                  next_read=self.o.weight, sinks=self.sinks)
-            self.o.forward(y, into=x, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None))
+            self.o.forward(y, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None), **result_target(b, x))
             ws.release(mark)
             return
         q = ws.take((T, s.heads, s.head_dim), self.ctx.dtype)
@@ -239,7 +257,7 @@ class GQAAttention(Part):
                      view.k_pool if writes else None, view.v_pool if writes else None,
                      b.tok_seq, b.tok_pos, table, s.heads, kvh, s.head_dim, rot, s.qk_norm_eps, b.stream)
         self._attend(q, y, b, view, table, ws)
-        self.o.forward(y, into=x, ws=ws, stream=b.stream)
+        self.o.forward(y, ws=ws, stream=b.stream, **result_target(b, x))
         ws.release(mark)
 
 
@@ -249,15 +267,18 @@ class GQAAttention(Part):
         s = self.spec
         T = h.shape[0]
         qkv = self.qkv.forward(h, ws=ws, stream=b.stream, out_dtype=torch.float32)
+        n_qkv = (s.heads + s.kv_heads) * self.key_run + s.kv_heads * self.value_run
         q = ws.take((T, s.heads, self.key_run), self.ctx.dtype)
         writes = view.writes
         ops.qkv_post_span(qkv, self.q_gain, self.k_gain, cos if rot else None, sin if rot else None, q,
                           view.k_pool if writes else None, view.v_pool if writes else None, b.tok_seq, b.tok_pos, table,
                           s.heads, s.kv_heads, self.key_run, self.value_run, rot, self.position.neighbours, self.whole_norm,
-                          s.qk_norm_eps, b.stream, norm_dim=s.head_dim)
+                          s.qk_norm_eps, b.stream, norm_dim=s.head_dim, bias=self.bias)
         y = ws.take((T, s.heads * self.value_run), self.ctx.dtype)
         self._attend(q, y, b, view, table, ws)
-        self.o.forward(y, into=x, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None))
+        if self.gated:
+            ops.sigmoid_gate(y, qkv[:, n_qkv:], b.stream)
+        self.o.forward(y, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None), **result_target(b, x))
 
 
 register_mixer("gqa_attention", GQAAttention)

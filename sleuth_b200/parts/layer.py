@@ -6,7 +6,8 @@
 ``prenorm``: x += mixer(norm1(x)); x += ffn(norm2(x)) (sleuth/forge/model/transformer.py:78,87-88,96,99); the feed-forward
 may be absent.
 ``sandwich``: a norm in front of and behind each sublayer, x += post1(mixer(norm1(x))), then x += post2(ffn(norm2(x)));
-with ``gated`` each sublayer's result is multiplied by sigmoid(W h + b) of the sublayer's own input h before its norm.
+with ``gated`` each sublayer's result is multiplied by sigmoid(W h + b) of the sublayer's own input h before its norm;
+without a front norm a sublayer reads the stream itself (rounded to the run dtype by the kernel that last wrote it).
 
 The layer owns the residual arrangement only; the parts it is given decide everything else. The sum
 itself is a float32 accumulation into the stream, done by the last product of the mixer or ffn.
@@ -179,15 +180,22 @@ class SandwichLayer(Part):
 
     def __init__(self, spec: LayerSpec, ctx: BuildContext):
         self.ctx, self.gated = ctx, bool(spec.gated)
-        self.hidden = spec.norm1.dim
-        self.norm1 = build_norm(spec.norm1, ctx)
+        self.hidden = spec.post1.dim
+        self.reads_stream = spec.norm1 is None
+        if self.reads_stream and spec.gated:
+            raise ValueError("sandwich layer: a gate goes with a front norm")
+        self.norm1 = build_norm(spec.norm1, ctx) if not self.reads_stream else None
         self.mixer = build_mixer(spec.mixer, ctx)
         self.post1 = build_norm(spec.post1, ctx)
         self.ffn = build_ffn(spec.ffn, ctx) if spec.ffn is not None else None
         self.children = {"norm1": self.norm1, "mixer": self.mixer, "post1": self.post1}
+        self.norm2 = None
         if self.ffn is not None:
-            self.norm2, self.post2 = build_norm(spec.norm2, ctx), build_norm(spec.post2, ctx)
+            if (spec.norm2 is None) != self.reads_stream:
+                raise ValueError("sandwich layer: both sublayers have a front norm, or neither has")
+            self.norm2, self.post2 = build_norm(spec.norm2, ctx) if not self.reads_stream else None, build_norm(spec.post2, ctx)
             self.children.update({"norm2": self.norm2, "ffn": self.ffn, "post2": self.post2})
+        self.children = {name: part for name, part in self.children.items() if part is not None}
         for name, part in self.children.items():
             if name.startswith("post") and not getattr(part, "fusable", False):
                 raise ValueError("sandwich layer: the norm behind a sublayer must be an RMS norm")
@@ -232,27 +240,54 @@ class SandwichLayer(Part):
     def _sublayer(self, norm, part, post, gate, bias, x, b, ws, view, after, rides):
         mark = ws.mark()
         y = ws.take(x.shape, torch.float32)
-        n = Normed(norm, x, ws, b.stream, self.ctx.dtype)
-        # the part alone reads the normed rows when the gate rides with it: it may then normalise inside its first product
-        h = n if rides and part.accepts_normed else n.tensor()
+        rounded = None
+        if norm is None:                # the sublayer reads the stream itself
+            h, rounded = self._stream_rows(x, b, ws)
+        else:
+            n = Normed(norm, x, ws, b.stream, self.ctx.dtype)
+            # the part alone reads the normed rows when the gate rides with it: it may then normalise inside its first product
+            h = n if rides and part.accepts_normed else n.tensor()
         if getattr(part, "stores_result", False):
             b.store_first = True        # the part's first delivery into y is a store
         else:
             y.zero_()
         b.rider = None
+        b.pair_wanted, b.pair = gate is None and not rides, None        # two results side by side may be joined by the closing kernel
         b.next_read = gate.weight if gate is not None else after
         if part is self.mixer:
             part.forward(h, y, b, view, ws)
         else:
             part.forward(h, y, b, ws)
+        b.pair_wanted, pair = False, b.pair
+        if pair is not None:            # views into the part's scratch memory, like a rider: the closing kernel comes next
+            b.pair, b.store_first = None, False
+            first, second, s1, s2 = pair
+            ops.gated_norm_add(x, first, None, None, post.weight, post.eps, b.stream, second=(second, s1, s2), rounded=rounded)
+            ws.release(mark)
+            return
         if getattr(b, "store_first", False):
             raise RuntimeError(f"{type(part).__name__} says it stores its result and did not")
         if rides:
             g = b.rider         # a view into the part's scratch memory: nothing takes scratch before the next kernel reads it
         else:
             g = gate.forward(n.tensor(), ws=ws, stream=b.stream, out_dtype=torch.float32, next_read=after) if gate is not None else None
-        ops.gated_norm_add(x, y, g, bias if g is not None else None, post.weight, post.eps, b.stream)
+        ops.gated_norm_add(x, y, g, bias if g is not None else None, post.weight, post.eps, b.stream, rounded=rounded)
         ws.release(mark)
+
+    def _stream_rows(self, x, b, ws):
+        """(the stream in the run dtype, where the closing kernel leaves its new rows in that dtype or None). The model keeps
+        one buffer of such rows for all its layers; ``b.rounded_ok`` says whether it holds the stream as it is now."""
+        if x.dtype == self.ctx.dtype:
+            return x, None
+        rows = getattr(b, "rounded", None)
+        if rows is None:                # a layer on its own
+            rows = ws.take(x.shape, self.ctx.dtype)
+            rows.copy_(x)
+            return rows, None
+        if not b.rounded_ok:
+            rows.copy_(x)
+        b.rounded_ok = True             # and stays so: the closing kernel writes both
+        return rows, rows
 
 
 class HyperLayer(Part):

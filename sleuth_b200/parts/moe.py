@@ -4,7 +4,8 @@ Router logits z = W_r h + b in float32 (W_r and b are kept in float32; h is the 
 dtype). A token uses the ``top`` experts with the largest logits, weighted by the softmax over those logits alone, or
 (``scoring="sigmoid"``) those with the largest sigmoid scores among the best groups of neighbouring experts, weighted
 by score / sum of the chosen scores, scaled, or (``scoring="softmax"``) those with the largest softmax score plus a
-correction per expert, weighted by the uncorrected scores times a scale, without division by their sum; an expert is down(f(gate h, up h)) with one of the gated activations. The
+correction per expert, weighted by the uncorrected scores times a scale, without division by their sum; an expert is down(f(gate h, up h)) with one of the gated activations,
+or (the last ``identity`` experts of the router, which have no matrices) h itself. The
 part's output, the weighted sum (plus a shared expert that every token runs, when the spec names one), is added into
 the stream.
 
@@ -36,8 +37,10 @@ class RoutedExperts(Part):
     def __init__(self, spec: RoutedExpertsSpec, ctx: BuildContext):
         if spec.activation not in ops.ACTIVATIONS:
             raise ValueError(f"routed_experts: activation {spec.activation!r} is not supported ({sorted(ops.ACTIVATIONS)})")
-        if not 0 < spec.top <= spec.experts:
-            raise ValueError(f"routed_experts: top {spec.top} of {spec.experts} experts")
+        if spec.identity < 0 or not 0 < spec.top <= spec.experts + spec.identity:
+            raise ValueError(f"routed_experts: top {spec.top} of {spec.experts} experts and {spec.identity} identity experts")
+        if spec.identity and spec.scoring not in ("softmax", "softmax_norm"):
+            raise ValueError("routed_experts: identity experts go with the softmax scoring over all experts")
         if spec.scoring not in ops.ROUTE_SCORINGS:
             raise ValueError(f"routed_experts: scoring {spec.scoring!r} is not one of {sorted(ops.ROUTE_SCORINGS)}")
         if spec.groups < 1 or spec.experts % spec.groups or not 1 <= spec.keep_groups <= spec.groups:
@@ -53,6 +56,7 @@ class RoutedExperts(Part):
         if spec.activation == "clamped_swish" and not spec.limit > 0:
             raise ValueError(f"routed_experts: the clamped swish needs a positive limit, got {spec.limit}")
         self.spec, self.ctx = spec, ctx
+        self.scored = spec.experts + spec.identity       # rows of the router
         self.w_router = self.bias = self.w_gate_up = self.w_down = self.router_product = self.pick_bias = None
         self.shared = build_ffn(spec.shared, ctx) if spec.shared is not None else None
 
@@ -61,11 +65,11 @@ class RoutedExperts(Part):
 
     def declare(self):
         s = self.spec
-        d = {"router.weight": ParamDecl((s.experts, s.hidden), "vector")}
+        d = {"router.weight": ParamDecl((self.scored, s.hidden), "vector")}
         if s.router_bias:
-            d["router.bias"] = ParamDecl((s.experts,), "vector")
+            d["router.bias"] = ParamDecl((self.scored,), "vector")
         if s.choice_bias:
-            d["correction"] = ParamDecl((s.experts,), "vector")
+            d["correction"] = ParamDecl((self.scored,), "vector")
         for e in range(s.experts):
             d[f"e{e}.gate.weight"] = ParamDecl((s.intermediate, s.hidden))
             d[f"e{e}.up.weight"] = ParamDecl((s.intermediate, s.hidden))
@@ -93,14 +97,13 @@ class RoutedExperts(Part):
         # are the float32 logits of the same inputs, from the tensor cores instead of a lane per token; a bias joins in
         # the choosing kernel.
         self.router_product = None
-        if (dt == torch.bfloat16 and s.hidden % 32 == 0 and s.experts >= 8
+        if (dt == torch.bfloat16 and s.hidden % 32 == 0 and self.scored >= 8
                 and torch.equal(self.w_router.to(torch.bfloat16).to(torch.float32), self.w_router)):
             self.router_product = Linear(self.w_router.to(torch.bfloat16), dt)
 
-    @property
-    def stores_result(self):
-        """The shared expert's last product reaches ``x`` first (and may store); the chosen experts add to it."""
-        return self.shared is not None
+    # The shared expert's last product reaches ``x`` first (and may store), the chosen experts add to it; without a shared
+    # expert the kernel that sums a token's choices stores.
+    stores_result = True
 
     def forward(self, h, x, b, ws):
         s, dt = self.spec, self.ctx.dtype
@@ -129,11 +132,13 @@ class RoutedExperts(Part):
                 ops.row_gate(h, self.w_shared_gate, own, x, accumulate=not store, stream=b.stream)
             b.next_read = after
         choice, rank, place, order = (ws.take((pairs,), torch.int32) for _ in range(4))
-        counts = ws.take((s.experts,), torch.int32)
+        store = bool(getattr(b, "store_first", False))      # still up only when no shared expert has delivered
+        b.store_first = False
+        counts = ws.take((self.scored,), torch.int32)
         weight = ws.take((pairs,), torch.float32)
         act = ws.take((pairs, s.intermediate), dt)
         y = ws.take((pairs, s.hidden), torch.float32)
-        logits = ws.take((T, s.experts), torch.float32)
+        logits = ws.take((T, self.scored), torch.float32)
         # (Letting the choosing kernel form a single token's logits itself, one launch instead of two, was measured
         # slower: 0.461 against 0.374 ms a step at width 1,024 and batch 1, 0.708 against 0.425 ms at width 2,048: one
         # block walks all of the router's rows.)
@@ -143,19 +148,20 @@ class RoutedExperts(Part):
         # steps of many pairs: the tcgen05 grouped products (bfloat16, inner sizes that TMA takes)
         grouped = (dt == torch.bfloat16 and pairs >= TC_PAIRS and s.hidden % 8 == 0
                    and s.intermediate % 8 == 0)
-        tiles = ws.take((ops.moe_tile_words(T, s.top, s.experts),), torch.int32) if grouped else None
+        tiles = ws.take((ops.moe_tile_words(T, s.top, self.scored),), torch.int32) if grouped else None
         ops.moe_route(h, self.w_router, self.bias, choice, weight, rank, counts, place, order, s.top, b.stream, logits, tiles,
                       layout=pairs > ops.MOE_FEW_PAIRS, scoring=s.scoring, groups=s.groups, keep=s.keep_groups,
-                      scale=s.route_scale, logits_ready=ready, pick_bias=self.pick_bias)
+                      scale=s.route_scale, logits_ready=ready, pick_bias=self.pick_bias, identity=s.identity)
         if grouped:
             xs = ws.take((pairs, s.hidden), dt)
             ops.moe_experts_tc(h, self.w_gate_up, self.w_down, order, place, weight, tiles, xs, act, y, x, s.top, b.stream,
-                               activation=s.activation, limit=s.limit, alpha=s.alpha)
+                               activation=s.activation, limit=s.limit, alpha=s.alpha, choice=choice if s.identity else None,
+                               store=store)
         else:
             if side is not None:
                 torch.cuda.current_stream().wait_stream(side)
             ops.moe_experts(h, self.w_gate_up, self.w_down, counts, order, weight, act, y, x, s.top, s.activation, b.stream,
-                            choice, place, limit=s.limit, alpha=s.alpha, extra=extra)
+                            choice, place, limit=s.limit, alpha=s.alpha, extra=extra, identity=s.identity, store=store)
         ws.release(mark)
 
     def _shared_beside(self, b, pairs: int, device) -> bool:

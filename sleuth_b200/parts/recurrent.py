@@ -20,6 +20,10 @@ and sequence, S_t = diag(a_t) S_(t-1) + k_t v_t^T with outputs S_t^T q_t, and sh
 a short convolution with silu; the second a decay per key channel, sigmoid(.)^(1/tau), from a low-rank projection. Their
 projections are stacked products with float32 results; decays, step sizes, the state, the skip term, the gates and the
 group norms are float32 (``csrc/state_mixers.cu``), rounded once where the output projection reads them.
+
+``retention`` (``RetentionSpec``) has one fixed decay a head and rotated queries and keys; ``gated_delta`` (``GatedDeltaSpec``)
+takes back what the state holds under the current key before it writes (``csrc/delta_rule.cu``). A step of one token a sequence
+runs everything between the projections (and the delta rule's convolution) and the output product as one kernel.
 """
 
 from __future__ import annotations
@@ -28,9 +32,9 @@ import torch
 
 from ..cache.paged import BundleRequest, StateRequest
 from ..kernels import ops
-from .base import BuildContext, Normed, ParamDecl, Part, register_mixer, result_target
+from .base import BuildContext, Normed, ParamDecl, Part, build_position, register_mixer, result_target
 from .linear import Linear
-from .spec import GatedLinearAttentionSpec, MinGRUSpec, StateSpaceSpec
+from .spec import GatedDeltaSpec, GatedLinearAttentionSpec, MinGRUSpec, RetentionSpec, StateSpaceSpec
 
 
 class MinGRU(Part):
@@ -199,6 +203,143 @@ class GatedLinearAttention(Part):
         ws.release(mark)
 
 
+def _stacked(weights, dtype) -> Linear:
+    """One product of several projections, with zero rows at the end up to a multiple of 32 (rows of its result then start on
+    whole sectors, which the product kernels' wide stores want)."""
+    w = torch.cat(weights, dim=0)
+    spare = -w.shape[0] % 32
+    if spare:
+        w = torch.cat([w, torch.zeros((spare, w.shape[1]), dtype=w.dtype, device=w.device)], dim=0)
+    return Linear(w, dtype)
+
+
+class Retention(Part):
+    stores_result = True
+
+    def __init__(self, spec: RetentionSpec, ctx: BuildContext):
+        s = spec
+        if not 1 <= s.head_dim <= 256 or len(s.decay) != s.heads or not all(d >= 0.0 for d in s.decay):
+            raise ValueError(f"retention: head_dim {s.head_dim} (at most 256), {len(s.decay)} decays for {s.heads} heads, none of them negative")
+        self.spec, self.ctx = spec, ctx
+        self.position = build_position(s.position, ctx)
+        self.nk, self.nv = s.heads * s.head_dim, s.heads * s.value_dim
+        self.decay = torch.tensor(s.decay, dtype=torch.float32, device=ctx.device)
+        self.proj = self.o = None
+
+    def declare(self):
+        s = self.spec
+        return {"q.weight": ParamDecl((self.nk, s.hidden)), "k.weight": ParamDecl((self.nk, s.hidden)),
+                "v.weight": ParamDecl((self.nv, s.hidden)), "g.weight": ParamDecl((self.nv, s.hidden)),
+                "o.weight": ParamDecl((s.hidden, self.nv))}
+
+    def bind(self, t):
+        self.proj = _stacked([t[n + ".weight"] for n in ("q", "k", "v", "g")], self.ctx.dtype)
+        self.o = Linear(t["o.weight"], self.ctx.dtype)
+
+    def cache_request(self):
+        s = self.spec
+        return StateRequest((s.heads, s.head_dim, s.value_dim), torch.float32)
+
+    def lead_weight(self):
+        return self.proj.weight if self.proj is not None else None
+
+    def forward(self, h, x, b, view, ws):
+        s, nk, nv = self.spec, self.nk, self.nv
+        if isinstance(h, Normed):
+            h = h.tensor()
+        T = h.shape[0]
+        mark = ws.mark()
+        p = self.proj.forward(h, ws=ws, stream=b.stream, out_dtype=torch.float32, next_read=self.o.weight)      # [q | k | v | g]
+        q, k, v, gate = p[:, :nk], p[:, nk:2 * nk], p[:, 2 * nk:2 * nk + nv], p[:, 2 * nk + nv:2 * nk + 2 * nv]
+        tables = self.position.tables()
+        cos, sin = tables if tables is not None else (None, None)
+        rot, q_scale = self.position.rot_dim, s.head_dim ** -0.5        # the keys' factor, applied to the queries: o is linear in both
+        g = ws.take((T, nv), self.ctx.dtype)
+        if b.max_count == 1 and ops.state_token_supported(s.head_dim, s.value_dim):
+            ops.state_token(q, k, v, gate, view.state, b.slots, g, s.heads, s.heads, s.eps, q_scale=q_scale, decay=self.decay, cos=cos,
+                            sin=sin, tok_pos=b.tok_pos, rot=rot, neighbours=self.position.neighbours, stream=b.stream)
+        else:
+            ops.rotate_rows(p, cos, sin, b.tok_pos, 2 * s.heads, s.head_dim, rot, self.position.neighbours, b.stream)
+            y = ws.take((T, nv), torch.float32)
+            need = ops.decay_scan_scratch_floats(b.n, b.max_count, s.heads, s.head_dim, s.value_dim, False)
+            scratch = ws.take((need,), torch.float32) if need else None
+            ops.decay_scan(q, k, v, self.decay.expand(T, s.heads), view.state, b.slots, b.seq_start, y, s.heads, s.heads, False,
+                           q_scale=q_scale, stream=b.stream, max_count=b.max_count, scratch=scratch)
+            ops.gated_group_norm(y, gate, None, g, s.heads, s.eps, False, stream=b.stream)
+        self.o.forward(g, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None), **result_target(b, x))
+        ws.release(mark)
+
+
+class GatedDelta(Part):
+    stores_result = True
+
+    def __init__(self, spec: GatedDeltaSpec, ctx: BuildContext):
+        s = spec
+        if s.heads % s.kv_heads or not 1 <= s.head_dim <= 256 or not 1 <= s.conv_taps <= 16:
+            raise ValueError(f"gated_delta: heads {s.heads}, kv_heads {s.kv_heads}, head_dim {s.head_dim} (at most 256), conv_taps {s.conv_taps} (1 to 16)")
+        self.spec, self.ctx = spec, ctx
+        self.nk, self.nv = s.kv_heads * s.head_dim, s.heads * s.value_dim
+        self.conv_rows = 2 * self.nk + self.nv
+        self.proj = self.o = None
+
+    def declare(self):
+        s = self.spec
+        d = {"q.weight": ParamDecl((self.nk, s.hidden)), "k.weight": ParamDecl((self.nk, s.hidden)),
+             "v.weight": ParamDecl((self.nv, s.hidden)), "g.weight": ParamDecl((self.nv, s.hidden)),
+             "b.weight": ParamDecl((s.heads, s.hidden)), "a.weight": ParamDecl((s.heads, s.hidden)),
+             "A_log": ParamDecl((s.heads,), "vector"), "dt_bias": ParamDecl((s.heads,), "vector"),
+             "norm.weight": ParamDecl((s.value_dim,), "vector", init="gain"), "o.weight": ParamDecl((s.hidden, self.nv))}
+        for n, rows in (("q", self.nk), ("k", self.nk), ("v", self.nv)):
+            d[f"{n}.conv"] = ParamDecl((rows, s.conv_taps), "vector")
+        return d
+
+    def bind(self, t):
+        self.proj = _stacked([t[n + ".weight"] for n in ("q", "k", "v", "g", "b", "a")], self.ctx.dtype)
+        self.o = Linear(t["o.weight"], self.ctx.dtype)
+        f = lambda n: t[n].to(torch.float32).contiguous()
+        self.conv = torch.cat([f("q.conv"), f("k.conv"), f("v.conv")], dim=0).contiguous()
+        self.a_log, self.dt_bias, self.gain = f("A_log"), f("dt_bias"), f("norm.weight")
+
+    def cache_request(self):
+        s = self.spec
+        parts = [("state", StateRequest((s.heads, s.head_dim, s.value_dim), torch.float32))]
+        if s.conv_taps > 1:
+            parts.append(("tail", StateRequest((s.conv_taps - 1, self.conv_rows), torch.float32)))
+        return BundleRequest(tuple(parts))
+
+    def lead_weight(self):
+        return self.proj.weight if self.proj is not None else None
+
+    def forward(self, h, x, b, view, ws):
+        s, nk, nv, H = self.spec, self.nk, self.nv, self.spec.heads
+        if isinstance(h, Normed):
+            h = h.tensor()
+        T = h.shape[0]
+        mark = ws.mark()
+        p = self.proj.forward(h, ws=ws, stream=b.stream, out_dtype=torch.float32, next_read=self.o.weight)      # [q | k | v | g | b | a]
+        rows = ws.take((T, self.conv_rows), torch.float32)
+        tail = view["tail"].state if s.conv_taps > 1 else p[:0]
+        ops.causal_conv(p, self.conv, None, tail, b.slots, b.tok_seq, b.seq_start, rows, True, b.stream, max_count=b.max_count)
+        q, k, v = rows[:, :nk], rows[:, nk:2 * nk], rows[:, 2 * nk:]
+        at = 2 * nk + nv
+        gate, raw_beta, raw_step = p[:, at:at + nv], p[:, at + nv:at + nv + H], p[:, at + nv + H:at + nv + 2 * H]
+        q_scale = s.head_dim ** -0.5
+        g = ws.take((T, nv), self.ctx.dtype)
+        if b.max_count == 1 and ops.state_token_supported(s.head_dim, s.value_dim):
+            ops.state_token(q, k, v, gate, view["state"].state, b.slots, g, H, s.kv_heads, s.eps, gain=self.gain, q_scale=q_scale,
+                            raw_beta=raw_beta, raw_step=raw_step, dt_bias=self.dt_bias, a_log=self.a_log, unit_eps=s.unit_eps, stream=b.stream)
+        else:
+            beta, log_decay = ws.take((T, H), torch.float32), ws.take((T, H), torch.float32)
+            ops.delta_prep(rows, raw_beta, raw_step, self.dt_bias, self.a_log, beta, log_decay, s.kv_heads, s.head_dim, q_scale, s.unit_eps, b.stream)
+            y = ws.take((T, nv), torch.float32)
+            ops.delta_scan(q, k, v, log_decay, beta, view["state"].state, b.slots, b.seq_start, y, H, s.kv_heads, b.stream)
+            ops.gated_group_norm(y, gate, self.gain, g, H, s.eps, False, stream=b.stream)
+        self.o.forward(g, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None), **result_target(b, x))
+        ws.release(mark)
+
+
+register_mixer("retention", Retention)
+register_mixer("gated_delta", GatedDelta)
 register_mixer("mingru", MinGRU)
 register_mixer("state_space", StateSpace)
 register_mixer("gated_linear_attention", GatedLinearAttention)

@@ -1,6 +1,6 @@
 """Two mixers side by side: both read the same normed input, each delivers into a float32 buffer of its own, and one
 kernel joins the two results into the stream (``SideBySideSpec``): half the sum of the two after an RMS norm each with a
-gain of its own, or a weighted sum. The pair's cache entry is a bundle of the two mixers' requests, so an attention's
+gain of its own, or a weighted sum (which a layer whose closing kernel can form it asks for unjoined, ``b.pair_wanted``). The pair's cache entry is a bundle of the two mixers' requests, so an attention's
 pages and a recurrence's state of one layer are taken, freed and reused together.
 
 The two mixers need nothing from each other. In a step that brings one token a sequence, where each is a chain of short
@@ -61,6 +61,7 @@ class SideBySide(Part):
             h = h.tensor()
         store = bool(getattr(b, "store_first", False))
         b.store_first = False
+        wanted, b.pair_wanted = bool(getattr(b, "pair_wanted", False)), False
         after = getattr(b, "next_read", None)
         mark = ws.mark()
         results = [ws.take(x.shape, torch.float32), ws.take(x.shape, torch.float32)]
@@ -99,6 +100,10 @@ class SideBySide(Part):
             run(0, "left", self.left, lead_weight_of(self.right))
             run(1, "right", self.right, after)
         b.next_read = after
+        if wanted and s.combine == "scaled" and store:
+            b.pair = (results[0], results[1], s.left_scale, s.right_scale)
+            ws.release(mark)
+            return
         if s.combine == "normed_mean":
             ops.pair_combine(results[0], results[1], x, self.gain_left, self.gain_right, 0.5, 0.5, s.eps, accumulate=not store,
                              stream=b.stream)

@@ -68,6 +68,9 @@ class AttentionSpec:
     qk_norm_span: str = "head"   # "head": one RMSNorm per head, gains [head_dim]; "projection": one over all heads of q
                                  # (and one over all heads of k) before they are split, gains of the projection's length
     sinks: bool = False          # a learned score per head joins the softmax denominator (no key, no value, unscaled)
+    unit_sink: bool = False      # one is added to the softmax denominator: a sink whose score is 0 (no tensor)
+    chunk: int = 0               # c > 0: a query sees the keys of its own chunk of c positions only, chunks counted from position 0
+    gate: str = "none"           # "channel": the heads' outputs are multiplied by sigmoid(W_g h) (tensor ``g_proj.weight``)
 
 
 @dataclass(frozen=True)
@@ -136,6 +139,39 @@ class GatedLinearAttentionSpec:
     tau: float
     eps: float = 1e-6
     kind: str = "gated_linear_attention"
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    """Linear attention with one fixed decay per head (``decay``). q = W_q h, k = W_k h (``heads`` x ``head_dim``), both
+    rotated by ``position``, k * head_dim^(-1/2), v = W_v h (``heads`` x ``value_dim``); per head S_t = decay S_(t-1) + k_t v_t^T,
+    o_t = S_t^T q_t; each head's o divided by its root mean square (no gain), the heads times silu(W_g h), then W_o."""
+    hidden: int
+    heads: int
+    head_dim: int
+    value_dim: int
+    decay: tuple
+    position: PositionSpec
+    eps: float = 1e-6
+    kind: str = "retention"
+
+
+@dataclass(frozen=True)
+class GatedDeltaSpec:
+    """The gated delta rule. q = W_q h and k = W_k h (``kv_heads`` x ``head_dim``), v = W_v h (``heads`` x ``value_dim``), each
+    through a short causal convolution (``conv_taps`` taps) and silu; head h reads q and k of group h // (heads / kv_heads);
+    q and k become unit vectors x / sqrt(sum x^2 + ``unit_eps``), q * head_dim^(-1/2). Per head beta = sigmoid(W_b h),
+    g = exp(-exp(A_log) softplus(W_a h + dt_bias)); S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q. Each head's o
+    RMS-normed over ``value_dim`` with a gain shared by the heads, the heads times silu(W_g h), then W_o."""
+    hidden: int
+    heads: int
+    kv_heads: int
+    head_dim: int
+    value_dim: int
+    conv_taps: int = 4
+    unit_eps: float = 1e-6
+    eps: float = 1e-6
+    kind: str = "gated_delta"
 
 
 @dataclass(frozen=True)
@@ -234,6 +270,8 @@ class RoutedExpertsSpec:
     route_scale: float = 1.0
     shared: object = None
     choice_bias: bool = False
+    identity: int = 0            # so many experts behind the ``experts`` that have matrices return the input itself; the router
+                                 # (and the correction) scores them like the others
     shared_gate: bool = False    # the shared expert's result is multiplied by sigmoid(w . h), one number a token (tensor ``shared_gate``)
 
 
@@ -244,7 +282,8 @@ class LayerSpec:
     x += mixer(norm1 x) + ffn(norm2 x), both of the same x; without ``norm2`` (None) the feed-forward reads norm1's
     output too; it may have no feed-forward (``ffn`` is None). ``kind="sandwich"``: a norm in front of and behind each
     sublayer, x += post1(mixer(norm1 x)), then x += post2(ffn(norm2 x)); with ``gated`` each sublayer's result is first
-    multiplied by sigmoid(W h + b) of the sublayer's own input h (tensors ``gate1.weight``, ``gate1.bias``, ``gate2...``).
+    multiplied by sigmoid(W h + b) of the sublayer's own input h (tensors ``gate1.weight``, ``gate1.bias``, ``gate2...``). With
+    ``norm1`` (``norm2``) None the sublayer reads the stream itself: x += post1(mixer(x)), then x += post2(ffn(x)).
 
     ``kind="hyper"``: hyper-connections. The model keeps ``streams`` copies of the stream; sublayer q (1 the mixer, 2 the
     feed-forward) reads u = sum_s in_q[s] x_s, y = sublayer(norm_q(u)), and all copies change at once from the old ones:
@@ -256,8 +295,8 @@ class LayerSpec:
     "ffn.down.weight", ...) to its name in the weight files."""
     mixer: object
     ffn: object
-    norm1: NormSpec
-    norm2: NormSpec
+    norm1: NormSpec | None
+    norm2: NormSpec | None
     names: Mapping[str, str] = field(default_factory=dict)
     kind: str = "prenorm"
     post1: NormSpec | None = None
