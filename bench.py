@@ -604,6 +604,20 @@ def fekitar_config(width, layers, heads, kv_heads, dim, window, state, lin_heads
             "layers": block}
 
 
+def levolix_config(width, layers, heads, kv_heads, dim, chunk, ret_heads, ret_dim, experts, identity, top, ff, vocab=32768) -> dict:
+    """Two layers with an attention inside chunks beside a gated delta rule, then a retention, and so on; every layer has
+    experts, some of which return their input."""
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": identity, "top": top}}
+    pair = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": chunk},
+                     "rot": {"base": 10000.0, "dims": dim}},
+            "right": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": 4}, "left_scale": 1.0, "right_scale": 1.0}
+    ret = {"heads": ret_heads, "dim": ret_dim, "vdim": heads * dim // ret_heads, "rot": {"base": 10000.0, "dims": ret_dim},
+           "decay": [1.0 - 2.0 ** (-5.0 - 6.0 * h / ret_heads) for h in range(ret_heads)]}
+    block = [("retention", ret) if i % 3 == 2 else ("parallel", pair) for i in range(layers)]
+    return {"architecture": "Levolix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [{"type": kind, "mixer": mixer, "mlp": moe} for kind, mixer in block]}
+
+
 def qwen3_like(width, layers, heads, head_dim, inter, vocab=32768) -> dict:
     return dict(CONFIG, vocab_size=vocab, hidden_size=width, num_hidden_layers=layers, num_attention_heads=heads,
                 num_key_value_heads=max(1, heads // 2), head_dim=head_dim, intermediate_size=inter, tie_word_embeddings=False)
@@ -660,13 +674,24 @@ NIROZEN_SIZES = {
     "w2048": (dict(width=2048, layers=6, heads=16, dim=128, vdim=128, q_rank=768, kv_rank=512, experts=64, top=6, ff=1408, shared_ff=1408),
               dict(width=2048, layers=6, heads=16, dim=128, rot=64, vdim=128, q_rank=768, kv_rank=512, experts=64, top=6, ff=1408)),
 }
+# Levolix beside Fekitar, the closest existing design (an attention and a recurrence with a matrix state side by side, routed
+# experts): equal width, depth, query and key/value heads, reach of the attention, state sizes and experts. Two thirds of the
+# layers are pairs in both; the others are retentions here and differential attentions there. Levolix has identity experts and
+# no shared one.
+LEVOLIX_SIZES = {
+    "w1024": (dict(width=1024, layers=9, heads=16, kv_heads=8, dim=64, chunk=1024, ret_heads=8, ret_dim=64, experts=16, identity=4, top=4, ff=768),
+              FEKITAR_SIZES["w1024"][0]),
+    "w2048": (dict(width=2048, layers=6, heads=16, kv_heads=8, dim=128, chunk=1024, ret_heads=8, ret_dim=128, experts=32, identity=8, top=4, ff=1024),
+              FEKITAR_SIZES["w2048"][0]),
+}
 DESIGNS = {"lezepel": (lezepel_config, DESIGN_SIZES), "rabadra": (rabadra_config, RABADRA_SIZES),
            "movalorn": (movalorn_config, MOVALORN_SIZES),
-           "nirozen": (nirozen_config, NIROZEN_SIZES), "fekitar": (fekitar_config, FEKITAR_SIZES)}
+           "nirozen": (nirozen_config, NIROZEN_SIZES), "fekitar": (fekitar_config, FEKITAR_SIZES),
+           "levolix": (levolix_config, LEVOLIX_SIZES)}
 # the model each design stands beside, and how its configuration is made from the second entry of a size
 TWINS = {"lezepel": ("qwen3", lambda kw: qwen3_like(**kw)), "rabadra": ("qwen3", lambda kw: qwen3_like(**kw)),
          "movalorn": ("lezepel", lambda kw: lezepel_config(**kw)), "nirozen": ("lezepel", lambda kw: lezepel_config(**kw)),
-         "fekitar": ("rabadra", lambda kw: rabadra_config(**kw))}
+         "fekitar": ("rabadra", lambda kw: rabadra_config(**kw)), "levolix": ("fekitar", lambda kw: fekitar_config(**kw))}
 
 
 def design_point(config: dict, prompt_len: int, batches, steps: int, warmup: int) -> dict:
@@ -728,9 +753,9 @@ def design_point(config: dict, prompt_len: int, batches, steps: int, warmup: int
 
 
 def run_design(args) -> dict:
-    """``--design lezepel`` / ``--design rabadra`` / ``--design movalorn`` / ``--design fekitar`` /
-    ``--design nirozen``: that design beside the closest existing model (the Qwen3 dense decoder for the first two, Lezepel
-    for Movalorn and Nirozen, Rabadra for Fekitar) at equal width, depth and active feed-forward width, random weights, bfloat16: prompt and decode throughput and where the time goes. The default workload of this file
+    """``--design lezepel`` / ``--design rabadra`` / ``--design movalorn`` / ``--design fekitar`` / ``--design nirozen`` /
+    ``--design levolix``: that design beside the closest existing model (the Qwen3 dense decoder for the first two, Lezepel
+    for Movalorn and Nirozen, Rabadra for Fekitar, Fekitar for Levolix) at equal width, depth and active feed-forward width, random weights, bfloat16: prompt and decode throughput and where the time goes. The default workload of this file
     does not change."""
     out = {"design": args.design, "dtype": "bf16", "data": "synthetic", "prompt": args.design_prompt, "sizes": {}}
     make, sizes = DESIGNS[args.design]

@@ -186,7 +186,7 @@ _SIGNATURES = {
     "slb_gated_group_norm": [P, P, L, P, I, P, L, P, I, P, I, I, I, I, F, I, P],
     "slb_rotate_rows": [P, L, P, P, P, I, I, I, I, I, P],
     "slb_delta_prep": [P, L, I, I, F, F, P, P, L, P, P, P, P, I, I, P],
-    "slb_delta_scan": [P, L, P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, P],
+    "slb_state_scan": [P, L, P, L, P, L, P, L, P, P, P, P, P, I, I, I, I, I, F, I, P, L, P],
     "slb_state_token": [P, L, P, L, P, L, P, L, P, P, P, L, P, P, P, P, P, I, I, P, P, P, P, I, I, I, I, I, F, F, F, I, P],
     "slb_unit_post": [P, L, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P],
     "slb_diff_combine": [P, P, L, P, I, I, I, F, F, F, I, I, P],

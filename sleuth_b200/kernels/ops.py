@@ -1371,18 +1371,33 @@ def _state_ok(state, heads: int, groups: int, what: str):
     return int(state.shape[2]), int(state.shape[3])
 
 
-def delta_scan(q, k, v, log_decay, beta, state, slots, seq_start, out, heads: int, groups: int, stream=None) -> None:
-    """The gated delta rule over each sequence's tokens of the step, from and back into ``state`` float32 [slots, heads, N, P]:
-    S <- exp(log_decay) S, u = beta (v - S^T k), S <- S + k u^T, out = S^T q. q, k: float32 rows of groups * N values (head h
-    reads group h // (heads / groups)); v: rows of heads * P; log_decay, beta, [T, heads]; out float32 [T, heads * P]."""
-    N, P = _state_ok(state, heads, groups, "delta_scan")
-    _cuda(log_decay, beta, slots, seq_start, out)
+def state_scan_scratch_floats(n_seqs: int, max_count: int, heads: int, N: int, P: int, delta: bool) -> int:
+    """Scratch floats ``state_scan`` needs for a step whose longest portion has ``max_count`` tokens (0: token by token)."""
+    fn = lib().dll.slb_state_scan_scratch_floats
+    fn.argtypes, fn.restype = [ctypes.c_int] * 6, ctypes.c_longlong
+    return int(fn(int(n_seqs), int(max_count), int(heads), int(N), int(P), 1 if delta else 0))
+
+
+def state_scan(q, k, v, log_decay, state, slots, seq_start, out, heads: int, groups: int, max_count: int, beta=None, q_scale: float = 1.0,
+               scratch=None, stream=None) -> None:
+    """A recurrence with a matrix state and one decay per head over each sequence's tokens of the step, from and back into
+    ``state`` float32 [slots, heads, N, P]: S <- exp(log_decay) S, u = beta (v - S^T k) (the gated delta rule) or, without
+    ``beta``, u = v; S <- S + k u^T, out = S^T q * ``q_scale``. q, k: float32 rows of groups * N values (head h reads group
+    h // (heads / groups)); v: rows of heads * P; log_decay: [T, heads], or [heads] for a fixed decay; beta: [T, heads]; out
+    float32 [T, heads * P]. Long portions run in chunks and need ``scratch`` (``state_scan_scratch_floats``)."""
+    N, P = _state_ok(state, heads, groups, "state_scan")
+    _cuda(log_decay, beta, slots, seq_start, out, scratch)
     T = out.shape[0]
-    _need(out.dtype == torch.float32 and out.shape == (T, heads * P) and log_decay.shape == beta.shape == (T, heads), "delta_scan: shapes disagree")
-    _need(slots.dtype == torch.int32 and seq_start.dtype == torch.int32 and seq_start.numel() >= slots.numel() + 1, "delta_scan: tables")
-    lib().call("slb_delta_scan", q.data_ptr(), _rows_f32(q, groups * N, "delta_scan q"), k.data_ptr(), _rows_f32(k, groups * N, "delta_scan k"),
-               v.data_ptr(), _rows_f32(v, heads * P, "delta_scan v"), _p(log_decay), _p(beta), _p(state), _p(slots), _p(seq_start), _p(out),
-               slots.numel(), heads, groups, N, P, _st(stream))
+    fixed = log_decay.dim() == 1
+    _need(out.dtype == torch.float32 and out.shape == (T, heads * P) and log_decay.dtype == torch.float32
+          and log_decay.shape == ((heads,) if fixed else (T, heads)), "state_scan: shapes disagree")
+    _need(beta is None or (beta.dtype == torch.float32 and beta.shape == (T, heads)), "state_scan: strengths")
+    _need(slots.dtype == torch.int32 and seq_start.dtype == torch.int32 and seq_start.numel() >= slots.numel() + 1, "state_scan: tables")
+    _need(q.shape[0] == k.shape[0] == v.shape[0] == T, "state_scan: one row a token")
+    lib().call("slb_state_scan", q.data_ptr(), _rows_f32(q, groups * N, "state_scan q"), k.data_ptr(), _rows_f32(k, groups * N, "state_scan k"),
+               v.data_ptr(), _rows_f32(v, heads * P, "state_scan v"), _p(log_decay), 0 if fixed else heads, _p(beta), _p(state), _p(slots),
+               _p(seq_start), _p(out), slots.numel(), heads, groups, N, P, float(q_scale), int(max_count), _p(scratch),
+               0 if scratch is None else scratch.numel(), _st(stream))
 
 
 def state_token_supported(N: int, P: int) -> bool:

@@ -51,7 +51,7 @@ class RoutedExperts(Part):
             raise ValueError("routed_experts: a choice correction goes with the softmax scoring over all experts")
         if spec.groups > 1 and spec.scoring != "sigmoid":
             raise ValueError("routed_experts: groups of experts go with the sigmoid scoring")
-        if spec.keep_groups * (spec.experts // spec.groups) < spec.top:
+        if spec.keep_groups * ((spec.experts + spec.identity) // spec.groups) < spec.top:
             raise ValueError(f"routed_experts: {spec.keep_groups} groups of {spec.experts // spec.groups} experts cannot give {spec.top} choices")
         if spec.activation == "clamped_swish" and not spec.limit > 0:
             raise ValueError(f"routed_experts: the clamped swish needs a positive limit, got {spec.limit}")

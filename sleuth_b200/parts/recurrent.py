@@ -224,6 +224,7 @@ class Retention(Part):
         self.position = build_position(s.position, ctx)
         self.nk, self.nv = s.heads * s.head_dim, s.heads * s.value_dim
         self.decay = torch.tensor(s.decay, dtype=torch.float32, device=ctx.device)
+        self.log_decay = torch.tensor(s.decay, dtype=torch.float64).log().to(torch.float32).to(ctx.device)
         self.proj = self.o = None
 
     def declare(self):
@@ -261,10 +262,10 @@ class Retention(Part):
         else:
             ops.rotate_rows(p, cos, sin, b.tok_pos, 2 * s.heads, s.head_dim, rot, self.position.neighbours, b.stream)
             y = ws.take((T, nv), torch.float32)
-            need = ops.decay_scan_scratch_floats(b.n, b.max_count, s.heads, s.head_dim, s.value_dim, False)
+            need = ops.state_scan_scratch_floats(b.n, b.max_count, s.heads, s.head_dim, s.value_dim, False)
             scratch = ws.take((need,), torch.float32) if need else None
-            ops.decay_scan(q, k, v, self.decay.expand(T, s.heads), view.state, b.slots, b.seq_start, y, s.heads, s.heads, False,
-                           q_scale=q_scale, stream=b.stream, max_count=b.max_count, scratch=scratch)
+            ops.state_scan(q, k, v, self.log_decay, view.state, b.slots, b.seq_start, y, s.heads, s.heads, b.max_count, q_scale=q_scale,
+                           scratch=scratch, stream=b.stream)
             ops.gated_group_norm(y, gate, None, g, s.heads, s.eps, False, stream=b.stream)
         self.o.forward(g, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None), **result_target(b, x))
         ws.release(mark)
@@ -332,7 +333,10 @@ class GatedDelta(Part):
             beta, log_decay = ws.take((T, H), torch.float32), ws.take((T, H), torch.float32)
             ops.delta_prep(rows, raw_beta, raw_step, self.dt_bias, self.a_log, beta, log_decay, s.kv_heads, s.head_dim, q_scale, s.unit_eps, b.stream)
             y = ws.take((T, nv), torch.float32)
-            ops.delta_scan(q, k, v, log_decay, beta, view["state"].state, b.slots, b.seq_start, y, H, s.kv_heads, b.stream)
+            need = ops.state_scan_scratch_floats(b.n, b.max_count, H, s.head_dim, s.value_dim, True)
+            scratch = ws.take((need,), torch.float32) if need else None
+            ops.state_scan(q, k, v, log_decay, view["state"].state, b.slots, b.seq_start, y, H, s.kv_heads, b.max_count, beta=beta,
+                           scratch=scratch, stream=b.stream)
             ops.gated_group_norm(y, gate, self.gain, g, H, s.eps, False, stream=b.stream)
         self.o.forward(g, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None), **result_target(b, x))
         ws.release(mark)

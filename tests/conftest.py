@@ -122,6 +122,22 @@ def nirozen_folders(tmp_path_factory):
     return out
 
 
+@pytest.fixture(scope="session")
+def levolix_folders(tmp_path_factory):
+    """Model folders of the tiny Levolix configurations, float32 weights, made once per session."""
+    import torch
+
+    import tiny_levolix
+    from sleuth_b200.weights.random_init import write_random_model
+    out = {}
+    for name, cfg in tiny_levolix.CONFIGS.items():
+        d = tmp_path_factory.mktemp(f"levolix_{name}")
+        write_random_model(d, cfg, seed=tiny_levolix.SEEDS[name], dtype=torch.float32, std=tiny_levolix.STD)
+        tiny_levolix.sharpen(d)
+        out[name] = str(d)
+    return out
+
+
 def pytest_terminal_summary(terminalreporter):
     """The largest differences from the plain implementation that the GPU tests saw (tests/closeness.py)."""
     import closeness

@@ -217,3 +217,14 @@ def forward(cfg, w, ids, work=torch.float64, margins=None):
             x = x + norm_about_one(experts(x, w, p + "mlp.", L["mlp"], margins), w[p + "norm2"], eps)
         after.append(x)
     return norm_about_one(x, w["final.norm"], eps) @ w["embed"].T, torch.stack(after)
+
+
+def greedy_generate(cfg, w, prompt, n, work=torch.float64):
+    """The ``n`` tokens that always taking the largest logit gives after ``prompt`` (the whole sequence is run again for
+    every token: slow and plain)."""
+    seq, out = list(prompt), []
+    for _ in range(n):
+        tok = int(torch.argmax(forward(cfg, w, torch.tensor(seq), work)[0][-1]))
+        out.append(tok)
+        seq.append(tok)
+    return out

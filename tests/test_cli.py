@@ -230,3 +230,31 @@ def test_the_commands_serve_a_nirozen_folder_too(tmp_path):
     lines = [ln for ln in r.stdout.splitlines() if ln.strip()]
     assert [[int(t) for t in ln.split()] for ln in lines] == [nirozen_plain.greedy_generate(cfg, w, p, 6) for p in prompts]
     assert any("NirozenConfig" in ln for ln in r.stderr.splitlines())
+
+
+@pytest.mark.gpu
+def test_the_commands_serve_a_levolix_folder_too(tmp_path):
+    """``random-model`` and ``generate`` with a Levolix ``config.json``, through the same registry: layers without front
+    norms, retentions, an attention beside a delta rule, identity experts, the embedding table as output matrix."""
+    import tiny_levolix
+    from plain import levolix_plain
+    env = dict(os.environ, PYTHONPATH=ROOT + os.pathsep + os.environ.get("PYTHONPATH", ""))
+    cfg_path = tmp_path / "config.json"
+    cfg_path.write_text(json.dumps(tiny_levolix.F))
+    folder = tmp_path / "model"
+    r = subprocess.run([sys.executable, "-m", "sleuth_b200", "random-model", str(cfg_path), str(folder), "--seed", "3",
+                        "--dtype", "fp32"], env=env, capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr
+    tiny_levolix.sharpen(folder)
+    cfg, w = plain.read_model(folder)
+    assert cfg["architecture"] == "Levolix" and w["l0.mlp.router"].shape == (7, 72) and "l0.mlp.e5.gate" not in w and "head" not in w
+    assert w["l1.mix.right.v.conv"].shape == (60, 3) and w["l1.mix.left.q.norm"].shape == (96,) and "l2.norm2" not in w
+    prompts = [[5, 17, 3, 200, 9], [150, 2], [77]]
+    text = "; ".join(",".join(map(str, p)) for p in prompts)
+    r = subprocess.run([sys.executable, "-m", "sleuth_b200", "generate", str(folder), "--prompt-ids", text, "--temperature", "0",
+                        "--max-new-tokens", "6", "--dtype", "fp32", "--max-seq-len", "128"],
+                       env=env, capture_output=True, text=True, timeout=900)
+    assert r.returncode == 0, r.stderr
+    lines = [ln for ln in r.stdout.splitlines() if ln.strip()]
+    assert [[int(t) for t in ln.split()] for ln in lines] == [levolix_plain.greedy_generate(cfg, w, p, 6) for p in prompts]
+    assert any("LevolixConfig" in ln for ln in r.stderr.splitlines())
