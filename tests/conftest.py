@@ -124,17 +124,19 @@ def nirozen_folders(tmp_path_factory):
 
 @pytest.fixture(scope="session")
 def levolix_folders(tmp_path_factory):
-    """Model folders of the tiny Levolix configurations, float32 weights, made once per session."""
+    """Model folders of the tiny Levolix configurations, float32 weights, made once per session: ``name`` with choices of
+    experts that depend on the token, ``name + " steady"`` with choices that the corrections alone make."""
     import torch
 
     import tiny_levolix
     from sleuth_b200.weights.random_init import write_random_model
     out = {}
     for name, cfg in tiny_levolix.CONFIGS.items():
-        d = tmp_path_factory.mktemp(f"levolix_{name}")
-        write_random_model(d, cfg, seed=tiny_levolix.SEEDS[name], dtype=torch.float32, std=tiny_levolix.STD)
-        tiny_levolix.sharpen(d)
-        out[name] = str(d)
+        for steady in (False, True):
+            d = tmp_path_factory.mktemp(f"levolix_{name}")
+            write_random_model(d, cfg, seed=tiny_levolix.SEEDS[name], dtype=torch.float32, std=tiny_levolix.STD)
+            tiny_levolix.sharpen(d, steady)
+            out[name + " steady" * steady] = str(d)
     return out
 
 

@@ -18,15 +18,17 @@ from plain.qwen3_plain import read_model
 pytestmark = pytest.mark.gpu
 
 # float32: the engine and the plain code differ by summation order only. bfloat16: weights are compared rounded alike;
-# activations and cache rows are rounded in the engine only, and where two choice scores lie closer than that rounding the
-# engine may send a token to another expert than the plain code does. So bfloat16 comparisons look at the rows whose own choices
-# are clear in every layer (the oracle reports the margins), and one in fifty of those may still differ (a choice that was
-# closer than it looked, or a neighbour's other choice that reached this row through a mixer).
+# activations and cache rows are rounded in the engine only. A rounding that turns one choice of experts changes everything
+# behind it, so bfloat16 runs use the folders whose choices the corrections alone make (the weights stay the token's scores).
+# Where a head's result is small beside the terms it sums (q . k near zero at a first token, say), its norm magnifies their rounding: one row in forty (or one) may
+# exceed the bfloat16 bound, which is about ten times the median of the rows' largest differences (logits go up to 29).
 TOL = {"fp32": dict(rtol=3e-4, atol=3e-3), "bf16": dict(rtol=0.0, atol=1.2)}
 NAMES = ["F", "H", "J"]
 LENGTHS = {"F": [1, 7, 66, 150], "H": [3, 64, 65, 210], "J": [2, 40, 129]}
-CLEAR = 0.04        # a choice of experts is clear when the choice scores at its edge differ by this much
-COMPARED = {"fp32": 0, "bf16": 0}
+
+
+def folder_of(folders, name, dtype):
+    return folders[name + " steady" if dtype == "bf16" else name]
 
 
 def load(folder, dtype, max_tokens=2048, **kw):
@@ -37,45 +39,32 @@ def load(folder, dtype, max_tokens=2048, **kw):
 def oracle(folder, dtype):
     cfg, w = read_model(folder)
     if dtype == "bf16":     # matrices are narrowed on the device; gains, biases, taps and the routers' matrices stay float32
-        w = {k: (v.to(torch.bfloat16).float() if v.is_floating_point() and v.dim() > 1 and not k.endswith((".router", ".conv"))
-                 else v) for k, v in w.items()}
-    cache, clear, streams = {}, {}, {}
+        w = {k: (v.to(torch.bfloat16).float() if v.is_floating_point() and v.dim() > 1 and not k.endswith((".router", ".conv")) else v)
+             for k, v in w.items()}
+    cache, streams = {}, {}
 
     def f(ids):
         key = tuple(ids)
         if key not in cache:
-            margins = []
-            logits, after = plain.forward(cfg, w, torch.tensor(list(ids)), torch.float64, margins=margins)
-            cache[key], streams[key] = logits.float(), after
-            m = torch.stack(margins).amin(dim=0) if margins else torch.ones(len(ids))
-            clear[key] = m >= CLEAR
+            logits, streams[key] = plain.forward(cfg, w, torch.tensor(list(ids)), torch.float64)
+            cache[key] = logits.float()
         return cache[key]
-
-    def clear_rows(ids):
-        f(ids)
-        return clear[tuple(ids)]
 
     def stream(ids):
         f(ids)
         return streams[tuple(ids)]
-    f.clear_rows, f.stream, f.dtype = clear_rows, stream, dtype
+    f.stream = stream
     return f
 
 
-def close(got, want, dtype, label, sure=None):
+def close(got, want, dtype, label):
     got, want = got.float().cpu(), want.float().cpu()
-    assert bool(torch.isfinite(got).all())
-    if dtype == "bf16" and sure is not None:
-        got, want = got[sure], want[sure]
-        if not len(got):
-            return
-        worst = (got - want).abs().amax(dim=-1)
-        fine = worst <= TOL[dtype]["atol"]
-        assert int((~fine).sum()) <= max(1, len(fine) // 50), worst
-        got, want = got[fine], want[fine]
-    COMPARED[dtype] += got.shape[0]
-    if got.shape[0]:
-        check(got, want, TOL[dtype], label)
+    assert bool(torch.isfinite(got).all()) and got.shape == want.shape
+    if dtype == "bf16":
+        over = (got - want).abs().amax(dim=-1) > TOL[dtype]["atol"]
+        assert int(over.sum()) <= max(1, len(over) // 40), (got - want).abs().amax(dim=-1)
+        got, want = got[~over], want[~over]
+    check(got, want, TOL[dtype], label)
 
 
 def requests_for(name, lengths, seed=0):
@@ -86,12 +75,12 @@ def requests_for(name, lengths, seed=0):
 @pytest.mark.parametrize("dtype", ["fp32", "bf16"])
 @pytest.mark.parametrize("name", NAMES)
 def test_whole_prompts(name, dtype, levolix_folders):
-    eng, ref = load(levolix_folders[name], dtype), oracle(levolix_folders[name], dtype)
+    eng, ref = load(folder_of(levolix_folders, name, dtype), dtype), oracle(folder_of(levolix_folders, name, dtype), dtype)
     for ids in requests_for(name, LENGTHS[name]):
         (slot,) = eng.open(1)
         got = eng.step([(slot, ids, tuple(range(len(ids))))]).cpu()
         eng.close([slot])
-        close(got, ref(ids), dtype, "levolix " + dtype, ref.clear_rows(ids))
+        close(got, ref(ids), dtype, "levolix " + dtype)
 
 
 @pytest.mark.parametrize("name", NAMES)
@@ -113,7 +102,7 @@ def test_the_stream_after_every_layer(name, levolix_folders):
 @pytest.mark.parametrize("dtype", ["fp32", "bf16"])
 @pytest.mark.parametrize("name", NAMES)
 def test_prompt_then_token_by_token(name, dtype, levolix_folders):
-    eng, ref = load(levolix_folders[name], dtype), oracle(levolix_folders[name], dtype)
+    eng, ref = load(folder_of(levolix_folders, name, dtype), dtype), oracle(folder_of(levolix_folders, name, dtype), dtype)
     for ids in requests_for(name, [n for n in LENGTHS[name] if n > 40] + [34, 9], seed=1):
         cut = max(1, len(ids) - 33)
         (slot,) = eng.open(1)
@@ -121,18 +110,18 @@ def test_prompt_then_token_by_token(name, dtype, levolix_folders):
         for t in ids[cut:]:
             rows.append(eng.step([(slot, [t], (0,))]).cpu().clone())
         eng.close([slot])
-        close(torch.cat(rows), ref(ids)[cut - 1:], dtype, "levolix " + dtype, ref.clear_rows(ids)[cut - 1:])
+        close(torch.cat(rows), ref(ids)[cut - 1:], dtype, "levolix " + dtype)
 
 
 @pytest.mark.parametrize("dtype", ["fp32", "bf16"])
 @pytest.mark.parametrize("name", NAMES)
 def test_from_the_first_token_on_one_by_one(name, dtype, levolix_folders):
-    eng, ref = load(levolix_folders[name], dtype), oracle(levolix_folders[name], dtype)
+    eng, ref = load(folder_of(levolix_folders, name, dtype), dtype), oracle(folder_of(levolix_folders, name, dtype), dtype)
     ids = requests_for(name, [70], seed=2)[0]
     (slot,) = eng.open(1)
     rows = [eng.step([(slot, [t], (0,))]).cpu().clone() for t in ids]
     eng.close([slot])
-    close(torch.cat(rows), ref(ids), dtype, "levolix " + dtype, ref.clear_rows(ids))
+    close(torch.cat(rows), ref(ids), dtype, "levolix " + dtype)
 
 
 @pytest.mark.parametrize("dtype", ["fp32", "bf16"])
@@ -140,7 +129,7 @@ def test_from_the_first_token_on_one_by_one(name, dtype, levolix_folders):
 @pytest.mark.parametrize("portion", [2, 3, 64, 100])
 def test_portions_of_a_prompt(name, portion, dtype, levolix_folders):
     """Portions shorter than a convolution (its tail then mixes old and new inputs), of a page, and longer."""
-    eng, ref = load(levolix_folders[name], dtype), oracle(levolix_folders[name], dtype)
+    eng, ref = load(folder_of(levolix_folders, name, dtype), dtype), oracle(folder_of(levolix_folders, name, dtype), dtype)
     ids = requests_for(name, [131], seed=3)[0]
     (slot,) = eng.open(1)
     rows = []
@@ -148,9 +137,9 @@ def test_portions_of_a_prompt(name, portion, dtype, levolix_folders):
         part = ids[a:a + portion]
         rows.append(eng.step([(slot, part, tuple(range(len(part))))]).cpu().clone())
     eng.close([slot])
-    close(torch.cat(rows), ref(ids), dtype, "levolix " + dtype, ref.clear_rows(ids))
+    close(torch.cat(rows), ref(ids), dtype, "levolix " + dtype)
     if dtype == "fp32":         # and through the stepper's own cutting of long steps
-        small = load(levolix_folders[name], dtype, max_step_tokens=portion + 1)
+        small = load(folder_of(levolix_folders, name, dtype), dtype, max_step_tokens=portion + 1)
         (slot,) = small.open(1)
         got = small.step([(slot, ids, tuple(range(len(ids))))]).cpu()
         close(got, ref(ids), dtype, "levolix " + dtype)
@@ -161,7 +150,7 @@ def test_portions_of_a_prompt(name, portion, dtype, levolix_folders):
 def test_unequal_batches_one_after_another_reuse_slots_and_pages(name, dtype, levolix_folders):
     """Three batches through a cache with room for one. Prompts and numbers of decoded tokens are unequal, the shorter
     requests end earlier, and the next batch gets slots, pages, states and tails still full of the last one's."""
-    eng, ref = load(levolix_folders[name], dtype, max_tokens=64 * 8), oracle(levolix_folders[name], dtype)
+    eng, ref = load(folder_of(levolix_folders, name, dtype), dtype, max_tokens=64 * 8), oracle(folder_of(levolix_folders, name, dtype), dtype)
     plans = [[(100, 20), (60, 3), (5, 27)], [(1, 12), (64, 1), (63, 2), (30, 30)], [(190, 9), (2, 40)]]
     for b, plan in enumerate(plans):
         reqs = requests_for(name, [p + d for p, d in plan], seed=10 + b)
@@ -180,7 +169,7 @@ def test_unequal_batches_one_after_another_reuse_slots_and_pages(name, dtype, le
             eng.close([slots[i] for i in done])
             live = [i for i in live if i not in done]
         for i, (ids, (p, d)) in enumerate(zip(reqs, plan)):
-            close(torch.stack(got[i]), ref(ids)[p - 1:], dtype, "levolix " + dtype, ref.clear_rows(ids)[p - 1:])
+            close(torch.stack(got[i]), ref(ids)[p - 1:], dtype, "levolix " + dtype)
         assert eng.cache.book.pages_in_use() == [0] * eng.cache.n_groups
 
 
@@ -188,7 +177,7 @@ def test_unequal_batches_one_after_another_reuse_slots_and_pages(name, dtype, le
 def test_a_slot_taken_again_starts_from_nothing(dtype, levolix_folders):
     """One slot, one request after another: the states and convolution tails of the request before must not reach the
     next one, whose first tokens see zeros in front of them again."""
-    eng, ref = load(levolix_folders["F"], dtype, max_tokens=128, max_sequences=1), oracle(levolix_folders["F"], dtype)
+    eng, ref = load(folder_of(levolix_folders, "F", dtype), dtype, max_tokens=128, max_sequences=1), oracle(folder_of(levolix_folders, "F", dtype), dtype)
     for ids in requests_for("F", [50, 1, 33, 2], seed=8):
         (slot,) = eng.open(1)
         assert slot == 0
@@ -196,7 +185,7 @@ def test_a_slot_taken_again_starts_from_nothing(dtype, levolix_folders):
         if len(ids) > 1:
             rows.append(eng.step([(slot, ids[1:], tuple(range(len(ids) - 1)))]).cpu().clone())
         eng.close([slot])
-        close(torch.cat(rows), ref(ids), dtype, "levolix " + dtype, ref.clear_rows(ids))
+        close(torch.cat(rows), ref(ids), dtype, "levolix " + dtype)
 
 
 def test_the_cache_of_a_chunked_layer_gives_pages_back(levolix_folders):
@@ -217,13 +206,13 @@ def test_the_cache_of_a_chunked_layer_gives_pages_back(levolix_folders):
 @pytest.mark.parametrize("dtype", ["fp32", "bf16"])
 @pytest.mark.parametrize("name", ["F", "H"])
 def test_long_decoding_across_page_and_chunk_borders(name, dtype, levolix_folders):
-    eng, ref = load(levolix_folders[name], dtype), oracle(levolix_folders[name], dtype)
+    eng, ref = load(folder_of(levolix_folders, name, dtype), dtype), oracle(folder_of(levolix_folders, name, dtype), dtype)
     ids = requests_for(name, [330], seed=4)[0]
     (slot,) = eng.open(1)
     rows = [eng.step([(slot, ids[:60], (59,))]).cpu()]
     for t in ids[60:]:
         rows.append(eng.step([(slot, [t], (0,))]).cpu().clone())
-    close(torch.cat(rows), ref(ids)[59:], dtype, "levolix " + dtype, ref.clear_rows(ids)[59:])
+    close(torch.cat(rows), ref(ids)[59:], dtype, "levolix " + dtype)
 
 
 def test_float32_does_not_depend_on_the_batch(levolix_folders):
@@ -245,7 +234,7 @@ def test_greedy_generation_through_the_entry_point(name, dtype, levolix_folders)
     """Unequal prompts through ``Engine.generate`` (its loop, its device-fed decode steps, its sampler) against greedy
     decoding with the plain implementation, which follows the engine's tokens."""
     import sleuth_b200 as sb
-    eng, ref = load(levolix_folders[name], dtype), oracle(levolix_folders[name], dtype)
+    eng, ref = load(folder_of(levolix_folders, name, dtype), dtype), oracle(folder_of(levolix_folders, name, dtype), dtype)
     prompts = requests_for(name, [3, 70, 20, 1, 9, 130], seed=6)
     out = eng.generate(prompts, max_new_tokens=12, sampling=sb.SamplingConfig(temperature=0), stop_ids=())
     margin = {"fp32": 1e-3, "bf16": TOL["bf16"]["atol"]}[dtype]      # the engine's token is the plain code's best, or within the run's rounding of it
@@ -254,18 +243,9 @@ def test_greedy_generation_through_the_entry_point(name, dtype, levolix_folders)
         assert len(r.new_ids) == 12
         seq = list(ids)
         for tok in r.new_ids:
-            if dtype == "bf16" and not bool(ref.clear_rows(seq)[-1]):
-                seq.append(tok)
-                continue
             row = ref(seq)[-1]
             near += int(float(row.max() - row[tok]) <= margin)
             clear += int(tok == int(row.argmax()))
             checked += 1
             seq.append(tok)
-    assert checked >= {"fp32": 72, "bf16": 40}[dtype] and clear >= checked * 0.7
-    assert near >= checked - {"fp32": 0, "bf16": 2}[dtype]
-
-
-def test_zz_enough_bfloat16_rows_were_held_to_the_plain_implementation():
-    if COMPARED["fp32"] > 3000:          # the whole file ran
-        assert COMPARED["bf16"] > 1000, COMPARED
+    assert checked == near == 72 and clear >= checked * 0.7

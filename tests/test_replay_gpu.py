@@ -269,7 +269,8 @@ def test_trace_run_serves_a_levolix_folder(levolix_folders, tmp_path, dtype):
     """The same program with a Levolix folder: unequal prompts in one batch, then one token each past the chunks, the
     shorter request ending first; then another request alone in the slot, pages, states and tails given back."""
     from plain import levolix_plain
-    cfg, w = plain.read_model(levolix_folders["F"])
+    folder = levolix_folders["F steady" if dtype == "bfloat16" else "F"]
+    cfg, w = plain.read_model(folder)
     if dtype == "bfloat16":
         w = {k: (v.to(torch.bfloat16).float() if v.is_floating_point() and v.dim() > 1 and not k.endswith((".router", ".conv")) else v)
              for k, v in w.items()}
@@ -295,16 +296,10 @@ def test_trace_run_serves_a_levolix_folder(levolix_folders, tmp_path, dtype):
     steps.append({"step": k, "entries": [{"id": "c", "tokens": reqs["c"], "want": [0, 36, 37, 65]}], "end": ["c"]})
     expect[k] = [("c", 0), ("c", 36), ("c", 37), ("c", 65)]
     out = tmp_path / "out"
-    replay(levolix_folders["F"], dtype, steps, out, max_tokens=89)
+    replay(folder, dtype, steps, out, max_tokens=89)
     tol = dict(rtol=3e-4, atol=3e-3) if dtype == "float32" else dict(rtol=0.0, atol=1.2)
-    wrong = total = 0
     for step, rows in expect.items():
         got = torch.from_numpy(np.fromfile(out / f"{step}.f32", dtype="<f4").reshape(len(rows), V).copy())
         want = torch.stack([ref[r][p] for r, p in rows])
         assert bool(torch.isfinite(got).all())
-        if dtype == "float32":
-            torch.testing.assert_close(got, want, **tol)
-        else:       # a token that chooses its experts by a hair may part ways with the plain code in bfloat16: count rows
-            wrong += int(((got - want).abs().amax(-1) > tol["atol"]).sum())
-            total += len(rows)
-    assert wrong <= total // 10
+        torch.testing.assert_close(got, want, **tol)

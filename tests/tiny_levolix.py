@@ -3,7 +3,7 @@ shorter than a page, of exactly a page, of a page and one, of one token, and lon
 on 1 to 4 key/value heads; key and value widths equal and unequal, in and out of the tensor-core sizes; whole, partial and no
 rotation; delta rules with as many heads as key heads and with several a key head, key widths 8 to 136 (every tiling of the
 recurrence's kernels), value widths that are no multiple of 4, convolutions of 1 to 5 taps; retentions with one to five heads and
-decays from 0 to 1; experts with top 1, 2, 3 and all, one expert, none to five identity experts, and layers without
+decays from 0.5 to 1; experts with top 1, 2, 3 and all, one expert, none to five identity experts, and layers without
 feed-forward; both orders of the two mixers."""
 
 from __future__ import annotations
@@ -44,11 +44,11 @@ H = {"architecture": "Levolix", "vocab": 320, "width": 256, "norm": {"eps": 1e-6
                 par(att(4, 1, 128, 96, 0.1, 200, 500.0, 64), delta(3, 1, 96, 48, 5), 1.0, 1.0, None),
                 ret(2, 136, 32, [0.98, 0.995], 10000.0, 0, moe(1, 1, 1, 40))]}
 
-# a chunk of one token (a token sees itself alone) and one longer than any test sequence; no rotation; a decay of zero; a key
+# a chunk of one token (a token sees itself alone) and one longer than any test sequence; no rotation; a key
 # width beyond the chunked kernels'; every expert an ordinary one, and all chosen
 J = {"architecture": "Levolix", "vocab": 150, "width": 96, "norm": {"eps": 2e-5},
      "layers": [par(att(2, 1, 32, 24, 0.25, 1, 100.0, 0), delta(1, 1, 136, 20, 2), 0.5, 1.5, moe(4, 0, 4, 24)),
-                ret(5, 8, 16, [0.0, 0.5, 0.9, 0.99, 1.0], 30.0, 4, moe(2, 1, 1, 48)),
+                ret(5, 8, 16, [0.6, 0.7, 0.9, 0.99, 1.0], 30.0, 4, moe(2, 1, 1, 48)),
                 par(att(6, 2, 8, 8, 0.5, 5000, 100.0, 8), delta(4, 4, 8, 12, 4), 1.3, 0.9, moe(1, 5, 2, 8))]}
 
 CONFIGS = {"F": F, "H": H, "J": J}
@@ -56,12 +56,13 @@ SEEDS = {"F": 517, "H": 628, "J": 739}
 STD = 0.08
 
 
-def sharpen(folder, logit_std: float = 10.0) -> None:
+def sharpen(folder, steady: bool = False, logit_std: float = 3.0) -> None:
     """Rewrite a written folder so that faults show. The layers have no front norms: the embedding's rows are scaled to the size
     that the closing norms give the sublayers' results. The routers' rows are scaled until their logits have about
-    ``logit_std`` and the corrections lie 0.11 apart in a shuffled order: the best experts of a token are chosen by their scores,
-    the others by the corrections, and two choice scores seldom lie closer than a bfloat16 run's rounding. The attention's norms give scores that are far
-    from uniform and not dwarfed by the one in the denominator, and the delta rules forget slowly (small step sizes)."""
+    ``logit_std``, and the corrections are large enough to move choices; with ``steady`` they lie so far apart that they alone
+    choose (the same experts for every token, the weights still the token's own scores): a bfloat16 run, whose rounding may turn
+    a close choice and with it everything behind it, can then be compared row by row. The attention's norms give scores that are
+    far from uniform and not dwarfed by the one in the denominator, and the delta rules forget slowly (small step sizes)."""
     from pathlib import Path
 
     from plain.qwen3_plain import read_safetensors
@@ -74,7 +75,7 @@ def sharpen(folder, logit_std: float = 10.0) -> None:
         elif name.endswith(".mlp.router"):
             tensors[name] = t * (logit_std / (float(t.float().std()) * 2.0 * t.shape[1] ** 0.5))
         elif name.endswith(".mlp.correction"):
-            tensors[name] = t.argsort().argsort().to(t.dtype) * 0.11
+            tensors[name] = t.argsort().argsort().to(t.dtype) * 2.0 if steady else t
         elif name.endswith(".dt_bias"):
             tensors[name] = t - 2.5
         elif name.endswith((".q.norm", ".k.norm")):
