@@ -77,7 +77,7 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(float* __restrict__ row
 struct ScanArgs {
   const float *q, *k, *v;              // float32 rows of G * N, G * N and H * P values
   long long q_stride, k_stride, v_stride;
-  const float* log_decay;              // [tokens, H] or (decay_stride 0) [H]
+  const float* log_decay;              // [tokens, H], or (decay_stride 0, the only form without beta) [H]
   long long decay_stride;
   const float* beta;                   // [tokens, H]; null: no correction, u = v
   float* state;                        // [slots, H, N, P]
@@ -89,6 +89,7 @@ struct ScanArgs {
   // the chunked form
   int chunks;                          // chunks of the longest portion
   float* w;                            // [n_seqs, chunks, H, N, 64]
+  float* ends;                         // [n_seqs, chunks, H, 68]: decays from a token to its chunk's end, then the whole chunk's
   float* starts;                       // [n_seqs, chunks, H, N, P]
   int vec;                             // q, k and v rows may be read 16 bytes at a time
 };
@@ -153,11 +154,11 @@ __global__ void __launch_bounds__(128) state_walk_kernel(ScanArgs a) {
 // never positive, formed from sums in double.
 constexpr int kChunk = 64;
 constexpr int kPad = kChunk + 4;       // row length of a transposed tile: 16-byte pieces of neighbouring rows fall into other banks
-constexpr int kSlice = 16;             // value columns of a block of the state kernel
 constexpr int kOutCols = 64;           // value columns of a block of the output kernel
 
-// Sums of the chunk's log decays into L[0 .. 63] (constant beyond the chunk's tokens); called by one whole warp.
-__device__ __forceinline__ void chunk_log_sums(const ScanArgs& a, int t0, int cnt, int h, double* L) {
+// Sums of the chunk's log decays, each as a pair of floats whose sum is the sum to double precision (constant beyond the
+// chunk's tokens); called by one whole warp.
+__device__ __forceinline__ void chunk_log_sums(const ScanArgs& a, int t0, int cnt, int h, float2* L) {
   const int lane = threadIdx.x & 31;
   double lo = 2 * lane < cnt ? (double)a.log_decay[(size_t)(t0 + 2 * lane) * a.decay_stride + h] : 0.0;
   double hi = 2 * lane + 1 < cnt ? (double)a.log_decay[(size_t)(t0 + 2 * lane + 1) * a.decay_stride + h] : 0.0;
@@ -169,24 +170,30 @@ __device__ __forceinline__ void chunk_log_sums(const ScanArgs& a, int t0, int cn
     const double v = __shfl_up_sync(0xffffffffu, run, o);
     if (lane >= o) run += v;
   }
-  L[2 * lane] = run - hi;
-  L[2 * lane + 1] = run;
+  const double first = run - hi;
+  const float f0 = (float)first, f1 = (float)run;
+  L[2 * lane] = make_float2(f0, (float)(first - (double)f0));
+  L[2 * lane + 1] = make_float2(f1, (float)(run - (double)f1));
 }
 
-__device__ __forceinline__ float exp_of(double x) { return expf((float)x); }
+__device__ __forceinline__ float decay_between(const float2& to, const float2& from) { return expf((to.x - from.x) + (to.y - from.y)); }
+__device__ __forceinline__ float decay_since_start(const float2& to) { return expf(to.x + to.y); }
 
-// A [64, N] tile of rows transposed into shared memory, dst[n][i]; rows from cnt on are zero. n_pad: rows of dst (>= N).
-__device__ __forceinline__ void load_transposed(float* dst, const float* src, long long stride, int cnt, int N, int n_pad) {
-  for (int idx = threadIdx.x; idx < n_pad * (kChunk / 4); idx += blockDim.x) {
-    const int n = idx % n_pad, i = (idx / n_pad) * 4;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (n < N) {
-      if (i < cnt) v.x = src[(size_t)i * stride + n];
-      if (i + 1 < cnt) v.y = src[(size_t)(i + 1) * stride + n];
-      if (i + 2 < cnt) v.z = src[(size_t)(i + 2) * stride + n];
-      if (i + 3 < cnt) v.w = src[(size_t)(i + 3) * stride + n];
-    }
+// A [64, N] tile of rows transposed into shared memory, dst[n][i]; rows from cnt on are zero.
+template <int THREADS>
+__device__ __forceinline__ void load_transposed(float* dst, const float* src, long long stride, int cnt, int N) {
+  int n = threadIdx.x, i = 0;
+  while (n >= N) { n -= N; i += 4; }
+  for (; i < kChunk;) {
+    const float* p = src + (size_t)i * stride + n;
+    float4 v;
+    v.x = i < cnt ? p[0] : 0.0f;
+    v.y = i + 1 < cnt ? p[stride] : 0.0f;
+    v.z = i + 2 < cnt ? p[2 * stride] : 0.0f;
+    v.w = i + 3 < cnt ? p[3 * stride] : 0.0f;
     *reinterpret_cast<float4*>(dst + n * kPad + i) = v;
+    n += THREADS;
+    while (n >= N) { n -= N; i += 4; }
   }
 }
 
@@ -197,190 +204,206 @@ __device__ __forceinline__ void fma4(float4& acc, float s, const float4& v) {
   acc.w = fmaf(s, v.w, acc.w);
 }
 
-// grid (chunks, H, sequences), 128 threads: U into `out`, W transposed into `w`.
+__device__ __forceinline__ void copy_async(float* dst, const float* src, bool valid, bool bytes16) {
+  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+  if (bytes16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(valid ? 16 : 0) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(d), "l"(src), "r"(valid ? 4 : 0) : "memory");
+}
+
+// `rows` rows of `cols` floats into shared memory (row length `ld`); rows from `valid` on and columns from `live` on become zero.
+template <int THREADS>
+__device__ __forceinline__ void copy_tile(float* dst, int ld, const float* src, long long stride, int rows, int cols, int valid, int live, bool vec) {
+  const int step = vec ? 4 : 1, per = cols / step;         // vec: cols, live and the addresses are multiples of 4 floats
+  int c = threadIdx.x, r = 0;
+  while (c >= per) { c -= per; ++r; }
+  while (r < rows) {
+    const bool in = r < valid && c * step < live;
+    copy_async(dst + r * ld + c * step, src + (in ? (size_t)r * stride + c * step : 0), in, vec);
+    c += THREADS;
+    while (c >= per) { c -= per; ++r; }
+  }
+}
+
+// grid (chunks, H, sequences), 128 threads: U into `out`, W transposed into `w`, the decays from every token to the chunk's end
+// (and behind them the whole chunk's) into `ends`.
 __global__ void __launch_bounds__(128) chunk_solve_kernel(ScanArgs a) {
   pdl_enter();
   extern __shared__ __align__(16) float sm[];
-  __shared__ double L[kChunk];
+  __shared__ float2 L[kChunk];
   __shared__ float sbeta[kChunk], sgrow[kChunk];
   const int chunk = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
   const int t0 = a.seq_start[seq] + chunk * kChunk, cnt = min(kChunk, a.seq_start[seq + 1] - t0);
   if (cnt <= 0) return;
   const int N = a.N, P = a.P, g = h / (a.H / a.G);
-  float* KT = sm;                      // [N][kPad]
+  float* KT = sm;                      // [N][kPad], then W in the same layout
   float* AT = KT + N * kPad;           // [64][kPad]: AT[j][i] = A_ij
-  float* X = AT + kChunk * kPad;       // [64][128]: a thread's column of the solution
   const float* krow = a.k + (size_t)t0 * a.k_stride + (size_t)g * N;
-  load_transposed(KT, krow, a.k_stride, cnt, N, N);
+  load_transposed<128>(KT, krow, a.k_stride, cnt, N);
   if (tid < 32) chunk_log_sums(a, t0, cnt, h, L);
   if (tid >= 64) sbeta[tid - 64] = tid - 64 < cnt ? a.beta[(size_t)(t0 + tid - 64) * a.H + h] : 0.0f;
   __syncthreads();
-  if (tid < kChunk) sgrow[tid] = exp_of(L[tid]);
+  float* ends = a.ends + (((size_t)seq * a.chunks + chunk) * a.H + h) * (kChunk + 4);
+  if (tid < kChunk) {
+    const float grow = decay_since_start(L[tid]);
+    sgrow[tid] = grow;
+    ends[tid] = tid < cnt ? decay_between(L[cnt - 1], L[tid]) : 0.0f;
+    if (tid == cnt - 1) ends[kChunk] = grow;
+  }
   {
-    const int i0 = (tid & 15) * 4, j0 = (tid >> 4) * 8;
-    if (j0 <= i0 + 3) {
+    // a warp takes 32 rows x 32 keys or so: lanes 8 (rows, 4 each) x 4 (keys, 8 each)
+    const int warp = tid >> 5, lane = tid & 31;
+    const int i0 = (warp & 1) * 32 + (lane & 7) * 4, j0 = (warp >> 1) * 32 + (lane >> 3) * 8;
+    if ((warp >> 1) <= (warp & 1)) {
       float4 acc[8];
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
       for (int n = 0; n < N; ++n) {
         const float4 ki = *reinterpret_cast<const float4*>(KT + n * kPad + i0);
         const float4 ka = *reinterpret_cast<const float4*>(KT + n * kPad + j0), kb = *reinterpret_cast<const float4*>(KT + n * kPad + j0 + 4);
         fma4(acc[0], ka.x, ki); fma4(acc[1], ka.y, ki); fma4(acc[2], ka.z, ki); fma4(acc[3], ka.w, ki);
         fma4(acc[4], kb.x, ki); fma4(acc[5], kb.y, ki); fma4(acc[6], kb.z, ki); fma4(acc[7], kb.w, ki);
       }
+      float2 li[4];
+      float bi[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) { li[i] = L[i0 + i]; bi[i] = sbeta[i0 + i]; }
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int jj = j0 + j;
-        const double lj = L[jj];
+        const float2 lj = L[jj];
         float4 r;
-        r.x = i0 > jj ? sbeta[i0] * exp_of(L[i0] - lj) * acc[j].x : 0.0f;
-        r.y = i0 + 1 > jj ? sbeta[i0 + 1] * exp_of(L[i0 + 1] - lj) * acc[j].y : 0.0f;
-        r.z = i0 + 2 > jj ? sbeta[i0 + 2] * exp_of(L[i0 + 2] - lj) * acc[j].z : 0.0f;
-        r.w = i0 + 3 > jj ? sbeta[i0 + 3] * exp_of(L[i0 + 3] - lj) * acc[j].w : 0.0f;
+        r.x = i0 > jj ? bi[0] * decay_between(li[0], lj) * acc[j].x : 0.0f;
+        r.y = i0 + 1 > jj ? bi[1] * decay_between(li[1], lj) * acc[j].y : 0.0f;
+        r.z = i0 + 2 > jj ? bi[2] * decay_between(li[2], lj) * acc[j].z : 0.0f;
+        r.w = i0 + 3 > jj ? bi[3] * decay_between(li[3], lj) * acc[j].w : 0.0f;
         *reinterpret_cast<float4*>(AT + jj * kPad + i0) = r;
       }
     }
   }
   __syncthreads();
-  // forward substitution, a column of [beta v | beta e^L k] a thread, sixteen rows at a time; nothing is shared but A
+  // forward substitution, a column of [beta v | beta e^L k] a thread, in registers; nothing is shared but A
   const float* vrow = a.v + (size_t)t0 * a.v_stride + (size_t)h * P;
-  float* wt = a.w + ((((size_t)seq * a.chunks + chunk) * a.H + h) * N) * kChunk;
   for (int c0 = 0; c0 < P + N; c0 += 128) {
     const int c = c0 + tid;
-    if (c >= P + N) break;
     const bool is_v = c < P;
-    for (int b = 0; b < kChunk; b += 16) {
-      float acc[16];
-#pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const int r = b + i;
-        acc[i] = r < cnt ? (is_v ? sbeta[r] * vrow[(size_t)r * a.v_stride + c] : sbeta[r] * sgrow[r] * krow[(size_t)r * a.k_stride + c - P]) : 0.0f;
-      }
-      for (int j = 0; j < b; ++j) {
-        const float x = -X[j * 128 + tid];
-        const float* ar = AT + j * kPad + b;
-#pragma unroll
-        for (int i = 0; i < 16; i += 4) {
-          const float4 m = *reinterpret_cast<const float4*>(ar + i);
-          acc[i] = fmaf(m.x, x, acc[i]);
-          acc[i + 1] = fmaf(m.y, x, acc[i + 1]);
-          acc[i + 2] = fmaf(m.z, x, acc[i + 2]);
-          acc[i + 3] = fmaf(m.w, x, acc[i + 3]);
-        }
-      }
-#pragma unroll
-      for (int j = 0; j < 15; ++j) {
-        const float x = -acc[j];
-        const float* ar = AT + (b + j) * kPad + b;
-#pragma unroll
-        for (int i = (j + 1) & ~3; i < 16; i += 4) {
-          const float4 m = *reinterpret_cast<const float4*>(ar + i);          // entries at or above the diagonal are zero
-          if (i > j) acc[i] = fmaf(m.x, x, acc[i]);
-          if (i + 1 > j) acc[i + 1] = fmaf(m.y, x, acc[i + 1]);
-          if (i + 2 > j) acc[i + 2] = fmaf(m.z, x, acc[i + 2]);
-          if (i + 3 > j) acc[i + 3] = fmaf(m.w, x, acc[i + 3]);
-        }
-      }
-#pragma unroll
-      for (int i = 0; i < 16; ++i) X[(b + i) * 128 + tid] = acc[i];
+    if (c < P + N) {
+      float x[kChunk];
       if (is_v) {
+        const float* p = vrow + c;
 #pragma unroll
-        for (int i = 0; i < 16; ++i)
-          if (b + i < cnt) a.out[(size_t)(t0 + b + i) * ((size_t)a.H * P) + (size_t)h * P + c] = acc[i];
+        for (int i = 0; i < kChunk; ++i) x[i] = i < cnt ? p[(size_t)i * a.v_stride] : 0.0f;
+#pragma unroll
+        for (int i = 0; i < kChunk; ++i) x[i] *= sbeta[i];
       } else {
+        const float* p = KT + (c - P) * kPad;
 #pragma unroll
-        for (int i = 0; i < 16; i += 4)
-          *reinterpret_cast<float4*>(wt + (size_t)(c - P) * kChunk + b + i) = make_float4(acc[i], acc[i + 1], acc[i + 2], acc[i + 3]);
+        for (int i = 0; i < kChunk; i += 4) {
+          const float4 v = *reinterpret_cast<const float4*>(p + i);
+          x[i] = v.x * (sbeta[i] * sgrow[i]);
+          x[i + 1] = v.y * (sbeta[i + 1] * sgrow[i + 1]);
+          x[i + 2] = v.z * (sbeta[i + 2] * sgrow[i + 2]);
+          x[i + 3] = v.w * (sbeta[i + 3] * sgrow[i + 3]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < kChunk - 1; ++j) {
+        const float f = -x[j];
+        const float* ar = AT + j * kPad;
+#pragma unroll
+        for (int i = (j + 1) & ~3; i < kChunk; i += 4) {
+          const float4 m = *reinterpret_cast<const float4*>(ar + i);
+          if (i > j) x[i] = fmaf(m.x, f, x[i]);
+          if (i + 1 > j) x[i + 1] = fmaf(m.y, f, x[i + 1]);
+          if (i + 2 > j) x[i + 2] = fmaf(m.z, f, x[i + 2]);
+          if (i + 3 > j) x[i + 3] = fmaf(m.w, f, x[i + 3]);
+        }
+      }
+      if (is_v) {
+        float* p = a.out + (size_t)t0 * ((size_t)a.H * P) + (size_t)h * P + c;
+#pragma unroll
+        for (int i = 0; i < kChunk; ++i)
+          if (i < cnt) p[(size_t)i * ((size_t)a.H * P)] = x[i];
+      } else {                         // this thread's own column of KT: nobody else reads it any more
+        float* p = KT + (c - P) * kPad;
+#pragma unroll
+        for (int i = 0; i < kChunk; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
       }
     }
   }
+  __syncthreads();
+  float* wt = a.w + ((((size_t)seq * a.chunks + chunk) * a.H + h) * N) * kChunk;
+  for (int i = tid; i < N * (kChunk / 4); i += 128)
+    reinterpret_cast<float4*>(wt)[i] = *reinterpret_cast<const float4*>(KT + (i >> 4) * kPad + (i & 15) * 4);
 }
 
-__device__ __forceinline__ void copy_async(float* dst, const float* src, bool valid, int bytes16) {
-  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
-  if (bytes16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(valid ? 16 : 0) : "memory");
-  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(d), "l"(src), "r"(valid ? 4 : 0) : "memory");
-}
-
-// grid (slices of 16 value columns, H, sequences), 128 threads: walks the sequence's chunks with its slice of the state in
-// registers (thread: RN rows x 2 columns) and a copy in shared memory; leaves every chunk's start state in `starts`, u in `out`
-// (delta rule) and the last state in the slot. The next chunk's W and k are on their way while one is worked on.
-template <int RN, bool DELTA>
-__global__ void __launch_bounds__(128) chunk_state_kernel(ScanArgs a) {
+// grid (slices of PS value columns, H, sequences), 256 threads: walks the sequence's chunks with its slice of the state; leaves
+// every chunk's start state in `starts`, u in `out` (delta rule) and the last state in the slot. Both products run as 4 x 2 (RN x 2)
+// outputs a thread with the inner dimension cut into KS pieces whose partial sums meet in shared memory; behind them a thread owns
+// elements tid, tid + 256, ... of the chunk's u and of the state. The next chunk's W, k and values are on their way meanwhile.
+template <int RN, int PS, bool DELTA>
+__global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
   pdl_enter();
   extern __shared__ __align__(16) float sm[];
   constexpr int NP = 16 * RN;          // rows of the state, padded
-  float* sS = sm;                      // [NP][16]
-  float* sV = sS + NP * kSlice;        // [64][16]: u times the decay to the chunk's end
-  float* sK = sV + kChunk * kSlice;    // [2][64][NP]
+  constexpr int CG = PS / 2;           // pairs of columns
+  constexpr int KS = 16 / CG;          // pieces of the inner dimension
+  constexpr int OS = NP * PS / 256, OU = kChunk * PS / 256;      // elements of the state and of u that a thread owns
+  constexpr int PARTS = KS * (NP > kChunk ? NP : kChunk) * PS;
+  float* sS = sm;                      // [NP][PS]
+  float* sV = sS + NP * PS;            // [64][PS]: u times the decay to the chunk's end
+  float* sP = sV + kChunk * PS;        // partial sums
+  float* sE = sP + PARTS;              // [2][68]: decays to the chunk's end, then the whole chunk's
+  float* sK = sE + 2 * (kChunk + 4);   // [2][64][NP]
   float* sW = sK + 2 * kChunk * NP;    // [2][NP][64] (delta rule)
-  __shared__ float to_end[2][kChunk];
-  __shared__ float whole[2];
-  __shared__ double L[kChunk];
   const int h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
   const int N = a.N, P = a.P, g = h / (a.H / a.G);
   const int first = a.seq_start[seq], total = a.seq_start[seq + 1] - first;
   const int live = (total + kChunk - 1) / kChunk;
   if (live <= 0) return;
-  const int tp = tid & 7, tr = tid >> 3;                  // columns 2 tp, 2 tp + 1; 16 groups of rows
-  const int p0 = blockIdx.x * kSlice + 2 * tp, n0 = tr * RN, i0 = tr * 4;
-  for (int i = tid; i < 2 * kChunk * NP; i += 128) {      // channels beyond N stay zero in every chunk
-    sK[i] = 0.0f;
-    if (DELTA) sW[i] = 0.0f;
-  }
-  float* st = a.state + (((size_t)a.slots[seq] * a.H + h) * N) * P;
-  float S[RN][2];
+  const int tp = tid % CG, tr = (tid / CG) & 15, piece = tid / (16 * CG);
+  const int c0 = blockIdx.x * PS, cols = min(PS, P - c0);
+  const size_t out_stride = (size_t)a.H * P;
+  const float log_fixed = DELTA ? 0.0f : fmaxf(a.log_decay[h], -1e30f);
+  if (DELTA && NP > N)                 // W's rows beyond N stay zero in every chunk
+    for (int i = tid; i < 2 * NP * kChunk; i += 256) sW[i] = 0.0f;
+  // element e = tid + 256 r of the state: (row part e / (16 PS), row group (e / PS) % 16, column e % PS) -> row group * RN + part
+  auto state_row = [&](int e) { return ((e / PS) & 15) * RN + e / (16 * PS); };
+  float* st = a.state + (((size_t)a.slots[seq] * a.H + h) * N) * P + c0;
+  float S[OS];
 #pragma unroll
-  for (int r = 0; r < RN; ++r) {
-#pragma unroll
-    for (int e = 0; e < 2; ++e) S[r][e] = n0 + r < N && p0 + e < P ? st[(size_t)(n0 + r) * P + p0 + e] : 0.0f;
-    *reinterpret_cast<float2*>(sS + (n0 + r) * kSlice + 2 * tp) = make_float2(S[r][0], S[r][1]);
+  for (int r = 0; r < OS; ++r) {
+    const int e = tid + 256 * r, n = state_row(e), p = e % PS;
+    S[r] = n < N && p < cols ? st[(size_t)n * P + p] : 0.0f;
+    sS[n * PS + p] = S[r];
   }
   __syncthreads();
   auto fetch = [&](int c) {            // one commit group a chunk
     if (c < live) {
-      const int t0 = first + c * kChunk, cnt = min(kChunk, total - c * kChunk);
-      float* kd = sK + (c & 1) * kChunk * NP;
-      const float* ks = a.k + (size_t)t0 * a.k_stride + (size_t)g * N;
-      if (a.vec) {
-        const int q = N >> 2;
-        for (int i = tid; i < kChunk * q; i += 128) {
-          const int r = i / q, n = (i - r * q) * 4;
-          copy_async(kd + r * NP + n, ks + (size_t)min(r, cnt - 1) * a.k_stride + n, r < cnt, 1);
-        }
-      } else {
-        for (int i = tid; i < kChunk * N; i += 128) {
-          const int r = i / N, n = i - r * N;
-          copy_async(kd + r * NP + n, ks + (size_t)min(r, cnt - 1) * a.k_stride + n, r < cnt, 0);
-        }
-      }
+      const int cnt = min(kChunk, total - c * kChunk), b = c & 1;
+      copy_tile<256>(sK + b * kChunk * NP, NP, a.k + (size_t)(first + c * kChunk) * a.k_stride + (size_t)g * N, a.k_stride, kChunk, NP, cnt, N, a.vec);
       if (DELTA) {
-        float* wd = sW + (c & 1) * NP * kChunk;
-        const float* ws = a.w + ((((size_t)seq * a.chunks + c) * a.H + h) * N) * kChunk;
-        for (int i = tid; i < N * (kChunk / 4); i += 128) copy_async(wd + i * 4, ws + i * 4, true, 1);
-      }
-      if (tid >= 96) {                 // the last warp: the chunk's decays
-        chunk_log_sums(a, t0, cnt, h, L);
-        __syncwarp();
-        const double end = L[cnt - 1];
-        for (int i = tid - 96; i < kChunk; i += 32) to_end[c & 1][i] = i < cnt ? exp_of(end - L[i]) : 0.0f;
-        if (tid == 96) whole[c & 1] = exp_of(end);
-        __syncwarp();
+        const size_t at = ((size_t)seq * a.chunks + c) * a.H + h;
+        float* wd = sW + b * NP * kChunk;
+        const float* ws = a.w + at * N * kChunk;
+        for (int i = tid; i < N * (kChunk / 4); i += 256) copy_async(wd + i * 4, ws + i * 4, true, true);
+        if (tid < kChunk / 4 + 1) copy_async(sE + b * (kChunk + 4) + tid * 4, a.ends + at * (kChunk + 4) + tid * 4, true, true);
+      } else if (tid <= kChunk) {      // a fixed decay: its powers
+        const float left = tid == kChunk ? (float)cnt : (float)(cnt - 1 - tid);
+        sE[b * (kChunk + 4) + tid] = left < 0.0f ? 0.0f : (left == 0.0f ? 1.0f : expf(left * log_fixed));
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  float uv[4][2];                      // this thread's values of U (or v) of the chunk
+  float uv[OU];                        // this thread's elements of U (or v) of the chunk, element e as for the state with 4 parts
+  auto u_row = [&](int e) { return ((e / PS) & 15) * 4 + e / (16 * PS); };
   auto values = [&](int c) {
     const int t0 = first + c * kChunk, cnt = c < live ? min(kChunk, total - c * kChunk) : 0;
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const bool in = i0 + i < cnt && p0 + e < P;
-        uv[i][e] = !in ? 0.0f : (DELTA ? a.out[(size_t)(t0 + i0 + i) * ((size_t)a.H * P) + (size_t)h * P + p0 + e]
-                                       : a.v[(size_t)(t0 + i0 + i) * a.v_stride + (size_t)h * P + p0 + e]);
-      }
+    for (int r = 0; r < OU; ++r) {
+      const int e = tid + 256 * r, i = u_row(e), p = e % PS;
+      uv[r] = i < cnt && p < cols ? (DELTA ? a.out[(size_t)(t0 + i) * out_stride + (size_t)h * P + c0 + p] : a.v[(size_t)(t0 + i) * a.v_stride + (size_t)h * P + c0 + p]) : 0.0f;
+    }
   };
   fetch(0);
   values(0);
@@ -388,22 +411,24 @@ __global__ void __launch_bounds__(128) chunk_state_kernel(ScanArgs a) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                   // chunk c is here; the other buffers are free; sS holds the state
     fetch(c + 1);
-    const int t0 = first + c * kChunk, cnt = min(kChunk, total - c * kChunk);
-    float* start = a.starts + ((((size_t)seq * a.chunks + c) * a.H + h) * N) * P;
+    const int t0 = first + c * kChunk, cnt = min(kChunk, total - c * kChunk), b = c & 1;
+    const float* ends = sE + b * (kChunk + 4);
+    float* start = a.starts + ((((size_t)seq * a.chunks + c) * a.H + h) * N) * P + c0;
 #pragma unroll
-    for (int r = 0; r < RN; ++r)
-#pragma unroll
-      for (int e = 0; e < 2; ++e)
-        if (n0 + r < N && p0 + e < P) start[(size_t)(n0 + r) * P + p0 + e] = S[r][e];
+    for (int r = 0; r < OS; ++r) {
+      const int e = tid + 256 * r, n = state_row(e), p = e % PS;
+      if (n < N && p < cols) start[(size_t)n * P + p] = S[r];
+    }
     if (DELTA) {
-      const float* w = sW + (c & 1) * NP * kChunk;
+      const float* w = sW + b * NP * kChunk + tr * 4;
       float acc[4][2];
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = 0.0f;
+      const int lo = piece * (NP / KS);
 #pragma unroll 8
-      for (int n = 0; n < NP; ++n) {
-        const float4 w4 = *reinterpret_cast<const float4*>(w + n * kChunk + i0);
-        const float2 s2 = *reinterpret_cast<const float2*>(sS + n * kSlice + 2 * tp);
+      for (int n = lo; n < lo + NP / KS; ++n) {
+        const float4 w4 = *reinterpret_cast<const float4*>(w + n * kChunk);
+        const float2 s2 = *reinterpret_cast<const float2*>(sS + n * PS + 2 * tp);
         acc[0][0] = fmaf(w4.x, s2.x, acc[0][0]); acc[0][1] = fmaf(w4.x, s2.y, acc[0][1]);
         acc[1][0] = fmaf(w4.y, s2.x, acc[1][0]); acc[1][1] = fmaf(w4.y, s2.y, acc[1][1]);
         acc[2][0] = fmaf(w4.z, s2.x, acc[2][0]); acc[2][1] = fmaf(w4.z, s2.y, acc[2][1]);
@@ -411,56 +436,77 @@ __global__ void __launch_bounds__(128) chunk_state_kernel(ScanArgs a) {
       }
 #pragma unroll
       for (int i = 0; i < 4; ++i)
+        *reinterpret_cast<float2*>(sP + piece * kChunk * PS + (i * 16 + tr) * PS + 2 * tp) = make_float2(acc[i][0], acc[i][1]);
+      __syncthreads();
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          uv[i][e] -= acc[i][e];
-          if (i0 + i < cnt && p0 + e < P) a.out[(size_t)(t0 + i0 + i) * ((size_t)a.H * P) + (size_t)h * P + p0 + e] = uv[i][e];
-        }
-    }
+      for (int r = 0; r < OU; ++r) {
+        const int e = tid + 256 * r, i = u_row(e), p = e % PS;
+        float sum = 0.0f;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const float f = to_end[c & 1][i0 + i];
-      *reinterpret_cast<float2*>(sV + (i0 + i) * kSlice + 2 * tp) = make_float2(uv[i][0] * f, uv[i][1] * f);
-    }
-    __syncthreads();
-    values(c + 1);
-    const float keep = whole[c & 1];
-#pragma unroll
-    for (int r = 0; r < RN; ++r) { S[r][0] *= keep; S[r][1] *= keep; }
-    const float* kk = sK + (c & 1) * kChunk * NP + n0;
-#pragma unroll 4
-    for (int i = 0; i < kChunk; ++i) {
-      const float2 u2 = *reinterpret_cast<const float2*>(sV + i * kSlice + 2 * tp);
-      if constexpr (RN >= 4) {
-#pragma unroll
-        for (int r = 0; r < RN; r += 4) {
-          const float4 k4 = *reinterpret_cast<const float4*>(kk + i * NP + r);
-          S[r][0] = fmaf(k4.x, u2.x, S[r][0]); S[r][1] = fmaf(k4.x, u2.y, S[r][1]);
-          S[r + 1][0] = fmaf(k4.y, u2.x, S[r + 1][0]); S[r + 1][1] = fmaf(k4.y, u2.y, S[r + 1][1]);
-          S[r + 2][0] = fmaf(k4.z, u2.x, S[r + 2][0]); S[r + 2][1] = fmaf(k4.z, u2.y, S[r + 2][1]);
-          S[r + 3][0] = fmaf(k4.w, u2.x, S[r + 3][0]); S[r + 3][1] = fmaf(k4.w, u2.y, S[r + 3][1]);
-        }
-      } else {
-        const float2 k2 = *reinterpret_cast<const float2*>(kk + i * NP);
-        S[0][0] = fmaf(k2.x, u2.x, S[0][0]); S[0][1] = fmaf(k2.x, u2.y, S[0][1]);
-        S[1][0] = fmaf(k2.y, u2.x, S[1][0]); S[1][1] = fmaf(k2.y, u2.y, S[1][1]);
+        for (int k = 0; k < KS; ++k) sum += sP[k * kChunk * PS + e];
+        uv[r] -= sum;
+        if (i < cnt && p < cols) a.out[(size_t)(t0 + i) * out_stride + (size_t)h * P + c0 + p] = uv[r];
       }
     }
 #pragma unroll
-    for (int r = 0; r < RN; ++r) *reinterpret_cast<float2*>(sS + (n0 + r) * kSlice + 2 * tp) = make_float2(S[r][0], S[r][1]);
+    for (int r = 0; r < OU; ++r) {
+      const int e = tid + 256 * r, i = u_row(e), p = e % PS;
+      sV[i * PS + p] = uv[r] * ends[i];
+    }
+    __syncthreads();
+    values(c + 1);
+    {
+      const float* kk = sK + b * kChunk * NP + tr * RN;
+      float acc[RN][2];
+#pragma unroll
+      for (int r = 0; r < RN; ++r) acc[r][0] = acc[r][1] = 0.0f;
+      const int lo = piece * (kChunk / KS);
+#pragma unroll 8
+      for (int i = lo; i < lo + kChunk / KS; ++i) {
+        const float2 u2 = *reinterpret_cast<const float2*>(sV + i * PS + 2 * tp);
+        if constexpr (RN >= 4) {
+#pragma unroll
+          for (int r = 0; r < RN; r += 4) {
+            const float4 k4 = *reinterpret_cast<const float4*>(kk + i * NP + r);
+            acc[r][0] = fmaf(k4.x, u2.x, acc[r][0]); acc[r][1] = fmaf(k4.x, u2.y, acc[r][1]);
+            acc[r + 1][0] = fmaf(k4.y, u2.x, acc[r + 1][0]); acc[r + 1][1] = fmaf(k4.y, u2.y, acc[r + 1][1]);
+            acc[r + 2][0] = fmaf(k4.z, u2.x, acc[r + 2][0]); acc[r + 2][1] = fmaf(k4.z, u2.y, acc[r + 2][1]);
+            acc[r + 3][0] = fmaf(k4.w, u2.x, acc[r + 3][0]); acc[r + 3][1] = fmaf(k4.w, u2.y, acc[r + 3][1]);
+          }
+        } else {
+          const float2 k2 = *reinterpret_cast<const float2*>(kk + i * NP);
+          acc[0][0] = fmaf(k2.x, u2.x, acc[0][0]); acc[0][1] = fmaf(k2.x, u2.y, acc[0][1]);
+          acc[1][0] = fmaf(k2.y, u2.x, acc[1][0]); acc[1][1] = fmaf(k2.y, u2.y, acc[1][1]);
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < RN; ++r)
+        *reinterpret_cast<float2*>(sP + piece * NP * PS + (r * 16 + tr) * PS + 2 * tp) = make_float2(acc[r][0], acc[r][1]);
+    }
+    __syncthreads();
+    const float keep = ends[kChunk];
+#pragma unroll
+    for (int r = 0; r < OS; ++r) {
+      const int e = tid + 256 * r;
+      float sum = 0.0f;
+#pragma unroll
+      for (int k = 0; k < KS; ++k) sum += sP[k * NP * PS + e];
+      S[r] = fmaf(keep, S[r], sum);
+      sS[state_row(e) * PS + e % PS] = S[r];
+    }
   }
 #pragma unroll
-  for (int r = 0; r < RN; ++r)
-#pragma unroll
-    for (int e = 0; e < 2; ++e)
-      if (n0 + r < N && p0 + e < P) st[(size_t)(n0 + r) * P + p0 + e] = S[r][e];
+  for (int r = 0; r < OS; ++r) {
+    const int e = tid + 256 * r, n = state_row(e), p = e % PS;
+    if (n < N && p < cols) st[(size_t)n * P + p] = S[r];
+  }
 }
 
-// grid (chunks, H * slices of 64 value columns, sequences), 128 threads (8 rows x 4 columns each): the chunk's outputs.
-__global__ void __launch_bounds__(128) chunk_out_kernel(ScanArgs a) {
+// grid (chunks, H * slices of 64 value columns, sequences), 256 threads (4 rows x 4 columns each): the chunk's outputs.
+__global__ void __launch_bounds__(256) chunk_out_kernel(ScanArgs a) {
   pdl_enter();
   extern __shared__ __align__(16) float sm[];
-  __shared__ double L[kChunk];
+  __shared__ float2 L[kChunk];
   const int slices = (a.P + kOutCols - 1) / kOutCols;
   const int chunk = blockIdx.x, h = blockIdx.y / slices, c0 = (blockIdx.y % slices) * kOutCols, seq = blockIdx.z, tid = threadIdx.x;
   const int t0 = a.seq_start[seq] + chunk * kChunk, cnt = min(kChunk, a.seq_start[seq + 1] - t0);
@@ -470,77 +516,82 @@ __global__ void __launch_bounds__(128) chunk_out_kernel(ScanArgs a) {
   float* KT = QT + N * kPad;           // [N][kPad], then the start state [N][64]
   float* AT = KT + N * kPad;           // [64][kPad]: AT[j][i] = e^(L_i - L_j) (q_i . k_j)
   float* V = AT + kChunk * kPad;       // [64][64]: u
-  load_transposed(QT, a.q + (size_t)t0 * a.q_stride + (size_t)g * N, a.q_stride, cnt, N, N);
-  load_transposed(KT, a.k + (size_t)t0 * a.k_stride + (size_t)g * N, a.k_stride, cnt, N, N);
-  const float* u = a.beta != nullptr ? a.out + (size_t)t0 * ((size_t)a.H * P) + (size_t)h * P + c0 : a.v + (size_t)t0 * a.v_stride + (size_t)h * P + c0;
-  const size_t u_stride = a.beta != nullptr ? (size_t)a.H * P : (size_t)a.v_stride;
-  for (int i = tid; i < kChunk * kOutCols; i += 128) {
-    const int r = i / kOutCols, c = i % kOutCols;
-    V[i] = r < cnt && c < cols ? u[(size_t)r * u_stride + c] : 0.0f;
-  }
+  const bool from_out = a.beta != nullptr;
+  const float* u = from_out ? a.out + (size_t)t0 * ((size_t)a.H * P) + (size_t)h * P + c0 : a.v + (size_t)t0 * a.v_stride + (size_t)h * P + c0;
+  copy_tile<256>(V, kOutCols, u, from_out ? (long long)a.H * P : a.v_stride, kChunk, kOutCols, cnt, cols, a.vec);
+  load_transposed<256>(QT, a.q + (size_t)t0 * a.q_stride + (size_t)g * N, a.q_stride, cnt, N);
+  load_transposed<256>(KT, a.k + (size_t)t0 * a.k_stride + (size_t)g * N, a.k_stride, cnt, N);
   if (tid < 32) chunk_log_sums(a, t0, cnt, h, L);
   __syncthreads();
-  const int i0 = (tid >> 4) * 8, j0 = (tid & 15) * 4;      // 8 rows; 4 keys, later 4 columns
+  // a warp takes 16 rows x 32 columns: lanes 4 x 8
+  const int warp = tid >> 5, lane = tid & 31;
+  const int i0 = (warp >> 1) * 16 + (lane >> 3) * 4, j0 = (warp & 1) * 32 + (lane & 7) * 4;      // 4 rows; 4 keys, later 4 columns
+  const int rows_end = (warp >> 1) * 16 + 16;               // keys from here on are behind all rows of the warp
   {
-    float4 lo[4], hi[4];               // [key]: rows i0 .. i0 + 3 and i0 + 4 .. i0 + 7
+    float4 acc[4];                     // [key]: the four rows
 #pragma unroll
-    for (int j = 0; j < 4; ++j) lo[j] = hi[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (j0 <= i0 + 7) {
+    for (int j = 0; j < 4; ++j) acc[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if ((warp & 1) * 32 < rows_end) {
+#pragma unroll 4
       for (int n = 0; n < N; ++n) {
-        const float4 qa = *reinterpret_cast<const float4*>(QT + n * kPad + i0), qb = *reinterpret_cast<const float4*>(QT + n * kPad + i0 + 4);
-        const float4 k4 = *reinterpret_cast<const float4*>(KT + n * kPad + j0);
-        fma4(lo[0], k4.x, qa); fma4(hi[0], k4.x, qb);
-        fma4(lo[1], k4.y, qa); fma4(hi[1], k4.y, qb);
-        fma4(lo[2], k4.z, qa); fma4(hi[2], k4.z, qb);
-        fma4(lo[3], k4.w, qa); fma4(hi[3], k4.w, qb);
+        const float4 q4 = *reinterpret_cast<const float4*>(QT + n * kPad + i0), k4 = *reinterpret_cast<const float4*>(KT + n * kPad + j0);
+        fma4(acc[0], k4.x, q4);
+        fma4(acc[1], k4.y, q4);
+        fma4(acc[2], k4.z, q4);
+        fma4(acc[3], k4.w, q4);
+      }
+      float2 li[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) li[i] = L[i0 + i];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int jj = j0 + j;
+        const float2 lj = L[jj];
+        acc[j].x = i0 >= jj ? acc[j].x * decay_between(li[0], lj) : 0.0f;
+        acc[j].y = i0 + 1 >= jj ? acc[j].y * decay_between(li[1], lj) : 0.0f;
+        acc[j].z = i0 + 2 >= jj ? acc[j].z * decay_between(li[2], lj) : 0.0f;
+        acc[j].w = i0 + 3 >= jj ? acc[j].w * decay_between(li[3], lj) : 0.0f;
       }
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int jj = j0 + j;
-      const double lj = L[jj];
-      float r[8] = {lo[j].x, lo[j].y, lo[j].z, lo[j].w, hi[j].x, hi[j].y, hi[j].z, hi[j].w};
-#pragma unroll
-      for (int i = 0; i < 8; ++i) r[i] = i0 + i >= jj ? r[i] * exp_of(L[i0 + i] - lj) : 0.0f;
-      *reinterpret_cast<float4*>(AT + jj * kPad + i0) = make_float4(r[0], r[1], r[2], r[3]);
-      *reinterpret_cast<float4*>(AT + jj * kPad + i0 + 4) = make_float4(r[4], r[5], r[6], r[7]);
-    }
+    for (int j = 0; j < 4; ++j) *reinterpret_cast<float4*>(AT + (j0 + j) * kPad + i0) = acc[j];
   }
   __syncthreads();                     // the keys have been read: their place takes the start state
-  const float* start = a.starts + ((((size_t)seq * a.chunks + chunk) * a.H + h) * N) * P + c0;
-  for (int i = tid; i < N * kOutCols; i += 128) {
-    const int n = i / kOutCols, c = i % kOutCols;
-    KT[i] = c < cols ? start[(size_t)n * P + c] : 0.0f;
-  }
+  copy_tile<256>(KT, kOutCols, a.starts + ((((size_t)seq * a.chunks + chunk) * a.H + h) * N) * P + c0, P, N, kOutCols, N, cols, a.vec);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
-  float4 o[8];
+  float4 o[4];
 #pragma unroll
-  for (int i = 0; i < 8; ++i) o[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int i = 0; i < 4; ++i) o[i] = make_float4(0.f, 0.f, 0.f, 0.f);
   auto accumulate = [&](const float* rows, const float* cols4) {
-    const float4 ra = *reinterpret_cast<const float4*>(rows), rb = *reinterpret_cast<const float4*>(rows + 4);
-    const float4 v4 = *reinterpret_cast<const float4*>(cols4);
-    fma4(o[0], ra.x, v4); fma4(o[1], ra.y, v4); fma4(o[2], ra.z, v4); fma4(o[3], ra.w, v4);
-    fma4(o[4], rb.x, v4); fma4(o[5], rb.y, v4); fma4(o[6], rb.z, v4); fma4(o[7], rb.w, v4);
+    const float4 r4 = *reinterpret_cast<const float4*>(rows), v4 = *reinterpret_cast<const float4*>(cols4);
+    fma4(o[0], r4.x, v4);
+    fma4(o[1], r4.y, v4);
+    fma4(o[2], r4.z, v4);
+    fma4(o[3], r4.w, v4);
   };
 #pragma unroll 4
   for (int n = 0; n < N; ++n) accumulate(QT + n * kPad + i0, KT + n * kOutCols + j0);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const float f = exp_of(L[i0 + i]);
+  for (int i = 0; i < 4; ++i) {
+    const float f = decay_since_start(L[i0 + i]);
     o[i] = make_float4(o[i].x * f, o[i].y * f, o[i].z * f, o[i].w * f);
   }
 #pragma unroll 4
-  for (int j = 0; j < i0 + 8; ++j) accumulate(AT + j * kPad + i0, V + j * kOutCols + j0);
+  for (int j = 0; j < rows_end; ++j) accumulate(AT + j * kPad + i0, V + j * kOutCols + j0);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
+  for (int i = 0; i < 4; ++i) {
     if (i0 + i >= cnt) continue;
     float* dst = a.out + (size_t)(t0 + i0 + i) * ((size_t)a.H * P) + (size_t)h * P + c0 + j0;
     const float r[4] = {o[i].x * a.q_scale, o[i].y * a.q_scale, o[i].z * a.q_scale, o[i].w * a.q_scale};
-    if (a.vec && j0 + 3 < cols) *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
-    else
+    if (a.vec && j0 + 3 < cols) {
+      *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
+    } else {
 #pragma unroll
       for (int e = 0; e < 4; ++e)
         if (j0 + e < cols) dst[e] = r[e];
+    }
   }
 }
 
@@ -686,23 +737,25 @@ static bool runs_in_chunks(int max_count, int N) { return max_count > kWalkToken
 extern "C" long long slb_state_scan_scratch_floats(int n_seqs, int max_count, int H, int N, int P, int delta) {
   if (!runs_in_chunks(max_count, N)) return 0;
   const long long chunks = (max_count + kChunk - 1) / kChunk;
-  return (long long)n_seqs * chunks * H * N * ((delta ? kChunk : 0) + (long long)P);
+  const long long starts = (((long long)n_seqs * chunks * H * N * P) + 3) & ~3ll;
+  return starts + (delta ? (long long)n_seqs * chunks * H * ((long long)N * kChunk + kChunk + 4) : 0);
 }
 
-template <int RN>
-static int launch_chunk_state(const ScanArgs& a, dim3 grid, cudaStream_t s) {
+template <int RN, int PS>
+static int launch_chunk_state(const ScanArgs& a, cudaStream_t s) {
+  const dim3 grid((a.P + PS - 1) / PS, a.H, a.n_seqs), block(256);
   const bool delta = a.beta != nullptr;
-  const int NP = 16 * RN;
-  const int smem = (NP * kSlice + kChunk * kSlice + (delta ? 4 : 2) * kChunk * NP) * 4;
+  constexpr int NP = 16 * RN, KS = 32 / PS;
+  const int smem = (NP * PS + kChunk * PS + KS * (NP > kChunk ? NP : kChunk) * PS + 2 * (kChunk + 4) + (delta ? 4 : 2) * kChunk * NP) * 4;
   static bool configured[2] = {false, false};
   if (!configured[delta]) {
-    const cudaError_t e = delta ? cudaFuncSetAttribute(chunk_state_kernel<RN, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)
-                                : cudaFuncSetAttribute(chunk_state_kernel<RN, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    const cudaError_t e = delta ? cudaFuncSetAttribute(chunk_state_kernel<RN, PS, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)
+                                : cudaFuncSetAttribute(chunk_state_kernel<RN, PS, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return fail(2, "state_scan: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));
     configured[delta] = true;
   }
-  if (delta) launch(chunk_state_kernel<RN, true>, grid, dim3(128), (size_t)smem, s, a);
-  else launch(chunk_state_kernel<RN, false>, grid, dim3(128), (size_t)smem, s, a);
+  if (delta) launch(chunk_state_kernel<RN, PS, true>, grid, block, (size_t)smem, s, a);
+  else launch(chunk_state_kernel<RN, PS, false>, grid, block, (size_t)smem, s, a);
   return check_launch("state_scan (states)");
 }
 
@@ -712,10 +765,10 @@ extern "C" int slb_state_scan(const float* q, long long q_stride, const float* k
                               float* scratch, long long scratch_floats, void* stream) {
   SLB_REQUIRE(n_seqs >= 0 && n_seqs < 65536 && H > 0 && G > 0 && H % G == 0 && N > 0 && N <= 256 && P > 0,
               "state_scan: heads=%d groups=%d N=%d (at most 256) P=%d", H, G, N, P);
-  SLB_REQUIRE(decay_stride == 0 || decay_stride >= H, "state_scan: decay rows of %lld values for %d heads", decay_stride, H);
+  SLB_REQUIRE(decay_stride == 0 || (beta != nullptr && decay_stride >= H), "state_scan: decay rows of %lld values for %d heads", decay_stride, H);
   if (n_seqs == 0 || max_count <= 0) return 0;
   ScanArgs a{q, k, v, q_stride, k_stride, v_stride, log_decay, decay_stride, beta, state, slots, seq_start, out, n_seqs, H, G, N, P, q_scale,
-             0, nullptr, nullptr, 0};
+             0, nullptr, nullptr, nullptr, 0};
   cudaStream_t s = (cudaStream_t)stream;
   const bool delta = beta != nullptr;
   const long long need = slb_state_scan_scratch_floats(n_seqs, max_count, H, N, P, delta);
@@ -730,14 +783,16 @@ extern "C" int slb_state_scan(const float* q, long long q_stride, const float* k
   }
   SLB_REQUIRE(scratch != nullptr && scratch_floats >= need, "state_scan: %lld floats of scratch memory are needed, %lld were given", need, scratch_floats);
   a.chunks = (max_count + kChunk - 1) / kChunk;
+  const size_t per = (size_t)n_seqs * a.chunks * H;
   a.w = scratch;
-  a.starts = scratch + (delta ? (size_t)n_seqs * a.chunks * H * N * kChunk : 0);
+  a.ends = a.w + (delta ? per * N * kChunk : 0);
+  a.starts = a.ends + (delta ? per * (kChunk + 4) : 0);
   a.vec = N % 4 == 0 && P % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && v_stride % 4 == 0 &&
           ((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)out | (uintptr_t)scratch) % 16 == 0;
   SLB_REQUIRE((uintptr_t)scratch % 16 == 0, "state_scan: the scratch memory must be 16-byte aligned");
   SLB_REQUIRE(H < 65536 && (long long)H * ((P + kOutCols - 1) / kOutCols) < 65536, "state_scan: too many heads (%d)", H);
   if (delta) {
-    const int smem = (N * kPad + kChunk * kPad + kChunk * 128) * 4;
+    const int smem = (N * kPad + kChunk * kPad) * 4;
     static int most = 0;
     if (smem > most) {
       const cudaError_t e = cudaFuncSetAttribute(chunk_solve_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -749,8 +804,12 @@ extern "C" int slb_state_scan(const float* q, long long q_stride, const float* k
     if (rc) return rc;
   }
   {
-    const dim3 grid((P + kSlice - 1) / kSlice, H, n_seqs);
-    const int rc = N <= 32 ? launch_chunk_state<2>(a, grid, s) : (N <= 64 ? launch_chunk_state<4>(a, grid, s) : launch_chunk_state<8>(a, grid, s));
+    // slices of 8 columns while all their blocks can be resident at once, else of 16 (with 128 rows one block fits an SM)
+    const bool narrow = (long long)((P + 7) / 8) * H * n_seqs <= (long long)sm_count() * (N <= 64 ? 2 : 1);
+    int rc;
+    if (N <= 32) rc = narrow ? launch_chunk_state<2, 8>(a, s) : launch_chunk_state<2, 16>(a, s);
+    else if (N <= 64) rc = narrow ? launch_chunk_state<4, 8>(a, s) : launch_chunk_state<4, 16>(a, s);
+    else rc = narrow ? launch_chunk_state<8, 8>(a, s) : launch_chunk_state<8, 16>(a, s);
     if (rc) return rc;
   }
   const int smem = (2 * N * kPad + kChunk * kPad + kChunk * kOutCols) * 4;
@@ -760,7 +819,7 @@ extern "C" int slb_state_scan(const float* q, long long q_stride, const float* k
     if (e != cudaSuccess) return fail(2, "state_scan: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));
     most_out = smem;
   }
-  launch(chunk_out_kernel, dim3(a.chunks, H * ((P + kOutCols - 1) / kOutCols), n_seqs), dim3(128), (size_t)smem, s, a);
+  launch(chunk_out_kernel, dim3(a.chunks, H * ((P + kOutCols - 1) / kOutCols), n_seqs), dim3(256), (size_t)smem, s, a);
   return check_launch("state_scan (outputs)");
 }
 

@@ -240,6 +240,28 @@ __global__ void __launch_bounds__(256) sigmoid_gate_kernel(T* __restrict__ y, co
   y[i] = from_f32<T>(to_f32(y[i]) / (1.0f + expf(-gate[(size_t)t * gate_stride + c])));
 }
 
+// Eight channels a thread (bfloat16, widths and row strides that are multiples of 8 and 4): 16-byte loads and stores.
+__global__ void __launch_bounds__(256) sigmoid_gate_vec_kernel(__nv_bfloat16* __restrict__ y, const float* __restrict__ gate,
+                                                               long long gate_stride, long long pieces, int per_row) {
+  pdl_enter();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= pieces) return;
+  const long long t = i / per_row;
+  const int c = (int)(i - t * per_row) * 8;
+  const float4* g = reinterpret_cast<const float4*>(gate + (size_t)t * gate_stride + c);
+  const float4 ga = g[0], gb = g[1];
+  Bf16x8* p = reinterpret_cast<Bf16x8*>(y) + i;
+  float f[8];
+  unpack8(*p, f);
+  const float z[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
+#pragma unroll
+  for (int k = 0; k < 8; ++k) f[k] = f[k] / (1.0f + expf(-z[k]));
+  Bf16x8 r;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) r.v[k] = __floats2bfloat162_rn(f[2 * k], f[2 * k + 1]);
+  *p = r;
+}
+
 }  // namespace slb
 
 using namespace slb;
@@ -326,6 +348,10 @@ extern "C" int slb_sigmoid_gate(void* y, const float* gate, long long gate_strid
   SLB_REQUIRE(rows >= 0 && C > 0 && gate_stride >= C, "sigmoid_gate: rows=%lld channels=%d", rows, C);
   if (rows == 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == kBF16 && C % 8 == 0 && gate_stride % 4 == 0 && ((uintptr_t)y | (uintptr_t)gate) % 16 == 0) {
+    launch(sigmoid_gate_vec_kernel, per_element(rows * (C / 8)), dim3(256), 0, s, (__nv_bfloat16*)y, gate, gate_stride, rows * (C / 8), C / 8);
+    return check_launch("sigmoid_gate");
+  }
   if (dtype == kF32) launch(sigmoid_gate_kernel<float>, per_element(rows * C), dim3(256), 0, s, (float*)y, gate, gate_stride, rows, C);
   else if (dtype == kBF16) launch(sigmoid_gate_kernel<__nv_bfloat16>, per_element(rows * C), dim3(256), 0, s, (__nv_bfloat16*)y, gate, gate_stride, rows, C);
   else return fail(1, "sigmoid_gate: unknown dtype %d", dtype);

@@ -4,6 +4,7 @@
 //
 //   causal_conv_kernel      y_t[c] = sum_j w[c, j] * u_(t - taps + 1 + j)[c] (+ bias, then silu): inputs before the step's
 //                           first token come from the sequence's state (its last taps - 1 inputs), zeros at its start
+//                           (causal_conv_tile_kernel: the same for prompts; causal_conv_short_kernel: for few tokens a sequence)
 //   conv_state_kernel       the state after the step: the sequence's last taps - 1 inputs
 //   decay_scan_kernel       S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head; a_t one factor per key channel
 //                           or one per head; v may carry a factor per (token, head)
@@ -11,6 +12,7 @@
 //   channel_decay_kernel    a = sigmoid(z + bias)^(1 / tau) = exp(-softplus(-(z + bias)) / tau)
 //   gated_group_norm_kernel rows cut into equal groups, each divided by its root mean square, times a gain, with a
 //                           silu gate in front of or behind the norm and an optional skip term D_h * x
+//                           (gated_head_norm_kernel: one warp a group, for groups of up to 256 channels gated behind the norm)
 #include <math.h>
 
 #include "common.cuh"
@@ -43,6 +45,82 @@ __global__ void __launch_bounds__(256) causal_conv_kernel(const float* __restric
     acc = fmaf(w[(size_t)c * taps + j], u, acc);
   }
   out[(size_t)t * out_stride + c] = act ? silu_f(acc) : acc;
+}
+
+// The same for steps of many tokens and up to four taps: a thread takes four (VEC) neighbouring channels, or one, and walks
+// kConvTile tokens with the last inputs in registers, so every input is read once; eight tokens' loads are under way before the
+// first is used. Where the tile crosses into another sequence the window is filled from that sequence's state.
+constexpr int kConvTile = 32;
+
+template <int TAPS, int VEC>
+__global__ void __launch_bounds__(128) causal_conv_tile_kernel(const float* __restrict__ in, long long in_stride,
+                                                               const float* __restrict__ w, const float* __restrict__ bias,
+                                                               const float* __restrict__ state, const int* __restrict__ slots,
+                                                               const int* __restrict__ tok_seq, const int* __restrict__ seq_start,
+                                                               float* __restrict__ out, long long out_stride, int tokens, int C,
+                                                               int act) {
+  pdl_enter();
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+  if (c >= C) return;
+  const int t0 = blockIdx.y * kConvTile, t1 = min(tokens, t0 + kConvTile);
+  float wt[VEC][TAPS], bs[VEC], win[TAPS - 1][VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) {
+    bs[e] = bias ? bias[c + e] : 0.0f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wt[e][j] = w[(size_t)(c + e) * TAPS + j];
+  }
+  auto load = [&](const float* p, float (&v)[VEC]) {
+    if constexpr (VEC == 4) {
+      const float4 q = *reinterpret_cast<const float4*>(p);
+      v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+    } else {
+      v[0] = *p;
+    }
+  };
+  int seq = tok_seq[t0];
+  // the window in front of token t of sequence s: the step's own inputs as far as they reach, then the state's
+  auto refill = [&](int t) {
+    const int at = t - seq_start[seq];
+    const float* st = state + ((size_t)slots[seq] * (TAPS - 1)) * C + c;
+#pragma unroll
+    for (int k = 0; k < TAPS - 1; ++k) {
+      const int src = at - (TAPS - 1) + k;
+      load(src >= 0 ? in + (size_t)(t - (TAPS - 1) + k) * in_stride + c : st + (size_t)(TAPS - 1 + src) * C, win[k]);
+    }
+  };
+  refill(t0);
+  for (int tb = t0; tb < t1; tb += 8) {
+    float u[8][VEC];
+    int sq[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const int t = min(tb + k, t1 - 1);
+      load(in + (size_t)t * in_stride + c, u[k]);
+      sq[k] = tok_seq[t];
+    }
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const int t = tb + k;
+      if (t >= t1) break;
+      if (sq[k] != seq) { seq = sq[k]; refill(t); }
+      float y[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        float acc = bs[e];
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(wt[e][j], win[j][e], acc);
+        acc = fmaf(wt[e][TAPS - 1], u[k][e], acc);
+        y[e] = act ? silu_f(acc) : acc;
+#pragma unroll
+        for (int j = 0; j < TAPS - 2; ++j) win[j][e] = win[j + 1][e];
+        win[TAPS - 2][e] = u[k][e];
+      }
+      float* dst = out + (size_t)t * out_stride + c;
+      if constexpr (VEC == 4) *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+      else *dst = y[0];
+    }
+  }
 }
 
 // One thread per (sequence, channel): the last taps - 1 inputs of the sequence, old ones kept where the step was short.
@@ -331,6 +409,82 @@ __global__ void __launch_bounds__(128) gated_group_norm_kernel(GroupNormArgs a) 
   }
 }
 
+// Groups of up to 256 channels without skip term and with the gate behind the norm (recurrences' heads): one warp per (token,
+// group), the group's values in registers between the sum of squares and the store. VEC neighbouring channels a lane and load.
+template <typename T, int VEC, int PER>
+__global__ void __launch_bounds__(256) gated_head_norm_kernel(GroupNormArgs a) {
+  pdl_enter();
+  const int lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (item >= (long long)a.tokens * a.groups) return;
+  const int t = (int)(item / a.groups), grp = (int)(item - (long long)t * a.groups);
+  const int width = a.inner / a.groups, c0 = grp * width;
+  const float* y = a.y + (size_t)t * a.inner + c0;
+  const float* gate = a.gate + (size_t)t * a.gate_stride + c0;
+  T* out = (T*)a.out + (size_t)t * a.inner + c0;
+  float v[PER][VEC], g[PER][VEC];
+  float ss = 0.0f;
+#pragma unroll
+  for (int k = 0; k < PER; ++k) {
+    const int c = (lane + 32 * k) * VEC;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[k][e] = g[k][e] = 0.0f;
+    if (c < width) {
+      if constexpr (VEC == 4) {
+        const float4 p = *reinterpret_cast<const float4*>(y + c), q = *reinterpret_cast<const float4*>(gate + c);
+        v[k][0] = p.x; v[k][1] = p.y; v[k][2] = p.z; v[k][3] = p.w;
+        g[k][0] = q.x; g[k][1] = q.y; g[k][2] = q.z; g[k][3] = q.w;
+      } else if constexpr (VEC == 2) {
+        const float2 p = *reinterpret_cast<const float2*>(y + c), q = *reinterpret_cast<const float2*>(gate + c);
+        v[k][0] = p.x; v[k][1] = p.y;
+        g[k][0] = q.x; g[k][1] = q.y;
+      } else {
+        v[k][0] = y[c];
+        g[k][0] = gate[c];
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(v[k][e], v[k][e], ss);
+  }
+  const float r = 1.0f / sqrtf(warp_sum(ss) / (float)width + a.eps);
+#pragma unroll
+  for (int k = 0; k < PER; ++k) {
+    const int c = (lane + 32 * k) * VEC;
+    if (c >= width) continue;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      float x = v[k][e] * r;
+      if (a.gain) x *= a.gain[(c0 + c + e) % a.gain_len];
+      v[k][e] = x * silu_f(g[k][e]);
+    }
+    if constexpr (VEC >= 2 && sizeof(T) == 2) {
+#pragma unroll
+      for (int e = 0; e < VEC; e += 2) *reinterpret_cast<__nv_bfloat162*>(out + c + e) = __floats2bfloat162_rn(v[k][e], v[k][e + 1]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) out[c + e] = from_f32<T>(v[k][e]);
+    }
+  }
+}
+
+template <typename T>
+static bool launch_head_norm(const GroupNormArgs& a, cudaStream_t s) {
+  const int width = a.inner / a.groups;
+  if (a.gate_first || a.skip || width > 256) return false;
+  const long long warps = (long long)a.tokens * a.groups;
+  const dim3 grid((unsigned)((warps + 7) / 8)), block(256);
+  const bool aligned = ((uintptr_t)a.y | (uintptr_t)a.gate | (uintptr_t)a.out) % 16 == 0 && a.inner % 4 == 0 && a.gate_stride % 4 == 0;
+  if (aligned && width % 4 == 0 && width > 64) {
+    if (width <= 128) launch(gated_head_norm_kernel<T, 4, 1>, grid, block, 0, s, a);
+    else launch(gated_head_norm_kernel<T, 4, 2>, grid, block, 0, s, a);
+  } else if (aligned && width % 2 == 0 && width <= 64) {
+    launch(gated_head_norm_kernel<T, 2, 1>, grid, block, 0, s, a);
+  } else {
+    launch(gated_head_norm_kernel<T, 1, 8>, grid, block, 0, s, a);
+  }
+  return true;
+}
+
 }  // namespace slb
 
 using namespace slb;
@@ -350,8 +504,20 @@ extern "C" int slb_causal_conv(const float* in, long long in_stride, const float
     return check_launch("causal_conv (short steps)");
   }
   const long long total = (long long)tokens * C;
-  launch(causal_conv_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, in, in_stride, w, bias,
-         (const float*)state, slots, tok_seq, seq_start, out, out_stride, tokens, C, taps, act);
+  if (taps >= 2 && taps <= 4 && tokens >= 64 && tokens / kConvTile < 65535) {
+    const bool vec = C % 4 == 0 && in_stride % 4 == 0 && out_stride % 4 == 0 && ((uintptr_t)in | (uintptr_t)out | (uintptr_t)state) % 16 == 0;
+    const dim3 grid((C / (vec ? 4 : 1) + 127) / 128, (tokens + kConvTile - 1) / kConvTile), block(128);
+    const float* st = state;
+    if (taps == 2 && vec) launch(causal_conv_tile_kernel<2, 4>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
+    else if (taps == 2) launch(causal_conv_tile_kernel<2, 1>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
+    else if (taps == 3 && vec) launch(causal_conv_tile_kernel<3, 4>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
+    else if (taps == 3) launch(causal_conv_tile_kernel<3, 1>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
+    else if (vec) launch(causal_conv_tile_kernel<4, 4>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
+    else launch(causal_conv_tile_kernel<4, 1>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
+  } else {
+    launch(causal_conv_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, in, in_stride, w, bias,
+           (const float*)state, slots, tok_seq, seq_start, out, out_stride, tokens, C, taps, act);
+  }
   int rc = check_launch("causal_conv");
   if (rc || taps == 1) return rc;
   const long long st = (long long)n_seqs * C;
@@ -478,6 +644,8 @@ extern "C" int slb_gated_group_norm(const float* y, const float* skip, long long
                   gate_first, eps};
   const dim3 grid((unsigned)(tokens * groups)), block(128);
   cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == kF32 && launch_head_norm<float>(a, s)) return check_launch("gated_group_norm");
+  if (dtype == kBF16 && launch_head_norm<__nv_bfloat16>(a, s)) return check_launch("gated_group_norm");
   if (dtype == kF32) launch(gated_group_norm_kernel<float>, grid, block, 0, s, a);
   else if (dtype == kBF16) launch(gated_group_norm_kernel<__nv_bfloat16>, grid, block, 0, s, a);
   else return fail(1, "gated_group_norm: unknown dtype %d", dtype);
