@@ -182,9 +182,7 @@ __device__ __forceinline__ float decay_since_start(const float2& to) { return ex
 // A [64, N] tile of rows transposed into shared memory, dst[n][i]; rows from cnt on are zero.
 template <int THREADS>
 __device__ __forceinline__ void load_transposed(float* dst, const float* src, long long stride, int cnt, int N) {
-  int n = threadIdx.x, i = 0;
-  while (n >= N) { n -= N; i += 4; }
-  for (; i < kChunk;) {
+  auto quad = [&](int n, int i) {
     const float* p = src + (size_t)i * stride + n;
     float4 v;
     v.x = i < cnt ? p[0] : 0.0f;
@@ -192,8 +190,13 @@ __device__ __forceinline__ void load_transposed(float* dst, const float* src, lo
     v.z = i + 2 < cnt ? p[2 * stride] : 0.0f;
     v.w = i + 3 < cnt ? p[3 * stride] : 0.0f;
     *reinterpret_cast<float4*>(dst + n * kPad + i) = v;
-    n += THREADS;
-    while (n >= N) { n -= N; i += 4; }
+  };
+  if (N == 64 || N == 128) {           // the usual widths: shifts instead of divisions
+    const int sh = N == 64 ? 6 : 7, n = threadIdx.x & (N - 1);
+#pragma unroll 4
+    for (int i = (threadIdx.x >> sh) * 4; i < kChunk; i += (THREADS >> sh) * 4) quad(n, i);
+  } else {
+    for (int idx = threadIdx.x; idx < N * (kChunk / 4); idx += THREADS) quad(idx % N, idx / N * 4);
   }
 }
 
@@ -210,17 +213,26 @@ __device__ __forceinline__ void copy_async(float* dst, const float* src, bool va
   else asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(d), "l"(src), "r"(valid ? 4 : 0) : "memory");
 }
 
-// `rows` rows of `cols` floats into shared memory (row length `ld`); rows from `valid` on and columns from `live` on become zero.
-template <int THREADS>
-__device__ __forceinline__ void copy_tile(float* dst, int ld, const float* src, long long stride, int rows, int cols, int valid, int live, bool vec) {
-  const int step = vec ? 4 : 1, per = cols / step;         // vec: cols, live and the addresses are multiples of 4 floats
-  int c = threadIdx.x, r = 0;
-  while (c >= per) { c -= per; ++r; }
-  while (r < rows) {
-    const bool in = r < valid && c * step < live;
-    copy_async(dst + r * ld + c * step, src + (in ? (size_t)r * stride + c * step : 0), in, vec);
-    c += THREADS;
-    while (c >= per) { c -= per; ++r; }
+// ROWS rows of COLS floats into shared memory; rows from `valid` on and columns from `live` on become zero. vec: `live` and the
+// source's addresses are multiples of 4 floats.
+template <int THREADS, int ROWS, int COLS>
+__device__ __forceinline__ void copy_tile(float* dst, const float* src, long long stride, int valid, int live, bool vec) {
+  if (vec) {
+    constexpr int per = COLS / 4;
+    const int c = (threadIdx.x % per) * 4;
+    const float* p = src + c + (long long)(threadIdx.x / per) * stride;
+#pragma unroll
+    for (int m = 0; m < ROWS * per / THREADS; ++m) {
+      const int r = threadIdx.x / per + m * (THREADS / per);
+      const bool in = r < valid && c < live;
+      copy_async(dst + r * COLS + c, in ? p + (long long)m * (THREADS / per) * stride : src, in, true);
+    }
+  } else {
+    const int c = threadIdx.x % COLS;
+    for (int r = threadIdx.x / COLS; r < ROWS; r += THREADS / COLS) {
+      const bool in = r < valid && c < live;
+      copy_async(dst + r * COLS + c, in ? src + (long long)r * stride + c : src, in, false);
+    }
   }
 }
 
@@ -381,12 +393,16 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
   auto fetch = [&](int c) {            // one commit group a chunk
     if (c < live) {
       const int cnt = min(kChunk, total - c * kChunk), b = c & 1;
-      copy_tile<256>(sK + b * kChunk * NP, NP, a.k + (size_t)(first + c * kChunk) * a.k_stride + (size_t)g * N, a.k_stride, kChunk, NP, cnt, N, a.vec);
+      copy_tile<256, kChunk, NP>(sK + b * kChunk * NP, a.k + (size_t)(first + c * kChunk) * a.k_stride + (size_t)g * N, a.k_stride, cnt, N, a.vec);
       if (DELTA) {
         const size_t at = ((size_t)seq * a.chunks + c) * a.H + h;
         float* wd = sW + b * NP * kChunk;
         const float* ws = a.w + at * N * kChunk;
-        for (int i = tid; i < N * (kChunk / 4); i += 256) copy_async(wd + i * 4, ws + i * 4, true, true);
+#pragma unroll
+        for (int m = 0; m < NP / 16; ++m) {
+          const int i = (tid + m * 256) * 4;
+          if (i < N * kChunk) copy_async(wd + i, ws + i, true, true);
+        }
         if (tid < kChunk / 4 + 1) copy_async(sE + b * (kChunk + 4) + tid * 4, a.ends + at * (kChunk + 4) + tid * 4, true, true);
       } else if (tid <= kChunk) {      // a fixed decay: its powers
         const float left = tid == kChunk ? (float)cnt : (float)(cnt - 1 - tid);
@@ -502,6 +518,10 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
   }
 }
 
+__host__ __device__ constexpr int out_keys_floats(int N) {
+  return N * kPad > (N + 15) / 16 * 16 * kOutCols ? N * kPad : (N + 15) / 16 * 16 * kOutCols;
+}
+
 // grid (chunks, H * slices of 64 value columns, sequences), 256 threads (4 rows x 4 columns each): the chunk's outputs.
 __global__ void __launch_bounds__(256) chunk_out_kernel(ScanArgs a) {
   pdl_enter();
@@ -513,12 +533,12 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(ScanArgs a) {
   if (cnt <= 0) return;
   const int N = a.N, P = a.P, g = h / (a.H / a.G), cols = min(kOutCols, P - c0);
   float* QT = sm;                      // [N][kPad]
-  float* KT = QT + N * kPad;           // [N][kPad], then the start state [N][64]
-  float* AT = KT + N * kPad;           // [64][kPad]: AT[j][i] = e^(L_i - L_j) (q_i . k_j)
+  float* KT = QT + N * kPad;           // [N][kPad], then the start state [N rounded up to 16][64]
+  float* AT = KT + out_keys_floats(N); // [64][kPad]: AT[j][i] = e^(L_i - L_j) (q_i . k_j)
   float* V = AT + kChunk * kPad;       // [64][64]: u
   const bool from_out = a.beta != nullptr;
   const float* u = from_out ? a.out + (size_t)t0 * ((size_t)a.H * P) + (size_t)h * P + c0 : a.v + (size_t)t0 * a.v_stride + (size_t)h * P + c0;
-  copy_tile<256>(V, kOutCols, u, from_out ? (long long)a.H * P : a.v_stride, kChunk, kOutCols, cnt, cols, a.vec);
+  copy_tile<256, kChunk, kOutCols>(V, u, from_out ? (long long)a.H * P : a.v_stride, cnt, cols, a.vec);
   load_transposed<256>(QT, a.q + (size_t)t0 * a.q_stride + (size_t)g * N, a.q_stride, cnt, N);
   load_transposed<256>(KT, a.k + (size_t)t0 * a.k_stride + (size_t)g * N, a.k_stride, cnt, N);
   if (tid < 32) chunk_log_sums(a, t0, cnt, h, L);
@@ -557,7 +577,8 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(ScanArgs a) {
     for (int j = 0; j < 4; ++j) *reinterpret_cast<float4*>(AT + (j0 + j) * kPad + i0) = acc[j];
   }
   __syncthreads();                     // the keys have been read: their place takes the start state
-  copy_tile<256>(KT, kOutCols, a.starts + ((((size_t)seq * a.chunks + chunk) * a.H + h) * N) * P + c0, P, N, kOutCols, N, cols, a.vec);
+  const float* start = a.starts + ((((size_t)seq * a.chunks + chunk) * a.H + h) * N) * P + c0;
+  for (int n = 0; n < N; n += 16) copy_tile<256, 16, kOutCols>(KT + n * kOutCols, start + (size_t)n * P, P, N - n, cols, a.vec);
   asm volatile("cp.async.commit_group;" ::: "memory");
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
@@ -812,7 +833,7 @@ extern "C" int slb_state_scan(const float* q, long long q_stride, const float* k
     else rc = narrow ? launch_chunk_state<8, 8>(a, s) : launch_chunk_state<8, 16>(a, s);
     if (rc) return rc;
   }
-  const int smem = (2 * N * kPad + kChunk * kPad + kChunk * kOutCols) * 4;
+  const int smem = (N * kPad + out_keys_floats(N) + kChunk * kPad + kChunk * kOutCols) * 4;
   static int most_out = 0;
   if (smem > most_out) {
     const cudaError_t e = cudaFuncSetAttribute(chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
