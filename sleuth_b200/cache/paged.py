@@ -3,7 +3,8 @@
 Each layer application has one cache *entry*. A part asks for what its entry needs through a request:
 
 * ``KVRequest(kv_heads, head_dim, window)``: keys and values of every position (or of the last
-  ``window`` positions, or, with a negative window, of the current chunk of ``-window`` positions). Entries with equal requests form a *group*; a group owns one tensor
+  ``window`` positions, or, with a negative window, of the current chunk of ``-window``
+  positions). Entries with equal requests form a *group*; a group owns one tensor
   ``[entries, 2, pages, kv_heads, 64, head_dim]`` (index 1: 0 = keys, 1 = values), so a page number
   means the same place in every entry of the group and one block table serves them all. With values of another
   width than the keys (``value_dim``) an entry is one flat run instead: all key pages ``[pages, kv_heads, 64,

@@ -61,6 +61,8 @@ struct FlashArgs {
   float softcap_log2;           // cap * log2(e), or 0
   const float* slopes;          // [H] or null
   int out_f32;                  // `out` is float32 [tokens, H * HD] instead of bfloat16
+  const float* gate;            // decode: null, or float32 pre-activations; the result is multiplied by sigmoid(gate[t * gate_stride + h * HD + d])
+  long long gate_stride;
 };
 
 constexpr float kLog2e = 1.4426950408889634f;
@@ -598,8 +600,9 @@ __global__ void __launch_bounds__(kFlashThreads) attn_decode_kernel(FlashArgs a)
     const int head = head0 + row;
     if (a.splits == 1) {
       if (a.sinks) l += exp2f(a.sinks[head] * kLog2e - m_use);
-      if (a.out_f32) reinterpret_cast<float*>(a.out)[((size_t)tok * a.heads + head) * HD + d] = acc / l;
-      else a.out[((size_t)tok * a.heads + head) * HD + d] = __float2bfloat16_rn(acc / l);
+      const float v = acc / l * (a.gate ? 1.0f / (1.0f + expf(-a.gate[(size_t)tok * a.gate_stride + (size_t)head * HD + d])) : 1.0f);
+      if (a.out_f32) reinterpret_cast<float*>(a.out)[((size_t)tok * a.heads + head) * HD + d] = v;
+      else a.out[((size_t)tok * a.heads + head) * HD + d] = __float2bfloat16_rn(v);
     } else {
       const size_t pi = ((size_t)seq * a.heads + head) * a.splits + split;
       a.part_o[pi * HD + d] = acc;
@@ -656,8 +659,9 @@ __global__ void __launch_bounds__(kFlashThreads) attn_decode_kernel(FlashArgs a)
       m = m_new;
     }
     if (a.sinks) l += exp2f(a.sinks[head] * kLog2e - m);
-    if (a.out_f32) reinterpret_cast<float*>(a.out)[((size_t)tok * a.heads + head) * HD + d] = acc / l;
-    else a.out[((size_t)tok * a.heads + head) * HD + d] = __float2bfloat16_rn(acc / l);
+    const float v = acc / l * (a.gate ? 1.0f / (1.0f + expf(-a.gate[(size_t)tok * a.gate_stride + (size_t)head * HD + d])) : 1.0f);
+    if (a.out_f32) reinterpret_cast<float*>(a.out)[((size_t)tok * a.heads + head) * HD + d] = v;
+    else a.out[((size_t)tok * a.heads + head) * HD + d] = __float2bfloat16_rn(v);
   }
   if (tid == 0) *counter = 0;
 }
@@ -773,7 +777,8 @@ static int attention_decode_any(const void* q, const void* k_pool, const void* v
                                 long long n_counters, const void* qkv, int qkv_kv_heads, const float* bias,
                                 const float* q_gain, const float* k_gain, const float* cos_table,
                                 const float* sin_table, float eps, const void* next, long long next_bytes,
-                                const float* sinks, const float* slopes, float softcap, int out_f32, void* stream) {
+                                const float* sinks, const float* slopes, float softcap, int out_f32, const float* gate,
+                                long long gate_stride, void* stream) {
   // qkv != null: `q` is ignored; the kernel takes the new token's raw projection rows [n, (H + 2 * qkv_kv_heads) * hd],
   // applies bias, QK-norm and the rotation itself, and (qkv_kv_heads == kv_heads) writes the token's key and value
   // into the cache. cos/sin tables, if given, are [positions, hd / 2]: the whole head rotates.
@@ -805,6 +810,8 @@ static int attention_decode_any(const void* q, const void* k_pool, const void* v
   a.qkv = (const __nv_bfloat16*)qkv; a.qkv_kv_heads = qkv_kv_heads; a.bias = bias; a.q_gain = q_gain; a.k_gain = k_gain;
   a.cos_table = cos_table; a.sin_table = sin_table; a.eps = eps; a.sinks = sinks;
   a.slopes = slopes; a.softcap_log2 = softcap > 0.0f ? softcap * 1.4426950408889634f : 0.0f; a.out_f32 = out_f32;
+  SLB_REQUIRE(gate == nullptr || gate_stride >= (long long)heads * head_dim, "attention (decode): gate rows are too short");
+  a.gate = gate; a.gate_stride = gate_stride;
   a.pages_after_wait = (qkv == nullptr || qkv_kv_heads == 0 || pdl_mode() == 1) ? 1 : 0;
   SLB_REQUIRE(next_bytes >= 0 && (uintptr_t)next % 16 == 0, "attention (decode): the range to prefetch must be 16-byte aligned");
   a.next.ptr = (const char*)next; a.next.bytes = next ? next_bytes : 0;
@@ -819,10 +826,10 @@ extern "C" int slb_attention_decode(const void* q, const void* k_pool, const voi
                                     long long n_counters, const void* qkv, int qkv_kv_heads, const float* bias,
                                     const float* q_gain, const float* k_gain, const float* cos_table,
                                     const float* sin_table, float eps, const void* next, long long next_bytes,
-                                    const float* sinks, void* stream) {
+                                    const float* sinks, const float* gate, long long gate_stride, void* stream) {
   return attention_decode_any(q, k_pool, v_pool, out, seq_start, past, block_table, table_stride, n_seqs, heads, kv_heads, head_dim,
                               window, scale, splits, scratch, scratch_floats, counters, n_counters, qkv, qkv_kv_heads, bias, q_gain,
-                              k_gain, cos_table, sin_table, eps, next, next_bytes, sinks, nullptr, 0.0f, 0, stream);
+                              k_gain, cos_table, sin_table, eps, next, next_bytes, sinks, nullptr, 0.0f, 0, gate, gate_stride, stream);
 }
 
 // One token a sequence with post-processed queries, a distance penalty per head (`slopes` or null) and a soft cap (0 = none).
@@ -834,5 +841,5 @@ extern "C" int slb_attention_decode_scored(const void* q, const void* k_pool, co
                                            float softcap, int out_f32, void* stream) {
   return attention_decode_any(q, k_pool, v_pool, out, seq_start, past, block_table, table_stride, n_seqs, heads, kv_heads, head_dim,
                               window, scale, splits, scratch, scratch_floats, counters, n_counters, nullptr, 0, nullptr, nullptr,
-                              nullptr, nullptr, nullptr, 0.0f, next, next_bytes, nullptr, slopes, softcap, out_f32, stream);
+                              nullptr, nullptr, nullptr, 0.0f, next, next_bytes, nullptr, slopes, softcap, out_f32, nullptr, 0, stream);
 }

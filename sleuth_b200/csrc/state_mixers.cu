@@ -50,7 +50,7 @@ __global__ void __launch_bounds__(256) causal_conv_kernel(const float* __restric
 // The same for steps of many tokens and up to four taps: a thread takes four (VEC) neighbouring channels, or one, and walks
 // kConvTile tokens with the last inputs in registers, so every input is read once; eight tokens' loads are under way before the
 // first is used. Where the tile crosses into another sequence the window is filled from that sequence's state.
-constexpr int kConvTile = 32;
+constexpr int kConvTile = 16;
 
 template <int TAPS, int VEC>
 __global__ void __launch_bounds__(128) causal_conv_tile_kernel(const float* __restrict__ in, long long in_stride,

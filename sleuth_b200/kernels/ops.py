@@ -449,7 +449,7 @@ def attention_tc(q, k_pool, v_pool, out, seq_start, past, counts, block_table, m
 def attention_decode(q, k_pool, v_pool, out, seq_start, past, block_table, heads: int, kv_heads: int, head_dim: int,
                      window: int, scale: float, splits: int, scratch, stream=None, qkv=None, qkv_kv_heads: int = 0,
                      bias=None, q_gain=None, k_gain=None, cos=None, sin=None, eps: float = 1e-6, next_read=None,
-                     sinks=None, slopes=None, softcap: float = 0.0, out_f32: bool = False) -> None:
+                     sinks=None, slopes=None, softcap: float = 0.0, out_f32: bool = False, gate=None) -> None:
     """Tensor-core attention for a step in which every sequence brings one token (split-KV).
 
     With ``qkv`` (the raw fused projection ``[n, (heads + 2 * qkv_kv_heads) * head_dim]``) the kernel also does what
@@ -457,7 +457,9 @@ def attention_decode(q, k_pool, v_pool, out, seq_start, past, block_table, heads
     ``qkv_kv_heads == kv_heads``, the write of its key and value into the cache; ``q`` is then not read.
     ``next_read``: a tensor that the kernel after this one reads and no kernel writes (a weight matrix); the blocks
     ask the L2 cache for it once their own pages are on their way. ``slopes`` / ``softcap``: the score rules of
-    ``attention_scored``, with post-processed queries only."""
+    ``attention_scored``, with post-processed queries only. ``gate``: float32 rows of heads * head_dim pre-activations (possibly a
+    view of wider rows); the result is multiplied by their sigmoid."""
+    _need(gate is None or not (slopes is not None or softcap or out_f32), "attention (decode): a gate goes with the plain score rules")
     _cuda(q, k_pool, v_pool, out, seq_start, past, block_table, scratch, qkv, bias, q_gain, k_gain, cos, sin, slopes)
     _sinks_ok(sinks, heads)
     _slopes_ok(slopes, heads, sinks)
@@ -488,7 +490,7 @@ def attention_decode(q, k_pool, v_pool, out, seq_start, past, block_table, heads
                int(splits), _p(scratch), 0 if scratch is None else scratch.numel(), _p(counters),
                0 if counters is None else counters.numel(), _p(qkv), int(qkv_kv_heads), _p(bias), _p(q_gain), _p(k_gain),
                _p(cos), _p(sin), float(eps), _p(next_read) if _nbytes(next_read) else None, _nbytes(next_read),
-               _p(sinks), stream if stream is not None else current_stream())
+               _p(sinks), _p(gate), 0 if gate is None else _rows_f32(gate, heads * head_dim, "attention (decode) gate"), stream if stream is not None else current_stream())
 
 
 _COUNTERS: dict = {}

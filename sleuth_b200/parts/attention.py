@@ -72,7 +72,8 @@ class GQAAttention(Part):
             raise ValueError(f"attention: gate {spec.gate!r} is not 'none' or 'channel'")
         if spec.chunk < 0 or spec.chunk and spec.window or spec.sinks and spec.unit_sink:
             raise ValueError(f"attention: chunk {spec.chunk} and window {spec.window} (one of them), learned sinks or a unit sink (one of them)")
-        self.reach = -spec.chunk if spec.chunk else spec.window         # the signed window of the cache and the kernels
+        # the signed window of the cache and the kernels (a chunk longer than any sequence is as good as 2^29 positions)
+        self.reach = -min(spec.chunk, 1 << 29) if spec.chunk else spec.window
         self.gated = spec.gate == "channel"
         self.wide = (self.value_dim != spec.head_dim or self.whole_norm or getattr(self.position, "neighbours", False) or self.gated)
         # The tensor-core attention kernels take keys and values of one width, 64 or 128. A bfloat16 run of the wide form
@@ -163,8 +164,9 @@ class GQAAttention(Part):
         return KVRequest(s.kv_heads, self.key_run, self.reach, 0 if self.value_run == self.key_run else self.value_run)
 
     # ---- one step ----
-    def _attend(self, q, y, b, view, table, ws):
-        """Attention of the step's (post-processed) queries over the cache into ``y``; the kernel by dtype and step shape."""
+    def _attend(self, q, y, b, view, table, ws, gate=None):
+        """Attention of the step's (post-processed) queries over the cache into ``y``, times the sigmoid of ``gate`` if given; the
+        kernel by dtype and step shape. Single tokens on the tensor cores gate in the attention kernel itself."""
         s = self.spec
         hd, vd = self.key_run, self.value_run
         flash = ops.flash_supported(hd, self.ctx.dtype) and vd == hd
@@ -177,7 +179,8 @@ class GQAAttention(Part):
             scratch = ws.take((floats,), torch.float32) if floats else None
             ops.attention_decode(q, view.k_pool, view.v_pool, y, b.seq_start, b.past, table, s.heads, s.kv_heads,
                                  hd, view.window, self.scale, splits, scratch, b.stream, sinks=self.sinks,
-                                 next_read=self.o.weight)
+                                 next_read=self.o.weight, gate=gate)
+            return
         elif use_tc_attention(s.heads, s.kv_heads, hd, self.ctx.dtype, b.max_count, self.scale):
             ops.attention_tc(q, view.k_pool, view.v_pool, y, b.seq_start, b.past, b.counts, table, b.max_count,
                              s.heads, s.kv_heads, hd, view.window, self.scale, b.stream, max_keys=b.max_len,
@@ -185,6 +188,8 @@ class GQAAttention(Part):
         else:
             ops.attention_prefill(q, view.k_pool, view.v_pool, y, b.seq_start, b.past, b.counts, table, b.max_count,
                                   s.heads, s.kv_heads, hd, view.window, self.scale, b.stream, sinks=self.sinks)
+        if gate is not None:
+            ops.sigmoid_gate(y, gate, b.stream)
 
     def lead_weight(self):
         return self.qkv.weight if self.qkv is not None else None
@@ -275,9 +280,7 @@ class GQAAttention(Part):
                           s.heads, s.kv_heads, self.key_run, self.value_run, rot, self.position.neighbours, self.whole_norm,
                           s.qk_norm_eps, b.stream, norm_dim=s.head_dim, bias=self.bias)
         y = ws.take((T, s.heads * self.value_run), self.ctx.dtype)
-        self._attend(q, y, b, view, table, ws)
-        if self.gated:
-            ops.sigmoid_gate(y, qkv[:, n_qkv:], b.stream)
+        self._attend(q, y, b, view, table, ws, gate=qkv[:, n_qkv:] if self.gated else None)
         self.o.forward(y, ws=ws, stream=b.stream, next_read=getattr(b, "next_read", None), **result_target(b, x))
 
 

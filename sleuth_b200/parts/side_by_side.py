@@ -1,6 +1,7 @@
 """Two mixers side by side: both read the same normed input, each delivers into a float32 buffer of its own, and one
 kernel joins the two results into the stream (``SideBySideSpec``): half the sum of the two after an RMS norm each with a
-gain of its own, or a weighted sum (which a layer whose closing kernel can form it asks for unjoined, ``b.pair_wanted``). The pair's cache entry is a bundle of the two mixers' requests, so an attention's
+gain of its own, or a weighted sum (which a layer whose closing kernel can form it asks for unjoined,
+``b.pair_wanted``). The pair's cache entry is a bundle of the two mixers' requests, so an attention's
 pages and a recurrence's state of one layer are taken, freed and reused together.
 
 The two mixers need nothing from each other. In a step that brings one token a sequence, where each is a chain of short

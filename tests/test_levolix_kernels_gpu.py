@@ -294,6 +294,26 @@ def test_a_loud_key_at_a_chunks_first_position_and_just_in_front_of_it(path, dty
     chunk_case(path, dtype, H, G, d, dv, [edge + 1, 66], [edge, 65], size, edge - 1)
 
 
+@pytest.mark.parametrize("d,splits", [(64, 1), (64, 4), (128, 3)])
+def test_single_tokens_are_gated_in_the_attention_kernel(d, splits):
+    o = ops()
+    H, G, n = 6, 2, 3
+    g = torch.Generator().manual_seed(d + splits)
+    pasts = [200, 63, 0]
+    k_pool, v_pool = (torch.randn(12, G, 64, d, generator=g).to(torch.bfloat16).to(DEV) for _ in range(2))
+    table = i32([[3, 1, 7, 5], [0, 2, 4, 6], [8, 9, 10, 11]])
+    q = torch.randn(n, H, d, generator=g).to(torch.bfloat16).to(DEV)
+    _, _, start = batch_tables([1] * n, pasts)
+    rows = torch.randn(n, H * d + 8, generator=g).to(DEV)
+    outs = []
+    for gate in (None, rows[:, 8:]):
+        out = torch.empty(n, H * d, dtype=torch.bfloat16, device=DEV)
+        scratch = torch.empty(max(o.decode_scratch_floats(n, H, d, splits), 1), device=DEV)
+        o.attention_decode(q, k_pool, v_pool, out, start, i32(pasts), table, H, G, d, -100, 0.2, splits, scratch, sinks=torch.zeros(H, device=DEV), gate=gate)
+        outs.append(out.float())
+    torch.testing.assert_close(outs[1], outs[0] * torch.sigmoid(rows[:, 8:]), rtol=2e-2, atol=2e-3)
+
+
 def test_the_one_in_the_denominator_counts_where_scores_are_low():
     """With every score far below zero almost nothing is attended to; a softmax without the one would return a mean."""
     o = ops()
