@@ -349,18 +349,18 @@ __global__ void __launch_bounds__(128) chunk_solve_kernel(ScanArgs a) {
     reinterpret_cast<float4*>(wt)[i] = *reinterpret_cast<const float4*>(KT + (i >> 4) * kPad + (i & 15) * 4);
 }
 
-// grid (slices of PS value columns, H, sequences), 256 threads: walks the sequence's chunks with its slice of the state; leaves
+// grid (slices of PS value columns, H, sequences), TH threads: walks the sequence's chunks with its slice of the state; leaves
 // every chunk's start state in `starts`, u in `out` (delta rule) and the last state in the slot. Both products run as 4 x 2 (RN x 2)
 // outputs a thread with the inner dimension cut into KS pieces whose partial sums meet in shared memory; behind them a thread owns
-// elements tid, tid + 256, ... of the chunk's u and of the state. The next chunk's W, k and values are on their way meanwhile.
-template <int RN, int PS, bool DELTA>
-__global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
+// elements tid, tid + TH, ... of the chunk's u and of the state. The next chunk's W, k and values are on their way meanwhile.
+template <int RN, int PS, int TH, bool DELTA>
+__global__ void __launch_bounds__(TH) chunk_state_kernel(ScanArgs a) {
   pdl_enter();
   extern __shared__ __align__(16) float sm[];
   constexpr int NP = 16 * RN;          // rows of the state, padded
   constexpr int CG = PS / 2;           // pairs of columns
-  constexpr int KS = 16 / CG;          // pieces of the inner dimension
-  constexpr int OS = NP * PS / 256, OU = kChunk * PS / 256;      // elements of the state and of u that a thread owns
+  constexpr int KS = TH / (16 * CG);   // pieces of the inner dimension
+  constexpr int OS = (NP * PS + TH - 1) / TH, OU = (kChunk * PS + TH - 1) / TH;      // elements of the state and of u that a thread owns
   constexpr int PARTS = KS * (NP > kChunk ? NP : kChunk) * PS;
   float* sS = sm;                      // [NP][PS]
   float* sV = sS + NP * PS;            // [64][PS]: u times the decay to the chunk's end
@@ -378,29 +378,29 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
   const size_t out_stride = (size_t)a.H * P;
   const float log_fixed = DELTA ? 0.0f : fmaxf(a.log_decay[h], -1e30f);
   if (DELTA && NP > N)                 // W's rows beyond N stay zero in every chunk
-    for (int i = tid; i < 2 * NP * kChunk; i += 256) sW[i] = 0.0f;
-  // element e = tid + 256 r of the state: (row part e / (16 PS), row group (e / PS) % 16, column e % PS) -> row group * RN + part
+    for (int i = tid; i < 2 * NP * kChunk; i += TH) sW[i] = 0.0f;
+  // element e = tid + TH r of the state: (row part e / (16 PS), row group (e / PS) % 16, column e % PS) -> row group * RN + part
   auto state_row = [&](int e) { return ((e / PS) & 15) * RN + e / (16 * PS); };
   float* st = a.state + (((size_t)a.slots[seq] * a.H + h) * N) * P + c0;
   float S[OS];
 #pragma unroll
   for (int r = 0; r < OS; ++r) {
-    const int e = tid + 256 * r, n = state_row(e), p = e % PS;
+    const int e = tid + TH * r, n = state_row(e), p = e % PS;
     S[r] = n < N && p < cols ? st[(size_t)n * P + p] : 0.0f;
-    sS[n * PS + p] = S[r];
+    if (e < NP * PS) sS[n * PS + p] = S[r];
   }
   __syncthreads();
   auto fetch = [&](int c) {            // one commit group a chunk
     if (c < live) {
       const int cnt = min(kChunk, total - c * kChunk), b = c & 1;
-      copy_tile<256, kChunk, NP>(sK + b * kChunk * NP, a.k + (size_t)(first + c * kChunk) * a.k_stride + (size_t)g * N, a.k_stride, cnt, N, a.vec);
+      copy_tile<TH, kChunk, NP>(sK + b * kChunk * NP, a.k + (size_t)(first + c * kChunk) * a.k_stride + (size_t)g * N, a.k_stride, cnt, N, a.vec);
       if (DELTA) {
         const size_t at = ((size_t)seq * a.chunks + c) * a.H + h;
         float* wd = sW + b * NP * kChunk;
         const float* ws = a.w + at * N * kChunk;
 #pragma unroll
-        for (int m = 0; m < NP / 16; ++m) {
-          const int i = (tid + m * 256) * 4;
+        for (int m = 0; m < (NP * kChunk / 4 + TH - 1) / TH; ++m) {
+          const int i = (tid + m * TH) * 4;
           if (i < N * kChunk) copy_async(wd + i, ws + i, true, true);
         }
         if (tid < kChunk / 4 + 1) copy_async(sE + b * (kChunk + 4) + tid * 4, a.ends + at * (kChunk + 4) + tid * 4, true, true);
@@ -417,7 +417,7 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
     const int t0 = first + c * kChunk, cnt = c < live ? min(kChunk, total - c * kChunk) : 0;
 #pragma unroll
     for (int r = 0; r < OU; ++r) {
-      const int e = tid + 256 * r, i = u_row(e), p = e % PS;
+      const int e = tid + TH * r, i = u_row(e), p = e % PS;
       uv[r] = i < cnt && p < cols ? (DELTA ? a.out[(size_t)(t0 + i) * out_stride + (size_t)h * P + c0 + p] : a.v[(size_t)(t0 + i) * a.v_stride + (size_t)h * P + c0 + p]) : 0.0f;
     }
   };
@@ -432,7 +432,7 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
     float* start = a.starts + ((((size_t)seq * a.chunks + c) * a.H + h) * N) * P + c0;
 #pragma unroll
     for (int r = 0; r < OS; ++r) {
-      const int e = tid + 256 * r, n = state_row(e), p = e % PS;
+      const int e = tid + TH * r, n = state_row(e), p = e % PS;
       if (n < N && p < cols) start[(size_t)n * P + p] = S[r];
     }
     if (DELTA) {
@@ -456,7 +456,7 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
       __syncthreads();
 #pragma unroll
       for (int r = 0; r < OU; ++r) {
-        const int e = tid + 256 * r, i = u_row(e), p = e % PS;
+        const int e = tid + TH * r, i = u_row(e), p = e % PS;
         float sum = 0.0f;
 #pragma unroll
         for (int k = 0; k < KS; ++k) sum += sP[k * kChunk * PS + e];
@@ -466,8 +466,8 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
     }
 #pragma unroll
     for (int r = 0; r < OU; ++r) {
-      const int e = tid + 256 * r, i = u_row(e), p = e % PS;
-      sV[i * PS + p] = uv[r] * ends[i];
+      const int e = tid + TH * r, i = u_row(e), p = e % PS;
+      if (e < kChunk * PS) sV[i * PS + p] = uv[r] * ends[i];
     }
     __syncthreads();
     values(c + 1);
@@ -503,7 +503,8 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
     const float keep = ends[kChunk];
 #pragma unroll
     for (int r = 0; r < OS; ++r) {
-      const int e = tid + 256 * r;
+      const int e = tid + TH * r;
+      if (e >= NP * PS) break;
       float sum = 0.0f;
 #pragma unroll
       for (int k = 0; k < KS; ++k) sum += sP[k * NP * PS + e];
@@ -513,16 +514,32 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ScanArgs a) {
   }
 #pragma unroll
   for (int r = 0; r < OS; ++r) {
-    const int e = tid + 256 * r, n = state_row(e), p = e % PS;
+    const int e = tid + TH * r, n = state_row(e), p = e % PS;
     if (n < N && p < cols) st[(size_t)n * P + p] = S[r];
   }
 }
 
-__host__ __device__ constexpr int out_keys_floats(int N) {
-  return N * kPad > (N + 15) / 16 * 16 * kOutCols ? N * kPad : (N + 15) / 16 * 16 * kOutCols;
+// Row length of the output kernel's tiles of queries and keys: a multiple of 4 floats, and 4 more than a multiple of 32, so that
+// 16-byte pieces of eight neighbouring rows lie in different banks.
+__host__ __device__ constexpr int out_row(int N) { return (N + 31) / 32 * 32 + 4; }
+__host__ __device__ constexpr int out_keys_floats(int N) {      // the keys' tile, later the start state [N rounded up to 16][64]
+  return kChunk * out_row(N) > (N + 15) / 16 * 16 * kOutCols ? kChunk * out_row(N) : (N + 15) / 16 * 16 * kOutCols;
 }
 
-// grid (chunks, H * slices of 64 value columns, sequences), 256 threads (4 rows x 4 columns each): the chunk's outputs.
+// A [64, N] tile of rows into shared memory (row length `ld`), zeros behind N up to a multiple of 4 and in rows from cnt on.
+__device__ __forceinline__ void copy_rows(float* dst, int ld, const float* src, long long stride, int cnt, int N, bool vec) {
+  const int step = vec ? 4 : 1, per = ((N + 3) & ~3) / step;
+  const int r0 = threadIdx.x / 32;                         // a warp a row, eight rows at a time
+  for (int r = r0; r < kChunk; r += 8)
+    for (int c = threadIdx.x & 31; c < per; c += 32) {
+      const bool in = r < cnt && c * step < N;
+      copy_async(dst + r * ld + c * step, in ? src + (size_t)r * stride + c * step : src, in, vec);
+    }
+}
+
+// grid (chunks, H * slices of 64 value columns, sequences), 256 threads: the chunk's outputs. A warp takes 16 rows x 32 columns,
+// lanes 4 x 8; a lane's four rows lie 4 apart, its four keys 8 apart (scores) and its four value columns side by side. Inner
+// dimensions go four values at a time: 8 loads of 16 bytes for 64 multiply-adds.
 __global__ void __launch_bounds__(256) chunk_out_kernel(ScanArgs a) {
   pdl_enter();
   extern __shared__ __align__(16) float sm[];
@@ -531,87 +548,98 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(ScanArgs a) {
   const int chunk = blockIdx.x, h = blockIdx.y / slices, c0 = (blockIdx.y % slices) * kOutCols, seq = blockIdx.z, tid = threadIdx.x;
   const int t0 = a.seq_start[seq] + chunk * kChunk, cnt = min(kChunk, a.seq_start[seq + 1] - t0);
   if (cnt <= 0) return;
-  const int N = a.N, P = a.P, g = h / (a.H / a.G), cols = min(kOutCols, P - c0);
-  float* QT = sm;                      // [N][kPad]
-  float* KT = QT + N * kPad;           // [N][kPad], then the start state [N rounded up to 16][64]
-  float* AT = KT + out_keys_floats(N); // [64][kPad]: AT[j][i] = e^(L_i - L_j) (q_i . k_j)
-  float* V = AT + kChunk * kPad;       // [64][64]: u
+  const int N = a.N, N4 = (N + 3) & ~3, P = a.P, g = h / (a.H / a.G), cols = min(kOutCols, P - c0), ld = out_row(N);
+  float* Q = sm;                       // [64][ld]
+  float* K = Q + kChunk * ld;          // [64][ld], then the start state [N4][64]
+  float* A = K + out_keys_floats(N);   // [64][kPad]: A[i][j] = e^(L_i - L_j) (q_i . k_j)
+  float* V = A + kChunk * kPad;        // [64][64]: u
+  copy_rows(Q, ld, a.q + (size_t)t0 * a.q_stride + (size_t)g * N, a.q_stride, cnt, N, a.vec);
+  copy_rows(K, ld, a.k + (size_t)t0 * a.k_stride + (size_t)g * N, a.k_stride, cnt, N, a.vec);
+  asm volatile("cp.async.commit_group;" ::: "memory");
   const bool from_out = a.beta != nullptr;
   const float* u = from_out ? a.out + (size_t)t0 * ((size_t)a.H * P) + (size_t)h * P + c0 : a.v + (size_t)t0 * a.v_stride + (size_t)h * P + c0;
   copy_tile<256, kChunk, kOutCols>(V, u, from_out ? (long long)a.H * P : a.v_stride, cnt, cols, a.vec);
-  load_transposed<256>(QT, a.q + (size_t)t0 * a.q_stride + (size_t)g * N, a.q_stride, cnt, N);
-  load_transposed<256>(KT, a.k + (size_t)t0 * a.k_stride + (size_t)g * N, a.k_stride, cnt, N);
+  asm volatile("cp.async.commit_group;" ::: "memory");
   if (tid < 32) chunk_log_sums(a, t0, cnt, h, L);
+  asm volatile("cp.async.wait_group 1;" ::: "memory");
   __syncthreads();
-  // a warp takes 16 rows x 32 columns: lanes 4 x 8
   const int warp = tid >> 5, lane = tid & 31;
-  const int i0 = (warp >> 1) * 16 + (lane >> 3) * 4, j0 = (warp & 1) * 32 + (lane & 7) * 4;      // 4 rows; 4 keys, later 4 columns
+  const int i0 = (warp >> 1) * 16 + (lane >> 3), j0 = (warp & 1) * 32 + (lane & 7), p0 = (warp & 1) * 32 + (lane & 7) * 4;
   const int rows_end = (warp >> 1) * 16 + 16;               // keys from here on are behind all rows of the warp
   {
-    float4 acc[4];                     // [key]: the four rows
+    float acc[4][4];                   // [row][key]
 #pragma unroll
-    for (int j = 0; j < 4; ++j) acc[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.0f;
     if ((warp & 1) * 32 < rows_end) {
-#pragma unroll 4
-      for (int n = 0; n < N; ++n) {
-        const float4 q4 = *reinterpret_cast<const float4*>(QT + n * kPad + i0), k4 = *reinterpret_cast<const float4*>(KT + n * kPad + j0);
-        fma4(acc[0], k4.x, q4);
-        fma4(acc[1], k4.y, q4);
-        fma4(acc[2], k4.z, q4);
-        fma4(acc[3], k4.w, q4);
-      }
-      float2 li[4];
+#pragma unroll 2
+      for (int n = 0; n < N4; n += 4) {
+        float4 q4[4], k4[4];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) li[i] = L[i0 + i];
+        for (int i = 0; i < 4; ++i) q4[i] = *reinterpret_cast<const float4*>(Q + (i0 + 4 * i) * ld + n);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int jj = j0 + j;
-        const float2 lj = L[jj];
-        acc[j].x = i0 >= jj ? acc[j].x * decay_between(li[0], lj) : 0.0f;
-        acc[j].y = i0 + 1 >= jj ? acc[j].y * decay_between(li[1], lj) : 0.0f;
-        acc[j].z = i0 + 2 >= jj ? acc[j].z * decay_between(li[2], lj) : 0.0f;
-        acc[j].w = i0 + 3 >= jj ? acc[j].w * decay_between(li[3], lj) : 0.0f;
+        for (int j = 0; j < 4; ++j) k4[j] = *reinterpret_cast<const float4*>(K + (j0 + 8 * j) * ld + n);
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            acc[i][j] = fmaf(q4[i].w, k4[j].w, fmaf(q4[i].z, k4[j].z, fmaf(q4[i].y, k4[j].y, fmaf(q4[i].x, k4[j].x, acc[i][j]))));
       }
     }
+    float2 lj[4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) *reinterpret_cast<float4*>(AT + (j0 + j) * kPad + i0) = acc[j];
+    for (int j = 0; j < 4; ++j) lj[j] = L[j0 + 8 * j];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 li = L[i0 + 4 * i];
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        A[(i0 + 4 * i) * kPad + j0 + 8 * j] = i0 + 4 * i >= j0 + 8 * j ? acc[i][j] * decay_between(li, lj[j]) : 0.0f;
+    }
   }
   __syncthreads();                     // the keys have been read: their place takes the start state
   const float* start = a.starts + ((((size_t)seq * a.chunks + chunk) * a.H + h) * N) * P + c0;
-  for (int n = 0; n < N; n += 16) copy_tile<256, 16, kOutCols>(KT + n * kOutCols, start + (size_t)n * P, P, N - n, cols, a.vec);
+  for (int n = 0; n < N; n += 16) copy_tile<256, 16, kOutCols>(K + n * kOutCols, start + (size_t)n * P, P, N - n, cols, a.vec);
   asm volatile("cp.async.commit_group;" ::: "memory");
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
   float4 o[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) o[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-  auto accumulate = [&](const float* rows, const float* cols4) {
-    const float4 r4 = *reinterpret_cast<const float4*>(rows), v4 = *reinterpret_cast<const float4*>(cols4);
-    fma4(o[0], r4.x, v4);
-    fma4(o[1], r4.y, v4);
-    fma4(o[2], r4.z, v4);
-    fma4(o[3], r4.w, v4);
+  auto accumulate = [&](const float* rows, int row_len, const float* col) {      // four inner values
+    float4 r4[4], v4[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) r4[i] = *reinterpret_cast<const float4*>(rows + 4 * i * row_len);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) v4[k] = *reinterpret_cast<const float4*>(col + k * kOutCols);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      fma4(o[i], r4[i].x, v4[0]);
+      fma4(o[i], r4[i].y, v4[1]);
+      fma4(o[i], r4[i].z, v4[2]);
+      fma4(o[i], r4[i].w, v4[3]);
+    }
   };
-#pragma unroll 4
-  for (int n = 0; n < N; ++n) accumulate(QT + n * kPad + i0, KT + n * kOutCols + j0);
+#pragma unroll 2
+  for (int n = 0; n < N4; n += 4) accumulate(Q + i0 * ld + n, ld, K + n * kOutCols + p0);
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    const float f = decay_since_start(L[i0 + i]);
+    const float f = decay_since_start(L[i0 + 4 * i]);
     o[i] = make_float4(o[i].x * f, o[i].y * f, o[i].z * f, o[i].w * f);
   }
-#pragma unroll 4
-  for (int j = 0; j < rows_end; ++j) accumulate(AT + j * kPad + i0, V + j * kOutCols + j0);
+#pragma unroll 2
+  for (int j = 0; j < rows_end; j += 4) accumulate(A + i0 * kPad + j, kPad, V + j * kOutCols + p0);
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    if (i0 + i >= cnt) continue;
-    float* dst = a.out + (size_t)(t0 + i0 + i) * ((size_t)a.H * P) + (size_t)h * P + c0 + j0;
+    const int row = i0 + 4 * i;
+    if (row >= cnt) continue;
+    float* dst = a.out + (size_t)(t0 + row) * ((size_t)a.H * P) + (size_t)h * P + c0 + p0;
     const float r[4] = {o[i].x * a.q_scale, o[i].y * a.q_scale, o[i].z * a.q_scale, o[i].w * a.q_scale};
-    if (a.vec && j0 + 3 < cols) {
+    if (a.vec && p0 + 3 < cols) {
       *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
     } else {
 #pragma unroll
       for (int e = 0; e < 4; ++e)
-        if (j0 + e < cols) dst[e] = r[e];
+        if (p0 + e < cols) dst[e] = r[e];
     }
   }
 }
@@ -762,21 +790,21 @@ extern "C" long long slb_state_scan_scratch_floats(int n_seqs, int max_count, in
   return starts + (delta ? (long long)n_seqs * chunks * H * ((long long)N * kChunk + kChunk + 4) : 0);
 }
 
-template <int RN, int PS>
+template <int RN, int PS, int TH>
 static int launch_chunk_state(const ScanArgs& a, cudaStream_t s) {
-  const dim3 grid((a.P + PS - 1) / PS, a.H, a.n_seqs), block(256);
+  const dim3 grid((a.P + PS - 1) / PS, a.H, a.n_seqs), block(TH);
   const bool delta = a.beta != nullptr;
-  constexpr int NP = 16 * RN, KS = 32 / PS;
+  constexpr int NP = 16 * RN, KS = TH / (8 * PS);
   const int smem = (NP * PS + kChunk * PS + KS * (NP > kChunk ? NP : kChunk) * PS + 2 * (kChunk + 4) + (delta ? 4 : 2) * kChunk * NP) * 4;
   static bool configured[2] = {false, false};
   if (!configured[delta]) {
-    const cudaError_t e = delta ? cudaFuncSetAttribute(chunk_state_kernel<RN, PS, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)
-                                : cudaFuncSetAttribute(chunk_state_kernel<RN, PS, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    const cudaError_t e = delta ? cudaFuncSetAttribute(chunk_state_kernel<RN, PS, TH, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)
+                                : cudaFuncSetAttribute(chunk_state_kernel<RN, PS, TH, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return fail(2, "state_scan: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));
     configured[delta] = true;
   }
-  if (delta) launch(chunk_state_kernel<RN, PS, true>, grid, block, (size_t)smem, s, a);
-  else launch(chunk_state_kernel<RN, PS, false>, grid, block, (size_t)smem, s, a);
+  if (delta) launch(chunk_state_kernel<RN, PS, TH, true>, grid, block, (size_t)smem, s, a);
+  else launch(chunk_state_kernel<RN, PS, TH, false>, grid, block, (size_t)smem, s, a);
   return check_launch("state_scan (states)");
 }
 
@@ -828,12 +856,12 @@ extern "C" int slb_state_scan(const float* q, long long q_stride, const float* k
     // slices of 8 columns while all their blocks can be resident at once, else of 16 (with 128 rows one block fits an SM)
     const bool narrow = (long long)((P + 7) / 8) * H * n_seqs <= (long long)sm_count() * (N <= 64 ? 2 : 1);
     int rc;
-    if (N <= 32) rc = narrow ? launch_chunk_state<2, 8>(a, s) : launch_chunk_state<2, 16>(a, s);
-    else if (N <= 64) rc = narrow ? launch_chunk_state<4, 8>(a, s) : launch_chunk_state<4, 16>(a, s);
-    else rc = narrow ? launch_chunk_state<8, 8>(a, s) : launch_chunk_state<8, 16>(a, s);
+    if (N <= 32) rc = narrow ? launch_chunk_state<2, 8, 256>(a, s) : launch_chunk_state<2, 16, 256>(a, s);
+    else if (N <= 64) rc = narrow ? launch_chunk_state<4, 8, 512>(a, s) : launch_chunk_state<4, 16, 512>(a, s);
+    else rc = narrow ? launch_chunk_state<8, 8, 512>(a, s) : launch_chunk_state<8, 16, 512>(a, s);
     if (rc) return rc;
   }
-  const int smem = (N * kPad + out_keys_floats(N) + kChunk * kPad + kChunk * kOutCols) * 4;
+  const int smem = (kChunk * out_row(N) + out_keys_floats(N) + kChunk * kPad + kChunk * kOutCols) * 4;
   static int most_out = 0;
   if (smem > most_out) {
     const cudaError_t e = cudaFuncSetAttribute(chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
