@@ -660,26 +660,31 @@ struct StateTokenArgs {
   const int* slots;
   const float* gain;                   // [P] or null (ones)
   void* out;                           // [n, H * P] in the run dtype
-  int H, G, N, P, PB;                  // PB: P rounded up to whole warps
+  int H, G, N, P, PB;                  // PB: columns of a block, rounded up to whole warps
+  int team;                            // blocks of a cluster that share a head, 64 columns each
   float q_scale, unit_eps, eps;
 };
 
-constexpr int kStateThreads = 512;
+constexpr int kStateThreads = 512, kTeamCols = 64, kTeamMost = 8;
 
-// grid (H, sequences). Thread (r, c), c = tid % PB, holds rows r, r + R, ... of column c of the head's state.
+// grid (H * team, sequences), clusters of `team` blocks. Thread (r, c), c = tid % PB, holds rows r, r + R, ... of column c of its
+// block's part of the head's state; the blocks of a head meet once, for the head's sum of squares.
 template <typename T, int NB>
-__global__ void __launch_bounds__(kStateThreads) state_token_kernel(StateTokenArgs a) {
+__global__ void __launch_bounds__(kStateThreads, NB <= 16 ? 2 : 1) state_token_kernel(StateTokenArgs a) {
   pdl_enter();
   __shared__ float sq[256], sk[256], part_k[kStateThreads], part_q[kStateThreads], scratch[33];
-  const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
+  __shared__ float team_ss[kTeamMost];
+  if (a.team > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");      // this block runs
+  const int h = blockIdx.x / a.team, rank = blockIdx.x % a.team, seq = blockIdx.y, tid = threadIdx.x;
   const int N = a.N, P = a.P, R = blockDim.x / a.PB;
-  const int c = tid % a.PB, r = tid / a.PB;
+  const int cb = tid % a.PB, r = tid / a.PB;               // column within the block
+  const int c = rank * kTeamCols + cb;
   const bool mine = c < P && r < R;
   const int g = h / (a.H / a.G);
   float* st = a.state + ((size_t)a.slots[seq] * a.H + h) * N * P + c;
   float S[NB];
 #pragma unroll
-  for (int j = 0; j < NB; ++j) S[j] = mine && r + j * R < N ? st[(size_t)(r + j * R) * P] : 0.0f;
+  for (int j = 0; j < NB; ++j) S[j] = mine && r + j * R < N ? st[(r + j * R) * P] : 0.0f;
   const float v = mine ? a.v[(size_t)seq * a.v_stride + (size_t)h * P + c] : 0.0f;
   const float gate = mine && r == 0 ? a.gate[(size_t)seq * a.gate_stride + (size_t)h * P + c] : 0.0f;
   const float gain = mine && r == 0 && a.gain ? a.gain[c] : 1.0f;
@@ -721,33 +726,56 @@ __global__ void __launch_bounds__(kStateThreads) state_token_kernel(StateTokenAr
       dk = fmaf(S[j], sk[n], dk);
       dq = fmaf(S[j], sq[n], dq);
     }
+    if ((j & 3) == 3) asm volatile("" ::: "memory");       // four rows' keys and queries at a time in registers, not all
   }
   part_k[tid] = dk;
   part_q[tid] = dq;
   __syncthreads();
   dk = dq = 0.0f;
   for (int i = 0; i < R; ++i) {
-    dk += part_k[i * a.PB + c];
-    dq += part_q[i * a.PB + c];
+    dk += part_k[i * a.PB + cb];
+    dq += part_q[i * a.PB + cb];
   }
   const float u = a.decay != nullptr ? v : beta * (v - dk);
+  float* back = st;
+  asm volatile("" : "+l"(back));       // the addresses are worked out again instead of being kept since the loads
 #pragma unroll
   for (int j = 0; j < NB; ++j) {
     const int n = r + j * R;
-    if (mine && n < N) st[(size_t)n * P] = fmaf(sk[n], u, S[j]);
+    if (mine && n < N) back[n * P] = fmaf(sk[n], u, S[j]);
+    if ((j & 3) == 3) asm volatile("" ::: "memory");
   }
   const float o = mine && r == 0 ? fmaf(u, kq, dq) : 0.0f;   // S_new^T q = (decayed S)^T q + u (k . q)
-  const float inv = 1.0f / sqrtf(block_sum(o * o, scratch) / (float)P + a.eps);
+  float ss = block_sum(o * o, scratch);
+  if (a.team > 1) {
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");                              // every block of the head runs
+    if (tid < a.team) {
+      uint32_t at;
+      asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(at) : "r"((uint32_t)__cvta_generic_to_shared(&team_ss[rank])), "r"(tid));
+      asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(at), "f"(ss) : "memory");
+    }
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    ss = 0.0f;
+    for (int i = 0; i < a.team; ++i) ss += team_ss[i];
+  }
+  const float inv = 1.0f / sqrtf(ss / (float)P + a.eps);
   if (mine && r == 0) ((T*)a.out)[((size_t)seq * a.H + h) * P + c] = from_f32<T>(o * inv * gain * silu_of(gate));
+}
+
+template <typename T, int NB>
+static void launch_state_token_nb(const StateTokenArgs& a, int n, cudaStream_t s) {
+  const dim3 grid(a.H * a.team, n), block(kStateThreads);
+  if (a.team > 1) launch_clusters(pdl_mode() == 1, a.team, state_token_kernel<T, NB>, grid, block, 0, s, a);
+  else launch(state_token_kernel<T, NB>, grid, block, 0, s, a);
 }
 
 template <typename T>
 static void launch_state_token(const StateTokenArgs& a, int n, int rows, cudaStream_t s) {
-  const dim3 grid(a.H, n), block(kStateThreads);
-  if (rows <= 8) launch(state_token_kernel<T, 8>, grid, block, 0, s, a);
-  else if (rows <= 16) launch(state_token_kernel<T, 16>, grid, block, 0, s, a);
-  else if (rows <= 32) launch(state_token_kernel<T, 32>, grid, block, 0, s, a);
-  else launch(state_token_kernel<T, 64>, grid, block, 0, s, a);
+  if (rows <= 4) launch_state_token_nb<T, 4>(a, n, s);
+  else if (rows <= 8) launch_state_token_nb<T, 8>(a, n, s);
+  else if (rows <= 16) launch_state_token_nb<T, 16>(a, n, s);
+  else launch_state_token_nb<T, 32>(a, n, s);
 }
 
 }  // namespace slb
@@ -874,9 +902,7 @@ extern "C" int slb_state_scan(const float* q, long long q_stride, const float* k
 
 // 1 when slb_state_token takes heads of N key and P value channels.
 extern "C" int slb_state_token_supported(int N, int P) {
-  if (N < 1 || N > 256 || P < 1 || P > kStateThreads) return 0;
-  const int PB = (P + 31) / 32 * 32, R = kStateThreads / PB;
-  return (N + R - 1) / R <= 64;
+  return N >= 1 && N <= 256 && P >= 1 && P <= kTeamCols * kTeamMost;
 }
 
 extern "C" int slb_state_token(const float* q, long long q_stride, const float* k, long long k_stride, const float* v, long long v_stride,
@@ -890,9 +916,11 @@ extern "C" int slb_state_token(const float* q, long long q_stride, const float* 
               "state_token: a fixed decay, or the delta rule's step sizes and strengths");
   SLB_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= N && (rot == 0 || (decay != nullptr && cos != nullptr && sin != nullptr)), "state_token: %d rotated channels of %d", rot, N);
   if (n == 0) return 0;
-  const int PB = (P + 31) / 32 * 32, R = kStateThreads / PB;
+  const int team = P <= kTeamCols ? 1 : (P + kTeamCols - 1) / kTeamCols;
+  const int PB = team > 1 ? kTeamCols : (P + 31) / 32 * 32, R = kStateThreads / PB;
+  SLB_REQUIRE((long long)H * team < 65536, "state_token: too many heads (%d)", H);
   const StateTokenArgs a{q, k, v, q_stride, k_stride, v_stride, gate, gate_stride, decay, raw_beta, raw_step, raw_stride, dt_bias, a_log,
-                         cos, sin, tok_pos, rot / 2, neighbours, state, slots, gain, out, H, G, N, P, PB, q_scale, unit_eps, eps};
+                         cos, sin, tok_pos, rot / 2, neighbours, state, slots, gain, out, H, G, N, P, PB, team, q_scale, unit_eps, eps};
   if (dtype == kF32) launch_state_token<float>(a, n, (N + R - 1) / R, (cudaStream_t)stream);
   else if (dtype == kBF16) launch_state_token<__nv_bfloat16>(a, n, (N + R - 1) / R, (cudaStream_t)stream);
   else return fail(1, "state_token: unknown dtype %d", dtype);

@@ -48,21 +48,19 @@ __global__ void __launch_bounds__(256) causal_conv_kernel(const float* __restric
 }
 
 // The same for steps of many tokens and up to four taps: a thread takes four (VEC) neighbouring channels, or one, and walks
-// kConvTile tokens with the last inputs in registers, so every input is read once; eight tokens' loads are under way before the
+// `tile` tokens with the last inputs in registers, so every input is read once; eight tokens' loads are under way before the
 // first is used. Where the tile crosses into another sequence the window is filled from that sequence's state.
-constexpr int kConvTile = 16;
-
 template <int TAPS, int VEC>
 __global__ void __launch_bounds__(128) causal_conv_tile_kernel(const float* __restrict__ in, long long in_stride,
                                                                const float* __restrict__ w, const float* __restrict__ bias,
                                                                const float* __restrict__ state, const int* __restrict__ slots,
                                                                const int* __restrict__ tok_seq, const int* __restrict__ seq_start,
                                                                float* __restrict__ out, long long out_stride, int tokens, int C,
-                                                               int act) {
+                                                               int act, int tile) {
   pdl_enter();
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
   if (c >= C) return;
-  const int t0 = blockIdx.y * kConvTile, t1 = min(tokens, t0 + kConvTile);
+  const int t0 = blockIdx.y * tile, t1 = min(tokens, t0 + tile);
   float wt[VEC][TAPS], bs[VEC], win[TAPS - 1][VEC];
 #pragma unroll
   for (int e = 0; e < VEC; ++e) {
@@ -504,16 +502,18 @@ extern "C" int slb_causal_conv(const float* in, long long in_stride, const float
     return check_launch("causal_conv (short steps)");
   }
   const long long total = (long long)tokens * C;
-  if (taps >= 2 && taps <= 4 && tokens >= 64 && tokens / kConvTile < 65535) {
+  if (taps >= 2 && taps <= 4 && tokens >= 64 && tokens / 16 < 65535) {
     const bool vec = C % 4 == 0 && in_stride % 4 == 0 && out_stride % 4 == 0 && ((uintptr_t)in | (uintptr_t)out | (uintptr_t)state) % 16 == 0;
-    const dim3 grid((C / (vec ? 4 : 1) + 127) / 128, (tokens + kConvTile - 1) / kConvTile), block(128);
+    // 32 tokens a thread where that still gives every SM two blocks, else 16 (a window is filled again for every tile)
+    const int across = (C / (vec ? 4 : 1) + 127) / 128, tile = (long long)across * (tokens / 32) >= 2ll * sm_count() ? 32 : 16;
+    const dim3 grid(across, (tokens + tile - 1) / tile), block(128);
     const float* st = state;
-    if (taps == 2 && vec) launch(causal_conv_tile_kernel<2, 4>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
-    else if (taps == 2) launch(causal_conv_tile_kernel<2, 1>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
-    else if (taps == 3 && vec) launch(causal_conv_tile_kernel<3, 4>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
-    else if (taps == 3) launch(causal_conv_tile_kernel<3, 1>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
-    else if (vec) launch(causal_conv_tile_kernel<4, 4>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
-    else launch(causal_conv_tile_kernel<4, 1>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act);
+    if (taps == 2 && vec) launch(causal_conv_tile_kernel<2, 4>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act, tile);
+    else if (taps == 2) launch(causal_conv_tile_kernel<2, 1>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act, tile);
+    else if (taps == 3 && vec) launch(causal_conv_tile_kernel<3, 4>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act, tile);
+    else if (taps == 3) launch(causal_conv_tile_kernel<3, 1>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act, tile);
+    else if (vec) launch(causal_conv_tile_kernel<4, 4>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act, tile);
+    else launch(causal_conv_tile_kernel<4, 1>, grid, block, 0, s, in, in_stride, w, bias, st, slots, tok_seq, seq_start, out, out_stride, tokens, C, act, tile);
   } else {
     launch(causal_conv_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, in, in_stride, w, bias,
            (const float*)state, slots, tok_seq, seq_start, out, out_stride, tokens, C, taps, act);

@@ -136,7 +136,7 @@ def test_equal_keys_and_extreme_decays(strength):
     scan_case(2, 2, 32, 16, True, [200, 64], [[], [64], [90, 30]], make=make)
 
 
-@pytest.mark.parametrize("N,P,H,G", [(12, 10, 3, 1), (64, 64, 4, 2), (128, 128, 2, 1), (40, 200, 2, 2), (136, 96, 1, 1), (256, 64, 1, 1)])
+@pytest.mark.parametrize("N,P,H,G", [(12, 10, 3, 1), (64, 64, 4, 2), (128, 128, 2, 1), (40, 200, 2, 2), (136, 96, 1, 1), (256, 64, 1, 1), (128, 256, 2, 2), (33, 130, 1, 1), (16, 520, 1, 1)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("delta", [True, False])
 def test_a_single_token_step_from_the_projections_to_the_gated_heads(N, P, H, G, dtype, delta):
@@ -144,7 +144,7 @@ def test_a_single_token_step_from_the_projections_to_the_gated_heads(N, P, H, G,
     if not delta:
         G = H
     if not o.state_token_supported(N, P):
-        assert N * P > 64 * 480
+        assert P > 512
         return
     g = torch.Generator().manual_seed(N + P)
     n, eps, T = 3, 1e-5, 4
